@@ -199,6 +199,91 @@ class ModelConfig:
 DeepSeekConfig = ModelConfig  # reference name
 
 
+@dataclass
+class LayerSpec:
+    """One entry of a layer list: which mixer the layer has, the mixer's sizes and constants, and its feed-forward (or ``None``)."""
+    type: str
+    mixer: Dict[str, Any]
+    mlp: Optional[Dict[str, Any]] = None
+
+
+@dataclass
+class VimodraConfig:
+    """Architecture of a Vimodra model: a list of layers with their own mixers (``latent_attention`` | ``delta``), Dynamic-Tanh norms
+    around every sublayer, and an optional range of layers that is run several times per token (``models/vimodra.py``)."""
+    vocab_size: int
+    hidden_size: int
+    layers: List[LayerSpec]
+    norm_eps: float = 1e-5
+    loop_start: int = 0
+    loop_stop: int = 0
+    loop_times: int = 0            # 0: no loop
+    seq_length: int = 4096         # default cache length and size of the rotary tables (both grow on demand)
+
+    MIXERS = {"latent_attention": ("heads", "dim", "rot_dim", "vdim", "kv_rank", "q_rank"),
+              "delta": ("heads", "kv_heads", "dim", "vdim", "conv")}
+
+    def __post_init__(self):
+        self.validate()
+
+    @property
+    def num_layers(self) -> int:
+        return len(self.layers)
+
+    def runs(self) -> List[Any]:
+        """[(layer, pass)] in the order the layers are run; ``pass`` is the loop pass that begins with this run, else ``None``."""
+        n = self.num_layers
+        if not self.loop_times:
+            return [(i, None) for i in range(n)]
+        body = [(i, t if i == self.loop_start else None) for t in range(self.loop_times) for i in range(self.loop_start, self.loop_stop)]
+        return [(i, None) for i in range(self.loop_start)] + body + [(i, None) for i in range(self.loop_stop, n)]
+
+    def validate(self) -> None:
+        if self.vocab_size < 1 or self.hidden_size < 1 or not self.layers:
+            raise ValueError("vocab_size, hidden_size and the layer list must not be empty")
+        if self.loop_times and not 0 <= self.loop_start < self.loop_stop <= self.num_layers:
+            raise ValueError(f"loop {self.loop_start}..{self.loop_stop} does not fit {self.num_layers} layers")
+        for i, layer in enumerate(self.layers):
+            if layer.type not in self.MIXERS:
+                raise ValueError(f"layer {i}: unknown mixer {layer.type!r} (known: {sorted(self.MIXERS)})")
+            m = layer.mixer
+            missing = [k for k in self.MIXERS[layer.type] if not isinstance(m.get(k), int) or m[k] < 1]
+            if missing:
+                raise ValueError(f"layer {i} ({layer.type}): sizes {missing} are missing or not positive")
+            if layer.type == "latent_attention":
+                rot = m.get("rot") or {}
+                if m["rot_dim"] % 2 or rot.get("dims", m["rot_dim"]) != m["rot_dim"]:
+                    raise ValueError(f"layer {i}: the rotated part must be even and rotated as a whole")
+                if "base" not in rot or "scale" not in m:
+                    raise ValueError(f"layer {i}: rot.base and scale are needed")
+                if (m.get("mask") or {}).get("size", 1) < 1:
+                    raise ValueError(f"layer {i}: the window must hold at least the token itself")
+                if m["vdim"] > 512:
+                    raise ValueError(f"layer {i}: value heads of up to 512 dimensions are built")
+            elif m["heads"] % m["kv_heads"]:
+                raise ValueError(f"layer {i}: heads {m['heads']} not divisible by kv_heads {m['kv_heads']}")
+            elif m["dim"] > 256:
+                raise ValueError(f"layer {i}: state rows of up to 256 are built")
+            if layer.mlp is not None and (layer.mlp.get("kind", "dense") != "dense" or int(layer.mlp.get("ff", 0)) < 1):
+                raise ValueError(f"layer {i}: unknown feed-forward {layer.mlp!r}")
+
+    @classmethod
+    def from_dict(cls, d: Dict[str, Any]) -> "VimodraConfig":
+        """From the keys of a model folder's ``config.json``."""
+        loop = d.get("loop") or {}
+        return cls(vocab_size=int(d["vocab"]), hidden_size=int(d["width"]), norm_eps=float((d.get("norm") or {}).get("eps", 1e-5)),
+                   layers=[LayerSpec(l["type"], dict(l["mixer"]), dict(l["mlp"]) if l.get("mlp") else None) for l in d["layers"]],
+                   loop_start=int(loop.get("start", 0)), loop_stop=int(loop.get("stop", 0)), loop_times=int(loop.get("times", 0)) if loop else 0,
+                   **({"seq_length": int(d["seq_length"])} if "seq_length" in d else {}))
+
+    def to_dict(self) -> Dict[str, Any]:
+        d: Dict[str, Any] = {"architecture": "Vimodra", "vocab": self.vocab_size, "width": self.hidden_size, "norm": {"eps": self.norm_eps},
+                             "seq_length": self.seq_length, "layers": [dataclasses.asdict(l) for l in self.layers]}
+        if self.loop_times:
+            d["loop"] = {"start": self.loop_start, "stop": self.loop_stop, "times": self.loop_times}
+        return d
+
+
 # --------------------------------------------------------------------------- #
 # Run configuration
 # --------------------------------------------------------------------------- #

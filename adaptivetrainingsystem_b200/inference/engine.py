@@ -20,7 +20,8 @@ from typing import Callable, Dict, Iterator, List, Optional, Sequence
 
 import torch
 
-from ..models.transformer import DeepSeekTransformer, KVCache
+from ..models.cache import SequenceCache
+from ..models.transformer import DeepSeekTransformer
 
 GENERATION_MODES: Dict[str, Dict[str, float]] = {
     "standard": dict(temperature=0.8, top_p=0.9, top_k=50, repetition_penalty=1.1),
@@ -158,19 +159,20 @@ class GenerationEngine:
         return n
 
     @torch.no_grad()
-    def prefill(self, input_ids: torch.Tensor, cache: KVCache) -> torch.Tensor:
-        """Runs the prompt, fills the cache, returns the logits of the last position [B, V]."""
+    def prefill(self, input_ids: torch.Tensor, cache: SequenceCache) -> torch.Tensor:
+        """Runs the prompt (or its next portion, after what the cache holds), fills the cache, returns the logits of the last position
+        [B, V]."""
         logits = self.model(input_ids, cache=cache, last_token_only=True, return_aux_loss=False)
         return logits[:, -1, :]
 
     @torch.no_grad()
-    def decode_step(self, tokens: torch.Tensor, cache: KVCache) -> torch.Tensor:
+    def decode_step(self, tokens: torch.Tensor, cache: SequenceCache) -> torch.Tensor:
         """tokens [B] -> logits [B, V] for the next position."""
         logits = self.model(tokens.view(-1, 1), cache=cache, last_token_only=True, return_aux_loss=False)
         return logits[:, -1, :]
 
     @torch.no_grad()
-    def graph_decoder(self, cache: KVCache) -> "GraphDecoder":
+    def graph_decoder(self, cache: SequenceCache) -> "GraphDecoder":
         """Capture one decode step (all layers, launch-bound at batch <= 64) into a CUDA graph bound to ``cache``."""
         return GraphDecoder(self.model, cache)
 
@@ -285,28 +287,28 @@ class GraphDecoder:
     """One decode step of the whole model as a CUDA graph.  A decode step at serving batch sizes is a few hundred small
     launches whose host-side cost exceeds their device time; replaying a captured graph removes that cost.  Everything that
     changes from step to step lives in device memory: the input tokens (a static buffer), the cache fill level and the RoPE
-    positions (``KVCache.device_lengths`` / ``device_positions``, advanced inside the graph)."""
+    positions (``SequenceCache.device_lengths`` / ``device_positions``, advanced inside the graph for the rows in ``device_active``)."""
 
-    def __init__(self, model: DeepSeekTransformer, cache: KVCache, warmup: int = 2):
+    def __init__(self, model: DeepSeekTransformer, cache: SequenceCache, warmup: int = 2):
         self.model, self.cache = model, cache
-        dev = cache.k[0].device
-        B = cache.k[0].shape[0]
+        dev, B = cache.device, cache.batch
         self.tokens = torch.zeros(B, 1, dtype=torch.long, device=dev)
         start = cache.length
         cache.enable_device_lengths()
+        cache.device_active.zero_()   # the warm-up steps must not move recurrent states or rings on
         side = torch.cuda.Stream(device=dev)
         side.wait_stream(torch.cuda.current_stream(dev))
         with torch.cuda.stream(side), torch.no_grad():
             for _ in range(warmup):  # builds every lazily created buffer / function attribute outside the capture
                 self._run()
         torch.cuda.current_stream(dev).wait_stream(side)
-        cache.device_lengths.fill_(start)   # the warm-up wrote K / V beyond the fill level: harmless, rewind the counters
-        cache.device_positions.fill_(start)
+        # (the warm-up wrote K / V beyond the fill level: harmless)
         self.graph = torch.cuda.CUDAGraph()
         with torch.cuda.graph(self.graph), torch.no_grad():
             self.logits = self._run()
         cache.device_lengths.fill_(start)   # capture does not execute, but keep the invariant explicit
         cache.device_positions.fill_(start)
+        cache.device_active.fill_(1)
 
     def _run(self) -> torch.Tensor:
         logits = self.model(self.tokens, cache=self.cache, last_token_only=True, return_aux_loss=False)[:, -1, :]

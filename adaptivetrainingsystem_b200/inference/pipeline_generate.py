@@ -18,6 +18,7 @@ from typing import List, Optional
 import torch
 import torch.distributed as dist
 
+from ..models.cache import SequenceCache
 from ..models.transformer import KVCache
 from ..parallel.pipeline import PipelineStage
 from .engine import SamplingParams, sample_next
@@ -27,13 +28,10 @@ class _StageCache(KVCache):
     """A cache that holds buffers for this stage's layers only (the other entries are empty placeholders)."""
 
     def __init__(self, num_layers: int, own: range, batch: int, max_len: int, n_kv: int, head_dim: int, dtype, device):
+        SequenceCache.__init__(self, batch, max_len, device)
         empty = torch.empty(0, dtype=dtype, device=device)
         self.k = [torch.zeros(batch, max_len, n_kv, head_dim, dtype=dtype, device=device) if i in own else empty for i in range(num_layers)]
         self.v = [torch.zeros(batch, max_len, n_kv, head_dim, dtype=dtype, device=device) if i in own else empty for i in range(num_layers)]
-        self.length = 0
-        self.max_len = max_len
-        self.device_lengths = None
-        self.device_positions = None
 
 
 class PipelineGenerator:

@@ -1,12 +1,13 @@
 """Continuous batching: a fixed pool of cache rows, requests of any length admitted and retired between decode steps.
 
-The pool is one ``KVCache`` of ``max_batch`` rows and one captured decode step over it (``GraphDecoder``).  A row is a
-sequence slot handed out by ``KVSlotManager``.  Every call of :meth:`ContinuousBatcher.step`
+The rows live in a :class:`SequencePool` (one cache of ``max_batch`` rows and one captured decode step over it).  Every call of
+:meth:`ContinuousBatcher.step`
 
-1. admits waiting requests into free rows: the prompt is prefilled straight into the row (a one-row view of the pool's cache), the
-   row's length and RoPE position are set in device memory, and the first token is sampled from the prefill logits;
-2. replays the decode graph once for all rows (each row attends over its own length; a free row has length 0 and its output is
-   ignored), samples one token per row in one launch;
+1. admits waiting requests into free rows and prefills them straight into the row (a one-row view of the pool's cache), either the
+   whole prompt at once or, with ``prefill_chunk``, at most that many prompt tokens per step, so that a long prompt does not hold up the
+   rows that are decoding; the first token is sampled from the logits of the prompt's last position;
+2. replays the decode graph once for all rows (each row at its own length; rows that are free or still in their prompt come out
+   unchanged and their output is ignored), samples one token per row in one launch;
 3. retires rows that produced a stop token or their token budget and frees their slots.
 
 The reference's own generator serves one sequence at a time and re-runs the context for every token (``Chat.py:355-465``); its
@@ -20,8 +21,8 @@ from typing import Dict, List, Optional, Sequence
 
 import torch
 
-from ..models.transformer import KVCache
-from .engine import GenerationEngine, GraphDecoder, KVSlotManager, SamplingParams, sample_next
+from .engine import GenerationEngine, SamplingParams, sample_next
+from .pool import SequencePool
 
 
 @dataclass
@@ -31,41 +32,26 @@ class Request:
     max_new_tokens: int
     tokens: List[int] = field(default_factory=list)
     slot: int = -1
+    prefilled: int = 0                        # prompt tokens the row already holds
     done: bool = False
 
 
-class _RowView(KVCache):
-    """One row of the pool's cache presented as a cache of batch 1 (prefill writes land in the pool)."""
-
-    def __init__(self, pool: KVCache, row: int):  # noqa: D401  (no buffers of its own)
-        self.k = [t[row:row + 1] for t in pool.k]
-        self.v = [t[row:row + 1] for t in pool.v]
-        self.length = 0
-        self.max_len = pool.max_len
-        self.device_lengths = None
-        self.device_positions = None
-
-
 class ContinuousBatcher:
-    def __init__(self, engine: GenerationEngine, max_batch: int = 64, max_len: int = 2048, params: Optional[SamplingParams] = None):
+    def __init__(self, engine: GenerationEngine, max_batch: int = 64, max_len: int = 2048, params: Optional[SamplingParams] = None,
+                 prefill_chunk: Optional[int] = None):
         self.engine, self.model = engine, engine.model
         self.params = params or SamplingParams.from_mode("greedy")
         self.max_batch, self.max_len = max_batch, max_len
+        self.prefill_chunk = prefill_chunk
         self.device = next(self.model.parameters()).device
-        if self.device.type != "cuda":
-            raise RuntimeError("continuous batching replays a CUDA graph of the decode step: a CUDA device is required")
         if getattr(self.model, "_ep_comm", None) is not None:
             # admission prefills one request on one rank, which the expert-parallel exchange (a collective of all ranks) cannot serve
             raise RuntimeError("continuous batching runs on one GPU (or on replicas): the model must not be expert-parallel")
-        self.cache = self.model.make_cache(max_batch, max_len)
-        self.slots = KVSlotManager(max_batch)
-        self.decoder = GraphDecoder(self.model, self.cache)        # captured once; rows come and go underneath it
-        self.cache.device_lengths.zero_()
-        self.cache.device_positions.zero_()
-        self.active = torch.zeros(max_batch, dtype=torch.int32, device=self.device)     # 1 for rows that hold a live sequence
-        self.last = torch.zeros(max_batch, dtype=torch.long, device=self.device)        # the token each row feeds next
+        self.pool = SequencePool(self.model, max_batch, max_len)
+        self.cache, self.slots = self.pool.cache, self.pool.slots
         self.history = torch.zeros(max_batch, self.params.repetition_window, dtype=torch.long, device=self.device)
-        self.by_slot: Dict[int, Request] = {}
+        self.by_slot: Dict[int, Request] = {}          # rows that decode
+        self.prefilling: List[Request] = []            # rows still in their prompt, oldest first
         self.waiting: List[Request] = []
         self.finished: Dict[int, Request] = {}
         self._next_id = 0
@@ -86,30 +72,41 @@ class ContinuousBatcher:
 
     @property
     def pending(self) -> int:
-        return len(self.waiting) + len(self.by_slot)
+        return len(self.waiting) + len(self.prefilling) + len(self.by_slot)
 
     # -- one scheduling step ---------------------------------------------------------------------------------------
     @torch.no_grad()
     def _admit(self) -> None:
-        while self.waiting and self.slots.available:
-            r = self.waiting.pop(0)
-            slot = int(self.slots.alloc(1)[0])
-            ids = r.prompt.to(self.device).view(1, -1)
-            logits = self.engine.prefill(ids, _RowView(self.cache, slot))
-            n = ids.shape[1]
-            self.cache.device_lengths[slot] = n
-            self.cache.device_positions[slot] = n
-            w = self.history.shape[1]
-            self.history[slot].fill_(int(ids[0, 0]))      # left padding of a short prompt repeats its first token
-            self.history[slot, -min(n, w):] = ids[0, -min(n, w):]
-            first = sample_next(logits, self.params, self.history[slot:slot + 1], self.generator)
-            self.last[slot:slot + 1] = first
-            self.history[slot] = torch.roll(self.history[slot], -1)
-            self.history[slot, -1:] = first
-            r.slot = slot
-            self.by_slot[slot] = r
-            self.active[slot] = 1
-            self._accept(slot, int(first))
+        budget = self.prefill_chunk or (1 << 62)       # prompt tokens this step may still run
+        while budget > 0:
+            if not self.prefilling:
+                if not (self.waiting and self.pool.available):
+                    return
+                r = self.waiting.pop(0)
+                r.slot = self.pool.open()
+                self.prefilling.append(r)
+            r = self.prefilling[0]
+            n = min(budget, r.prompt.numel() - r.prefilled)
+            budget -= n
+            part = r.prompt[r.prefilled:r.prefilled + n]
+            r.prefilled += n
+            done = r.prefilled == r.prompt.numel()
+            logits = self.pool.extend(r.slot, part, active=done)
+            if done:
+                self.prefilling.pop(0)
+                self._first_token(r, logits)
+
+    def _first_token(self, r: Request, logits: torch.Tensor) -> None:
+        slot, ids, w = r.slot, r.prompt.to(self.device), self.history.shape[1]
+        n = ids.numel()
+        self.history[slot].fill_(int(r.prompt[0]))     # left padding of a short prompt repeats its first token
+        self.history[slot, -min(n, w):] = ids[-min(n, w):]
+        first = sample_next(logits, self.params, self.history[slot:slot + 1], self.generator)
+        self.pool.last[slot:slot + 1] = first
+        self.history[slot] = torch.roll(self.history[slot], -1)
+        self.history[slot, -1:] = first
+        self.by_slot[slot] = r
+        self._accept(slot, int(first))
 
     def _accept(self, slot: int, token: int) -> None:
         """Host-side bookkeeping of one generated token (the device-side state was updated for all rows at once)."""
@@ -122,10 +119,7 @@ class ContinuousBatcher:
         r = self.by_slot.pop(slot)
         r.done = True
         self.finished[r.rid] = r
-        self.active[slot] = 0
-        self.cache.device_lengths[slot] = 0
-        self.cache.device_positions[slot] = 0
-        self.slots.free(torch.tensor([slot]))
+        self.pool.close(slot)
 
     @torch.no_grad()
     def step(self) -> int:
@@ -134,13 +128,9 @@ class ContinuousBatcher:
         live = sorted(self.by_slot)
         if not live:
             return 0
-        self.decoder.tokens.copy_(self.last.view(-1, 1))
-        self.decoder.graph.replay()
-        # the captured step advanced every row's counters: free rows go back to zero so that they never walk off their buffer
-        self.cache.device_lengths.mul_(self.active)
-        self.cache.device_positions.mul_(self.active)
-        nxt_dev = sample_next(self.decoder.logits, self.params, self.history, self.generator)
-        self.last.copy_(nxt_dev)
+        logits = self.pool.decode(live)
+        nxt_dev = sample_next(logits, self.params, self.history, self.generator)
+        self.pool.last.copy_(nxt_dev)
         self.history = torch.roll(self.history, -1, dims=1)
         self.history[:, -1] = nxt_dev
         nxt = nxt_dev.tolist()                       # the one device-to-host read of the step

@@ -2,3 +2,7 @@ from .transformer import (DeepSeekTransformer, TransformerBlock, GroupedQueryAtt
                           MoEFFNLayer, MoDRouter, MoDFFN, RMSNorm, LayerNorm, RotaryEmbedding, KVCache,
                           estimate_parameters)
 from ..config import ModelConfig, DeepSeekConfig
+from ..config import LayerSpec, VimodraConfig
+from .cache import LayerStateCache, SequenceCache
+from .vimodra import Vimodra
+from .registry import MODELS, ModelEntry, load_model, read_config, register_model

@@ -20,7 +20,7 @@ reference's state-dict names (``layers.N.self_attn.q_proj.weight``, ``layers.N.f
 from __future__ import annotations
 
 import math
-from typing import Any, Dict, List, Optional, Tuple
+from typing import Any, Dict, List, Optional, Sequence, Tuple
 
 import torch
 import torch.nn as nn
@@ -31,6 +31,7 @@ from ..config import ModelConfig
 from .. import ops
 from ..ops import moe as moe_ops
 from ..ops import mod as mod_ops
+from .cache import SequenceCache
 
 
 class RMSNorm(nn.Module):
@@ -85,29 +86,19 @@ class RotaryEmbedding(nn.Module):
         return self.cos[:length], self.sin[:length]
 
 
-class KVCache:
-    """Contiguous per-layer K/V buffers ``[B, max_len, Hkv, D]`` plus the filled length."""
+class KVCache(SequenceCache):
+    """Contiguous per-layer K/V buffers ``[B, max_len, Hkv, D]``."""
 
     def __init__(self, num_layers: int, batch: int, max_len: int, n_kv: int, head_dim: int, dtype, device):
+        super().__init__(batch, max_len, device)
         self.k = [torch.zeros(batch, max_len, n_kv, head_dim, dtype=dtype, device=device) for _ in range(num_layers)]
         self.v = [torch.zeros(batch, max_len, n_kv, head_dim, dtype=dtype, device=device) for _ in range(num_layers)]
-        self.length = 0
-        self.max_len = max_len
-        # device-side copy of the fill level, used when the decode step is replayed from a CUDA graph (a Python integer
-        # would be frozen into the captured launches): per-sequence lengths for the attention kernel, positions for RoPE
-        self.device_lengths: Optional[torch.Tensor] = None
-        self.device_positions: Optional[torch.Tensor] = None
 
-    def enable_device_lengths(self) -> None:
-        dev = self.k[0].device
-        B = self.k[0].shape[0]
-        self.device_lengths = torch.full((B,), self.length, dtype=torch.int32, device=dev)
-        self.device_positions = torch.full((B,), self.length, dtype=torch.int32, device=dev)
-
-    def device_advance(self) -> None:
-        """One decoded token: called inside the captured step."""
-        self.device_lengths += 1
-        self.device_positions += 1
+    def row(self, i: int) -> "KVCache":
+        view = KVCache(0, 1, self.max_len, 0, 0, None, self.device)
+        view.k = [t[i:i + 1] for t in self.k]
+        view.v = [t[i:i + 1] for t in self.v]
+        return view
 
     def append(self, layer: int, k: torch.Tensor, v: torch.Tensor) -> Tuple[torch.Tensor, torch.Tensor]:
         n = k.shape[1]
@@ -116,12 +107,6 @@ class KVCache:
         self.k[layer][:, self.length:self.length + n] = k
         self.v[layer][:, self.length:self.length + n] = v
         return self.k[layer][:, : self.length + n], self.v[layer][:, : self.length + n]
-
-    def advance(self, n: int) -> None:
-        self.length += n
-
-    def reset(self) -> None:
-        self.length = 0
 
 
 class GroupedQueryAttention(nn.Module):
@@ -592,10 +577,13 @@ class DeepSeekTransformer(nn.Module):
 
     def forward(self, input_ids: torch.Tensor, attention_mask: Optional[torch.Tensor] = None,
                 return_hidden_states: bool = False, return_aux_loss: Optional[bool] = None,
-                cache: Optional[KVCache] = None, last_token_only: bool = False):
+                cache: Optional[KVCache] = None, last_token_only: bool = False, logits_at: Optional[Sequence[int]] = None):
+        """``last_token_only`` / ``logits_at``: the output head runs only on the last position / on these positions of ``input_ids``."""
         x, aux_losses = self.hidden_states(input_ids, attention_mask, cache, decode=cache is not None and input_ids.shape[1] == 1)
         if last_token_only:
             x = x[:, -1:, :]
+        elif logits_at is not None:
+            x = x[:, list(logits_at), :]
         logits = ops.linear(x, self.lm_head)
         if self.config.scale_lm_head_output:
             logits = logits / math.sqrt(self.config.hidden_size)

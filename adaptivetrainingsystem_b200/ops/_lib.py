@@ -15,7 +15,8 @@ import os
 import shutil
 import subprocess
 import threading
-from typing import List, Optional
+from concurrent.futures import ThreadPoolExecutor
+from typing import List, Optional, Sequence
 
 import torch
 
@@ -31,7 +32,9 @@ DEBUG_BUILD = os.environ.get("ATS_DEBUG_BUILD", "0") == "1"
 HOST_LIB = os.path.join(OUT_DIR, "libats_host.so")
 
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
-              "--use_fast_math", "-Xcompiler", "-fPIC", "-Xcompiler", "-fvisibility=hidden", "-shared"]
+              "-Xcompiler", "-fPIC", "-Xcompiler", "-fvisibility=hidden"]
+# Every source is compiled with --use_fast_math except these: their kernels also serve models that run in true 32-bit.
+PRECISE_MATH = {"dyt.cu", "latent_attention.cu", "delta_rule.cu"}
 # Kernels that may only run in single-GPU jobs (none at present) would be listed here and built into a
 # separate library so the main one never names a multicast load.
 SINGLE_GPU_ONLY: List[str] = []
@@ -59,43 +62,64 @@ def cuda_sources() -> List[str]:
     return sorted(s for s in glob.glob(os.path.join(CSRC, "*.cu")) if os.path.basename(s) not in SINGLE_GPU_ONLY)
 
 
-def build_debug(force: bool = False) -> None:
-    """The bounds-checking build: -DATS_DEBUG, relocatable device code (one report word shared by all translation units)."""
-    os.makedirs(OUT_DIR, exist_ok=True)
-    srcs = cuda_sources()
-    headers = glob.glob(os.path.join(CSRC, "*.cuh")) + glob.glob(os.path.join(CSRC, "*.h"))
-    if not (force or _stale(DEBUG_LIB, srcs + headers)):
-        return
+def _nvcc_or_raise() -> str:
     nvcc = _nvcc()
     if nvcc is None:
         raise RuntimeError("nvcc not found; cannot build the sm_100a kernels")
-    cmd = [nvcc] + NVCC_FLAGS + ["-DATS_DEBUG", "-rdc=true", "-I", CSRC, "-o", DEBUG_LIB + ".tmp"] + srcs
+    return nvcc
+
+
+def _compile_objects(srcs: List[str], tag: str, extra: List[str], force: bool, verbose: bool = False) -> List[str]:
+    """One object per source under ``_C/obj_<tag>``, compiled in parallel; up-to-date objects are kept."""
+    nvcc = _nvcc_or_raise()
+    headers = glob.glob(os.path.join(CSRC, "*.cuh")) + glob.glob(os.path.join(CSRC, "*.h"))
+    obj_dir = os.path.join(OUT_DIR, f"obj_{tag}")
+    os.makedirs(obj_dir, exist_ok=True)
+
+    def one(src: str) -> str:
+        obj = os.path.join(obj_dir, os.path.basename(src)[:-3] + ".o")
+        if not (force or _stale(obj, [src] + headers)):
+            return obj
+        math = [] if os.path.basename(src) in PRECISE_MATH else ["--use_fast_math"]
+        cmd = [nvcc] + NVCC_FLAGS + math + extra + ["-I", CSRC, "-c", "-o", obj + ".tmp.o", src]
+        if verbose:
+            cmd[1:1] = ["-Xptxas", "-v"]
+        r = subprocess.run(cmd, capture_output=True, text=True)
+        if r.returncode != 0:
+            raise RuntimeError(f"nvcc failed on {os.path.basename(src)}:\n" + r.stdout + r.stderr)
+        if verbose:
+            print(r.stderr)
+        os.replace(obj + ".tmp.o", obj)
+        return obj
+    with ThreadPoolExecutor(max_workers=min(len(srcs), os.cpu_count() or 4)) as pool:
+        return list(pool.map(one, srcs))
+
+
+def _link(target: str, objects: List[str], extra: List[str]) -> None:
+    cmd = [_nvcc_or_raise()] + NVCC_FLAGS + extra + ["-shared", "-o", target + ".tmp"] + objects
     r = subprocess.run(cmd, capture_output=True, text=True)
     if r.returncode != 0:
-        raise RuntimeError("nvcc (debug build) failed:\n" + r.stdout + r.stderr)
-    os.replace(DEBUG_LIB + ".tmp", DEBUG_LIB)
+        raise RuntimeError("nvcc (link) failed:\n" + r.stdout + r.stderr)
+    os.replace(target + ".tmp", target)
+
+
+def _build_library(target: str, srcs: List[str], tag: str, extra: List[str], force: bool, verbose: bool = False) -> None:
+    headers = glob.glob(os.path.join(CSRC, "*.cuh")) + glob.glob(os.path.join(CSRC, "*.h"))
+    if force or _stale(target, srcs + headers):
+        _link(target, _compile_objects(srcs, tag, extra, force, verbose), extra)
+
+
+def build_debug(force: bool = False) -> None:
+    """The bounds-checking build: -DATS_DEBUG, relocatable device code (one report word shared by all translation units)."""
+    os.makedirs(OUT_DIR, exist_ok=True)
+    _build_library(DEBUG_LIB, cuda_sources(), "debug", ["-DATS_DEBUG", "-rdc=true"], force)
 
 
 def build(force: bool = False, verbose: bool = False) -> None:
     """Compile every native source for sm_100a (cross-compiles without a GPU)."""
     os.makedirs(OUT_DIR, exist_ok=True)
-    srcs = cuda_sources()
-    headers = glob.glob(os.path.join(CSRC, "*.cuh")) + glob.glob(os.path.join(CSRC, "*.h"))
-    if srcs and (force or _stale(CUDA_LIB, srcs + headers)):
-        nvcc = _nvcc()
-        if nvcc is None:
-            raise RuntimeError("nvcc not found; cannot build the sm_100a kernels")
-        extra = os.environ.get("ATS_NVCC_EXTRA", "").split()  # e.g. -DATS_AB_SPLIT=4 for kernel tuning experiments
-        cmd = [nvcc] + NVCC_FLAGS + extra + ["-I", CSRC, "-o", CUDA_LIB + ".tmp"] + srcs
-        if verbose:
-            cmd.insert(1, "-Xptxas")
-            cmd.insert(2, "-v")
-        r = subprocess.run(cmd, capture_output=True, text=True)
-        if r.returncode != 0:
-            raise RuntimeError("nvcc failed:\n" + r.stdout + r.stderr)
-        if verbose:
-            print(r.stderr)
-        os.replace(CUDA_LIB + ".tmp", CUDA_LIB)
+    extra = os.environ.get("ATS_NVCC_EXTRA", "").split()  # e.g. -DATS_AB_SPLIT=4 for kernel tuning experiments
+    _build_library(CUDA_LIB, cuda_sources(), "release", extra, force, verbose)
     host_srcs = sorted(glob.glob(os.path.join(CSRC, "host", "*.cpp")))
     if host_srcs and (force or _stale(HOST_LIB, host_srcs)):
         cxx = shutil.which("g++") or "g++"
@@ -104,6 +128,19 @@ def build(force: bool = False, verbose: bool = False) -> None:
         if r.returncode != 0:
             raise RuntimeError("g++ failed:\n" + r.stdout + r.stderr)
         os.replace(HOST_LIB + ".tmp", HOST_LIB)
+
+
+def load_for(sources: Sequence[str], name: str) -> ctypes.CDLL:
+    """The kernel library for a program that serves one model: the full library when it has been built, otherwise a library of
+    only the named ``csrc`` files (``libats_<name>.so``), so that a fresh checkout compiles what the model needs and no more."""
+    global _cuda
+    with _lock:
+        if _cuda is None and not DEBUG_BUILD and not os.path.exists(CUDA_LIB):
+            part = os.path.join(OUT_DIR, f"libats_{name}.so")
+            os.makedirs(OUT_DIR, exist_ok=True)
+            _build_library(part, [os.path.join(CSRC, s) for s in sources], "release", [], False)
+            _cuda = ctypes.CDLL(part)
+    return cuda_lib()
 
 
 def cuda_lib() -> ctypes.CDLL:

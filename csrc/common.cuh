@@ -377,6 +377,8 @@ __device__ __forceinline__ void ld_global_32B(const void* ptr, uint4& lo, uint4&
                : "l"(ptr)
                : "memory");
 }
+// tanh from one exponential and one fast division (absolute error of a few 1e-7); saturates at +-1 for large |x|.
+__device__ __forceinline__ float tanh_fast(float x) { return 1.f - __fdividef(2.f, 1.f + __expf(2.f * fminf(x, 40.f))); }
 __device__ __forceinline__ float silu_f(float x) { return x / (1.f + __expf(-x)); }
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll

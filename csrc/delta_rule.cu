@@ -1,0 +1,575 @@
+// Gated delta rule: a linear recurrence over a per-head matrix state S [dim, vdim] (fp32)
+//
+//   S <- g_t S;   u = beta_t (v_t - S^T k_t);   S <- S + k_t u^T;   o_t = S^T q_t
+//
+// with short causal convolutions (+ silu) on q, k, v, unit-length q and k, and an output norm with a silu gate.  `heads` value heads,
+// `kv_heads` query / key heads (head h uses query / key head h / (heads / kv_heads)).
+//
+// * delta_prep: convolutions and activations, reciprocal lengths of q and k (kept apart in fp32, the vectors stay in the element
+//   type), decay g and step size beta.  One warp per (token, head).
+// * delta_pairs + delta_scan: portions of a prompt.  The recurrence is advanced in groups of DC = 8 tokens: with S the state before the
+//   group, u_i = beta_i (v_i - G_i S^T k_i - sum_{j < i} D_ij (k_j . k_i) u_j), D_ij = g_{j+1} .. g_i, G_i = g_1 .. g_i, a unit lower
+//   triangular system whose 8 x 8 inverse does not depend on the value column; delta_pairs computes it (and the read-out
+//   coefficients) for all groups in parallel, so that the sequential kernel only does three products with the state per token.
+//   Columns of S are independent: eight lanes share a column (or two), everything in fp32 with packed fma.f32x2.
+// * delta_output: output norm over vdim, weight, silu gate.
+// * delta_step: one decoded token per sequence: state read once and written once, output norm and gate in the same launch.
+//
+// A sequence at position 0 starts from a zero state and zero convolution inputs whatever its buffers hold.
+#include "typed.cuh"
+
+namespace ats {
+
+struct DeltaArgs {
+  const void* proj;        // [B * L, ld]: q at 0, k at kv_heads * dim, v at 2 * kv_heads * dim; gate / a / b at the columns below
+  long long ld;
+  int g_col, a_col, b_col;
+  int B, L, H, KH, dim, vdim, taps, C;   // C = 2 * KH * dim + H * vdim convolved channels
+  const float* conv;       // [C, taps]
+  const float* neg_rate;   // [H] -exp(A_log)
+  const float* dt_bias;    // [H]
+  void* tail;              // [B, taps - 1, C] last inputs of the convolutions (oldest first)
+  long long tail_bs;
+  int pos0;
+  const int* lengths;      // decoding: position per sequence
+  const int* active;       // decoding: rows with 0 leave tail and state alone
+  void* mixed;             // [B * L, Cp] convolved q, k, v
+  long long ldm;
+  float* rlen;             // [B * L, 2 * KH] 1 / |q| (times dim^-1/2), 1 / |k|
+  float* gb;               // [B * L, 2 * H] decay, step size
+};
+
+template <typename T>
+__global__ void __launch_bounds__(256) delta_prep_kernel(const DeltaArgs p) {
+  pdl_prologue();
+  const int units = 2 * p.KH + p.H + 1, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const long long w = blockIdx.x * 8ll + warp;
+  if (w >= (long long)p.B * p.L * units) return;
+  const long long row = w / units;
+  const int unit = int(w % units), b = int(row / p.L), t = int(row % p.L);
+  const int pos0 = p.lengths ? p.lengths[b] : p.pos0;
+  const T* in = static_cast<const T*>(p.proj) + row * p.ld;
+  if (unit == units - 1) {  // decay and step size of every head
+    for (int h = lane; h < p.H; h += 32) {
+      const float a = Typed<T>::load(in + p.a_col + h) + p.dt_bias[h], bt = Typed<T>::load(in + p.b_col + h);
+      const float sp = a > 20.f ? a : log1pf(expf(a));
+      p.gb[row * 2 * p.H + h] = expf(p.neg_rate[h] * sp);
+      p.gb[row * 2 * p.H + p.H + h] = 1.f / (1.f + expf(-bt));
+    }
+    return;
+  }
+  const int width = unit < 2 * p.KH ? p.dim : p.vdim;
+  const int c0 = unit < 2 * p.KH ? unit * p.dim : 2 * p.KH * p.dim + (unit - 2 * p.KH) * p.vdim;
+  T* tail = static_cast<T*>(p.tail) + (long long)b * p.tail_bs;
+  T* out = static_cast<T*>(p.mixed) + row * p.ldm;
+  const bool keep = p.lengths && !(p.active && !p.active[b]);
+  float ss = 0.f;
+  for (int i = lane; i < width; i += 32) {
+    const int c = c0 + i;
+    const float* cw = p.conv + (long long)c * p.taps;
+    const T cur = in[c];
+    float acc = Typed<T>::load(&cur) * cw[p.taps - 1];
+    for (int j = 1; j < p.taps; ++j) {  // j tokens back
+      float x = 0.f;
+      if (t - j >= 0) x = Typed<T>::load(in - j * p.ld + c);
+      else if (pos0 > 0) x = Typed<T>::load(tail + (long long)(p.taps - 1 + t - j) * p.C + c);
+      acc += x * cw[p.taps - 1 - j];
+    }
+    if (keep) {  // decoding: shift the channel's inputs (this thread is the only one that touches them)
+      for (int j = 0; j < p.taps - 2; ++j) {
+        T v = tail[(long long)(j + 1) * p.C + c];
+        if (pos0 == 0) Typed<T>::store(&v, 0.f);
+        tail[(long long)j * p.C + c] = v;
+      }
+      if (p.taps > 1) tail[(long long)(p.taps - 2) * p.C + c] = cur;
+    }
+    const float y = acc * Typed<T>::sigmoid_(acc);
+    T yt;
+    Typed<T>::store(&yt, y);
+    out[c] = yt;
+    const float yr = Typed<T>::load(&yt);
+    ss += yr * yr;
+  }
+  if (unit < 2 * p.KH) {
+    ss = warp_sum(ss);
+    if (lane == 0) p.rlen[row * 2 * p.KH + unit] = (unit < p.KH ? 1.f / sqrtf(float(p.dim)) : 1.f) / sqrtf(ss + 1e-6f);
+  }
+}
+
+// After a portion: the last taps - 1 inputs of every channel (one thread per channel, oldest first, in place).
+template <typename T>
+__global__ void __launch_bounds__(256) delta_tail_kernel(const DeltaArgs p) {
+  pdl_prologue();
+  const int c = blockIdx.x * 256 + threadIdx.x, b = blockIdx.y, n = p.taps - 1;
+  if (c >= p.C) return;
+  T* tail = static_cast<T*>(p.tail) + (long long)b * p.tail_bs + c;
+  const T* in = static_cast<const T*>(p.proj) + (long long)b * p.L * p.ld + c;
+  for (int j = 0; j < n; ++j) {
+    const int t = p.L - n + j;
+    T v;
+    Typed<T>::store(&v, 0.f);
+    if (t >= 0) v = in[t * p.ld];
+    else if (p.pos0 > 0) v = tail[(long long)(n + t) * p.C];
+    tail[(long long)j * p.C] = v;
+  }
+}
+
+// ------------------------------------------------------------------------------------------------ portions
+constexpr int DC = 8;  // tokens per group
+
+struct ScanArgs {
+  const void* mixed;
+  long long ldm;
+  const float* rlen;
+  const float* gb;
+  float* coef;             // [B, groups, H, DC, 2 * DC]: inverse of the triangular system (times beta), read-out coefficients
+  float* state;            // [B, H, dim, vdim]
+  long long state_bs;
+  void* o;                 // [B * L, H * vdim]
+  long long ldo;
+  int B, L, H, KH, dim, vdim, groups, fresh;
+};
+
+// One warp per (group, kv head, sequence): 8 x 8 products of the keys with keys and queries, then per value head the inverse.
+template <typename T>
+__global__ void __launch_bounds__(128) delta_pairs_kernel(const ScanArgs p) {
+  pdl_prologue();
+  __shared__ float s_kk[4][DC][DC + 1], s_kq[4][DC][DC + 1];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, rep = p.H / p.KH;
+  const long long w = blockIdx.x * 4ll + warp;
+  if (w >= (long long)p.B * p.groups * p.KH) return;  // whole warp; only __syncwarp below
+  const int kh = int(w % p.KH), grp = int((w / p.KH) % p.groups), b = int(w / p.KH / p.groups);
+  const int t0 = grp * DC, n = min(DC, p.L - t0);
+  const long long row0 = (long long)b * p.L + t0;
+  const T* base = static_cast<const T*>(p.mixed) + row0 * p.ldm;
+  const T* q = base + (long long)kh * p.dim;
+  const T* k = base + (long long)(p.KH + kh) * p.dim;
+  float kk[DC][DC], kq[DC][DC];
+#pragma unroll
+  for (int i = 0; i < DC; ++i)
+#pragma unroll
+    for (int j = 0; j < DC; ++j) kk[i][j] = kq[i][j] = 0.f;
+  for (int d = lane; d < p.dim; d += 32) {
+    float kv[DC], qv[DC];
+#pragma unroll
+    for (int i = 0; i < DC; ++i) {
+      kv[i] = i < n ? Typed<T>::load(k + i * p.ldm + d) : 0.f;
+      qv[i] = i < n ? Typed<T>::load(q + i * p.ldm + d) : 0.f;
+    }
+#pragma unroll
+    for (int i = 0; i < DC; ++i)
+#pragma unroll
+      for (int j = 0; j <= i; ++j) {
+        kk[i][j] += kv[i] * kv[j];
+        kq[i][j] += qv[i] * kv[j];
+      }
+  }
+  const float* rl = p.rlen + row0 * 2 * p.KH;
+#pragma unroll
+  for (int i = 0; i < DC; ++i)
+#pragma unroll
+    for (int j = 0; j <= i; ++j) {
+      const float a = warp_sum(kk[i][j]), c = warp_sum(kq[i][j]);
+      if (lane == 0) {
+        const float rkj = j < n ? rl[(long long)j * 2 * p.KH + p.KH + kh] : 0.f;
+        const float rki = i < n ? rl[(long long)i * 2 * p.KH + p.KH + kh] : 0.f, rqi = i < n ? rl[(long long)i * 2 * p.KH + kh] : 0.f;
+        s_kk[warp][i][j] = a * rki * rkj;
+        s_kq[warp][i][j] = c * rqi * rkj;
+      }
+    }
+  __syncwarp();
+  // lane = (value head of the group r, column c of the 8 x 8 inverse)
+  for (int x = lane; x < rep * DC; x += 32) {
+    const int h = kh * rep + x / DC, c = x % DC;
+    float g[DC], beta[DC];
+#pragma unroll
+    for (int i = 0; i < DC; ++i) {
+      g[i] = i < n ? p.gb[(row0 + i) * 2 * p.H + h] : 1.f;
+      beta[i] = i < n ? p.gb[(row0 + i) * 2 * p.H + p.H + h] : 0.f;
+    }
+    // column c of (1 + M)^-1, M_ij = beta_i D_ij kk_ij: forward substitution; the result is multiplied by beta_c (the right-hand
+    // side of the system is beta_c (v_c - G_c S^T k_c))
+    float y[DC];
+    float* co = p.coef + ((((long long)b * p.groups + grp) * p.H + h) * DC) * 2 * DC;
+#pragma unroll
+    for (int i = 0; i < DC; ++i) {
+      float acc = i == c ? 1.f : 0.f, dec = 1.f;
+#pragma unroll
+      for (int j = i - 1; j >= 0; --j) {
+        dec *= g[j + 1];
+        acc -= beta[i] * dec * s_kk[warp][i][j] * y[j];
+      }
+      y[i] = acc;
+      co[i * 2 * DC + c] = acc * beta[c];
+    }
+    // read-out coefficients of write c: D_ic (k_c . q_i) for i >= c
+    float dec = 1.f;
+#pragma unroll
+    for (int i = 0; i < DC; ++i) {
+      if (i > c) dec *= g[i];
+      co[i * 2 * DC + DC + c] = i >= c ? dec * s_kq[warp][i][c] : 0.f;
+    }
+  }
+}
+
+__device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
+  float2 r;
+  asm("{\n\t.reg .b64 x, y, z, w;\n\tmov.b64 x, {%2, %3};\n\tmov.b64 y, {%4, %5};\n\tmov.b64 z, {%6, %7};\n\t"
+      "fma.rn.f32x2 w, x, y, z;\n\tmov.b64 {%0, %1}, w;\n\t}"
+      : "=f"(r.x), "=f"(r.y)
+      : "f"(a.x), "f"(a.y), "f"(b.x), "f"(b.y), "f"(c.x), "f"(c.y));
+  return r;
+}
+
+// Eight per-lane values of which the sum over the eight lanes of a group is wanted: lane l ends up with the sum of value l.
+__device__ __forceinline__ float transpose_sum8(float (&v)[DC], int l) {
+#pragma unroll
+  for (int s = 4; s > 0; s >>= 1) {
+    const bool up = (l & s) != 0;
+#pragma unroll
+    for (int i = 0; i < s; ++i) {
+      const float send = up ? v[i] : v[i + s], have = up ? v[i + s] : v[i];
+      v[i] = have + __shfl_xor_sync(0xffffffffu, send, s);
+    }
+  }
+  return v[0];
+}
+
+// EPL: state rows per lane (dim <= 8 * EPL), CPL: value columns per lane group.  CTA = 4 warps of 4 lane groups -> 16 * CPL columns
+// of one head.
+template <typename T, int EPL, int CPL>
+__global__ void __launch_bounds__(128) delta_scan_kernel(const ScanArgs p) {
+  pdl_prologue();
+  constexpr int DK = 8 * EPL;
+  __shared__ __align__(16) float s_k[2][DC][DK];
+  __shared__ __align__(16) float s_q[2][DC][DK];
+  __shared__ float s_c[2][DC][2 * DC + 1];
+  __shared__ float s_g[2][2][DC];           // G_i = g_1 .. g_i and D_Ci = g_{i+1} .. g_C
+  const int tid = threadIdx.x, lane = tid & 31, l8 = lane & 7;
+  const int h = blockIdx.y, b = blockIdx.z, kh = h / (p.H / p.KH);
+  const int col0 = (blockIdx.x * 16 + (tid >> 3)) * CPL;
+  float2 S[CPL][EPL / 2];
+  float* st = p.state + (long long)b * p.state_bs + (long long)h * p.dim * p.vdim;
+#pragma unroll
+  for (int c = 0; c < CPL; ++c)
+#pragma unroll
+    for (int e = 0; e < EPL / 2; ++e) {
+      const int d = ((e >> 1) * 8 + l8) * 4 + (e & 1) * 2;
+      const bool ok = !p.fresh && col0 + c < p.vdim;
+      S[c][e].x = (ok && d < p.dim) ? st[(long long)d * p.vdim + col0 + c] : 0.f;
+      S[c][e].y = (ok && d + 1 < p.dim) ? st[(long long)(d + 1) * p.vdim + col0 + c] : 0.f;
+    }
+  const T* base = static_cast<const T*>(p.mixed) + (long long)b * p.L * p.ldm;
+  auto stage = [&](int grp, int buf) {
+    const int t0 = grp * DC, n = min(DC, p.L - t0);
+    const long long row0 = (long long)b * p.L + t0;
+    for (int i = tid; i < DC * DK; i += 128) {
+      const int t = i / DK, d = i % DK;
+      float kv = 0.f, qv = 0.f;
+      if (t < n && d < p.dim) {
+        const T* r = base + (t0 + t) * p.ldm + d;
+        kv = Typed<T>::load(r + (long long)(p.KH + kh) * p.dim) * p.rlen[(row0 + t) * 2 * p.KH + p.KH + kh];
+        qv = Typed<T>::load(r + (long long)kh * p.dim) * p.rlen[(row0 + t) * 2 * p.KH + kh];
+      }
+      s_k[buf][t][d] = kv;
+      s_q[buf][t][d] = qv;
+    }
+    const float* co = p.coef + (((long long)b * p.groups + grp) * p.H + h) * DC * 2 * DC;
+    for (int i = tid; i < DC * 2 * DC; i += 128) s_c[buf][i / (2 * DC)][i % (2 * DC)] = co[i];
+    if (tid < DC) {
+      float G = 1.f, D = 1.f;
+      for (int i = 0; i < DC; ++i) {
+        const float g = i < n ? p.gb[(row0 + i) * 2 * p.H + h] : 1.f;
+        if (i <= tid) G *= g;
+        else D *= g;
+      }
+      s_g[buf][0][tid] = G;
+      s_g[buf][1][tid] = D;
+    }
+  };
+  stage(0, 0);
+  __syncthreads();
+  for (int grp = 0; grp < p.groups; ++grp) {
+    const int buf = grp & 1, t0 = grp * DC, n = min(DC, p.L - t0);
+    // value of this lane's token (lane l8 <-> token l8), requested before the products
+    float v[CPL];
+#pragma unroll
+    for (int c = 0; c < CPL; ++c)
+      v[c] = (l8 < n && col0 + c < p.vdim)
+                 ? Typed<T>::load(base + (t0 + l8) * p.ldm + 2 * p.KH * p.dim + (long long)h * p.vdim + col0 + c) : 0.f;
+    if (grp + 1 < p.groups) stage(grp + 1, buf ^ 1);
+    float sk[CPL][DC], sq[CPL][DC];
+#pragma unroll
+    for (int i = 0; i < DC; ++i) {
+      float2 ak[CPL], aq[CPL];
+#pragma unroll
+      for (int c = 0; c < CPL; ++c) ak[c] = aq[c] = make_float2(0.f, 0.f);
+#pragma unroll
+      for (int e = 0; e < EPL / 4; ++e) {
+        const float4 k4 = *reinterpret_cast<const float4*>(&s_k[buf][i][(e * 8 + l8) * 4]);
+        const float4 q4 = *reinterpret_cast<const float4*>(&s_q[buf][i][(e * 8 + l8) * 4]);
+#pragma unroll
+        for (int c = 0; c < CPL; ++c) {
+          ak[c] = fma2(S[c][2 * e], make_float2(k4.x, k4.y), ak[c]);
+          ak[c] = fma2(S[c][2 * e + 1], make_float2(k4.z, k4.w), ak[c]);
+          aq[c] = fma2(S[c][2 * e], make_float2(q4.x, q4.y), aq[c]);
+          aq[c] = fma2(S[c][2 * e + 1], make_float2(q4.z, q4.w), aq[c]);
+        }
+      }
+#pragma unroll
+      for (int c = 0; c < CPL; ++c) {
+        sk[c][i] = ak[c].x + ak[c].y;
+        sq[c][i] = aq[c].x + aq[c].y;
+      }
+    }
+    const float G = s_g[buf][0][l8], GC = s_g[buf][0][DC - 1];
+    float w[CPL][DC];  // D_Cj u_j of every token, in every lane
+#pragma unroll
+    for (int c = 0; c < CPL; ++c) {
+      const float a = transpose_sum8(sk[c], l8), r = transpose_sum8(sq[c], l8);
+      const float rhs = v[c] - G * a;
+      float u = 0.f, o = G * r;
+#pragma unroll
+      for (int j = 0; j < DC; ++j) u += s_c[buf][l8][j] * __shfl_sync(0xffffffffu, rhs, j, 8);
+#pragma unroll
+      for (int j = 0; j < DC; ++j) {
+        const float uj = __shfl_sync(0xffffffffu, u, j, 8);
+        o += s_c[buf][l8][DC + j] * uj;
+        w[c][j] = uj * s_g[buf][1][j];
+      }
+      if (l8 < n && col0 + c < p.vdim)
+        Typed<T>::store(static_cast<T*>(p.o) + ((long long)b * p.L + t0 + l8) * p.ldo + (long long)h * p.vdim + col0 + c, o);
+    }
+#pragma unroll
+    for (int c = 0; c < CPL; ++c)
+#pragma unroll
+      for (int e = 0; e < EPL / 2; ++e) S[c][e] = make_float2(S[c][e].x * GC, S[c][e].y * GC);
+#pragma unroll
+    for (int j = 0; j < DC; ++j)
+#pragma unroll
+      for (int e = 0; e < EPL / 4; ++e) {
+        const float4 k4 = *reinterpret_cast<const float4*>(&s_k[buf][j][(e * 8 + l8) * 4]);
+#pragma unroll
+        for (int c = 0; c < CPL; ++c) {
+          const float2 uu = make_float2(w[c][j], w[c][j]);
+          S[c][2 * e] = fma2(make_float2(k4.x, k4.y), uu, S[c][2 * e]);
+          S[c][2 * e + 1] = fma2(make_float2(k4.z, k4.w), uu, S[c][2 * e + 1]);
+        }
+      }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int c = 0; c < CPL; ++c) {
+    if (col0 + c >= p.vdim) continue;
+#pragma unroll
+    for (int e = 0; e < EPL / 2; ++e) {
+      const int d = ((e >> 1) * 8 + l8) * 4 + (e & 1) * 2;
+      if (d < p.dim) st[(long long)d * p.vdim + col0 + c] = S[c][e].x;
+      if (d + 1 < p.dim) st[(long long)(d + 1) * p.vdim + col0 + c] = S[c][e].y;
+    }
+  }
+}
+
+struct DeltaOutArgs {
+  const void* o;           // [rows, ldo] read-out of the recurrence
+  long long ldo;
+  const void* gate;        // [rows, ldg] + h * vdim
+  long long ldg;
+  const float* w;          // [vdim]
+  float eps;
+  void* out;               // [rows, ldout]; columns H * vdim .. ldout are zeroed
+  long long ldout;
+  long long rows;
+  int H, vdim;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(256) delta_output_kernel(const DeltaOutArgs p) {
+  pdl_prologue();
+  const long long w = blockIdx.x * 8ll + (threadIdx.x >> 5);
+  const int lane = threadIdx.x & 31;
+  if (w >= p.rows * p.H) return;
+  const long long row = w / p.H;
+  const int h = int(w % p.H);
+  const T* o = static_cast<const T*>(p.o) + row * p.ldo + (long long)h * p.vdim;
+  const T* g = static_cast<const T*>(p.gate) + row * p.ldg + (long long)h * p.vdim;
+  T* out = static_cast<T*>(p.out) + row * p.ldout;
+  float ss = 0.f;
+  for (int c = lane; c < p.vdim; c += 32) {
+    const float v = Typed<T>::load(o + c);
+    ss += v * v;
+  }
+  const float r = 1.f / sqrtf(warp_sum(ss) / float(p.vdim) + p.eps);
+  for (int c = lane; c < p.vdim; c += 32) {
+    const float z = Typed<T>::load(g + c);
+    Typed<T>::store(out + (long long)h * p.vdim + c, Typed<T>::load(o + c) * r * p.w[c] * z * Typed<T>::sigmoid_(z));
+  }
+  if (h == 0)
+    for (int c = p.H * p.vdim + lane; c < p.ldout; c += 32) Typed<T>::store(out + c, 0.f);
+}
+
+// ------------------------------------------------------------------------------------------------ decoding
+struct StepArgs {
+  const void* mixed;       // [B, ldm]
+  long long ldm;
+  const float* rlen;
+  const float* gb;
+  float* state;
+  long long state_bs;
+  const int* lengths;
+  const int* active;
+  const void* gate;        // [B, ldg] + h * vdim
+  long long ldg;
+  const float* w;          // [vdim]
+  float eps;
+  void* out;               // [B, ldout]
+  long long ldout;
+  int B, H, KH, dim, vdim;
+};
+
+constexpr int ST_THREADS = 512;
+// One CTA per (head, sequence).  Threads are (row group, column): CW columns, 512 / CW row groups, RPT rows per thread in registers.
+template <typename T, int RPT>
+__global__ void __launch_bounds__(ST_THREADS) delta_step_kernel(const StepArgs p, int CW) {
+  pdl_prologue();
+  extern __shared__ float sm[];
+  const int RG = ST_THREADS / CW, tid = threadIdx.x, c = tid % CW, rg = tid / CW, h = blockIdx.x, b = blockIdx.y;
+  float* s_k = sm;                 // [dim]
+  float* s_q = s_k + p.dim;        // [dim]
+  float* s_o = s_q + p.dim;        // [vdim]
+  float* s_r = s_o + p.vdim;       // [RG][CW]
+  float* s_red = s_r + ST_THREADS; // [40]
+  const int kh = h / (p.H / p.KH);
+  const bool fresh = p.lengths[b] == 0, keep = !(p.active && !p.active[b]);
+  const T* mixed = static_cast<const T*>(p.mixed) + (long long)b * p.ldm;
+  const float rq = p.rlen[(long long)b * 2 * p.KH + kh], rk = p.rlen[(long long)b * 2 * p.KH + p.KH + kh];
+  for (int d = tid; d < p.dim; d += ST_THREADS) {
+    s_k[d] = Typed<T>::load(mixed + (long long)(p.KH + kh) * p.dim + d) * rk;
+    s_q[d] = Typed<T>::load(mixed + (long long)kh * p.dim + d) * rq;
+  }
+  const float g = p.gb[(long long)b * 2 * p.H + h], beta = p.gb[(long long)b * 2 * p.H + p.H + h];
+  float* st = p.state + (long long)b * p.state_bs + (long long)h * p.dim * p.vdim;
+  __syncthreads();
+  float ss = 0.f;
+  for (int v0 = 0; v0 < p.vdim; v0 += CW) {
+    const int v = v0 + c;
+    const bool ok = v < p.vdim;
+    float S[RPT], a = 0.f;
+#pragma unroll
+    for (int i = 0; i < RPT; ++i) {
+      const int d = rg + i * RG;
+      S[i] = (ok && d < p.dim && !fresh) ? st[(long long)d * p.vdim + v] * g : 0.f;
+    }
+#pragma unroll
+    for (int i = 0; i < RPT; ++i) {
+      const int d = rg + i * RG;
+      if (d < p.dim) a += S[i] * s_k[d];
+    }
+    s_r[tid] = a;
+    __syncthreads();
+    float sk = 0.f;
+    for (int r = 0; r < RG; ++r) sk += s_r[r * CW + c];
+    __syncthreads();
+    const float u = ok ? beta * (Typed<T>::load(mixed + 2ll * p.KH * p.dim + (long long)h * p.vdim + v) - sk) : 0.f;
+    float o = 0.f;
+#pragma unroll
+    for (int i = 0; i < RPT; ++i) {
+      const int d = rg + i * RG;
+      if (d < p.dim) {
+        S[i] += s_k[d] * u;
+        o += S[i] * s_q[d];
+        if (ok && keep) st[(long long)d * p.vdim + v] = S[i];
+      }
+    }
+    s_r[tid] = o;
+    __syncthreads();
+    if (rg == 0 && ok) {
+      float t = 0.f;
+      for (int r = 0; r < RG; ++r) t += s_r[r * CW + c];
+      s_o[v] = t;
+      ss += t * t;
+    }
+    __syncthreads();
+  }
+  ss = block_sum(ss, s_red);
+  const float r = 1.f / sqrtf(ss / float(p.vdim) + p.eps);
+  T* out = static_cast<T*>(p.out) + (long long)b * p.ldout;
+  const T* gt = static_cast<const T*>(p.gate) + (long long)b * p.ldg + (long long)h * p.vdim;
+  for (int v = tid; v < p.vdim; v += ST_THREADS) {
+    const float z = Typed<T>::load(gt + v);
+    Typed<T>::store(out + (long long)h * p.vdim + v, s_o[v] * r * p.w[v] * z * Typed<T>::sigmoid_(z));
+  }
+  if (h == 0)
+    for (int v = p.H * p.vdim + tid; v < p.ldout; v += ST_THREADS) Typed<T>::store(out + v, 0.f);
+}
+
+template <typename T>
+static int launch_scan(const ScanArgs& p, cudaStream_t s) {
+  const long long pw = (long long)p.B * p.groups * p.KH;
+  launch_pdl(delta_pairs_kernel<T>, dim3(unsigned((pw + 3) / 4)), dim3(128), 0, s, p);
+  auto grid = [&](int cpl) { return dim3((p.vdim + 16 * cpl - 1) / (16 * cpl), p.H, p.B); };
+  if (p.dim <= 32) launch_pdl(delta_scan_kernel<T, 4, 2>, grid(2), dim3(128), 0, s, p);
+  else if (p.dim <= 64) launch_pdl(delta_scan_kernel<T, 8, 2>, grid(2), dim3(128), 0, s, p);
+  else if (p.dim <= 128) launch_pdl(delta_scan_kernel<T, 16, 2>, grid(2), dim3(128), 0, s, p);
+  else if (p.dim <= 256) launch_pdl(delta_scan_kernel<T, 32, 1>, grid(1), dim3(128), 0, s, p);
+  else return 1006;
+  return int(cudaGetLastError());
+}
+
+template <typename T>
+static int launch_step(const StepArgs& p, cudaStream_t s) {
+  int CW = 32;
+  while (CW < p.vdim && CW < 128) CW *= 2;
+  const int rg = ST_THREADS / CW, rows = (p.dim + rg - 1) / rg;
+  const size_t smem = size_t(2 * p.dim + p.vdim + ST_THREADS + 40) * sizeof(float);
+  if (smem > 48 * 1024) return 1010;
+  const dim3 grid(p.H, p.B);
+  if (rows <= 8) launch_pdl(delta_step_kernel<T, 8>, grid, dim3(ST_THREADS), smem, s, p, CW);
+  else if (rows <= 16) launch_pdl(delta_step_kernel<T, 16>, grid, dim3(ST_THREADS), smem, s, p, CW);
+  else if (rows <= 32) launch_pdl(delta_step_kernel<T, 32>, grid, dim3(ST_THREADS), smem, s, p, CW);
+  else if (rows <= 64) launch_pdl(delta_step_kernel<T, 64>, grid, dim3(ST_THREADS), smem, s, p, CW);
+  else return 1006;
+  return int(cudaGetLastError());
+}
+
+}  // namespace ats
+
+using namespace ats;
+
+// Every entry point takes its argument struct by address (the ctypes mirror is in ops/delta.py); `fp32` selects the element type.
+ATS_API int ats_delta_prep(const DeltaArgs* p, int fp32, void* stream) {
+  if (p->taps < 1 || (p->lengths && p->L != 1) || p->KH < 1 || p->H % p->KH) return 1006;
+  const long long warps = (long long)p->B * p->L * (2 * p->KH + p->H + 1);
+  if (warps <= 0) return 0;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  const dim3 grid(unsigned((warps + 7) / 8));
+  if (fp32) launch_pdl(delta_prep_kernel<float>, grid, dim3(256), 0, s, *p);
+  else launch_pdl(delta_prep_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, *p);
+  if (!p->lengths && p->taps > 1) {
+    const dim3 tg((p->C + 255) / 256, p->B);
+    if (fp32) launch_pdl(delta_tail_kernel<float>, tg, dim3(256), 0, s, *p);
+    else launch_pdl(delta_tail_kernel<__nv_bfloat16>, tg, dim3(256), 0, s, *p);
+  }
+  return int(cudaGetLastError());
+}
+
+ATS_API int ats_delta_scan(const ScanArgs* p, int fp32, void* stream) {
+  if (p->B <= 0 || p->L <= 0) return 0;
+  if (p->groups != (p->L + DC - 1) / DC) return 1006;
+  return fp32 ? launch_scan<float>(*p, static_cast<cudaStream_t>(stream)) : launch_scan<__nv_bfloat16>(*p, static_cast<cudaStream_t>(stream));
+}
+
+ATS_API int ats_delta_output(const DeltaOutArgs* p, int fp32, void* stream) {
+  const long long warps = p->rows * p->H;
+  if (warps <= 0) return 0;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  const dim3 grid(unsigned((warps + 7) / 8));
+  if (fp32) launch_pdl(delta_output_kernel<float>, grid, dim3(256), 0, s, *p);
+  else launch_pdl(delta_output_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, *p);
+  return int(cudaGetLastError());
+}
+
+ATS_API int ats_delta_step(const StepArgs* p, int fp32, void* stream) {
+  if (p->B <= 0) return 0;
+  return fp32 ? launch_step<float>(*p, static_cast<cudaStream_t>(stream)) : launch_step<__nv_bfloat16>(*p, static_cast<cudaStream_t>(stream));
+}
