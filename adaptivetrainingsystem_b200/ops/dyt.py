@@ -11,6 +11,7 @@ The residual ``x`` is fp32 whatever the element type of the products.  CPU tenso
 from __future__ import annotations
 
 import ctypes
+import os
 from dataclasses import dataclass
 from typing import Optional, Tuple
 
@@ -29,6 +30,7 @@ def _fns():
     if not _sig:
         for name, args in (("ats_fold_dyt", [_vp, _ci, _cll, _vp, _vp, _vp, _vp, _cf, _vp, _vp, _cf, _vp, _ci, _cll, _ci, _vp]),
                            ("ats_fold_gelu", [_vp, _ci, _cll, _vp, _vp, _ci, _cll, _ci, _vp]),
+                           ("ats_gemm_bf16_block", [_vp, _cll, _vp, _cll, _vp, _ci, _ci, _ci, _ci, _vp, _vp, _ci, _vp, _vp, _cf, _vp, _vp, _cf, _vp, _ci, _vp]),
                            ("ats_embed_dyt", [_vp, _vp, _ci, _ci, _vp, _vp, _vp, _vp, _cf, _vp, _cll, _ci, _vp])):
             f = getattr(lib, name)
             f.restype, f.argtypes = _ci, args
@@ -84,6 +86,24 @@ def _product_f32(a: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
     return part
 
 
+# bf16 products whose reduction is not split over the SMs do the element-wise step in their epilogue; ATS_BLOCK_EPILOGUE=0 runs it as a
+# launch of its own instead (for comparison)
+FUSED_EPILOGUE = os.environ.get("ATS_BLOCK_EPILOGUE", "1") == "1"
+
+
+def _fused(a: torch.Tensor, w: torch.Tensor) -> bool:
+    return FUSED_EPILOGUE and a.dtype == torch.bfloat16 and (not G.SPLIT_K_SKINNY or G._skinny_splits(a.shape[0], w.shape[0], a.shape[1]) == 1)
+
+
+def _block_gemm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: Optional[torch.Tensor], x: Optional[torch.Tensor], c: Optional[DytChain]) -> None:
+    a = G._check2d(a)
+    (T, K), N = a.shape, w.shape[0]
+    w1, b1, a1, w2, b2, a2 = (c.w1, c.b1, c.a1, c.w2, c.b2, c.a2) if c is not None else (None, None, 0.0, None, None, 0.0)
+    _lib.check(_fns().ats_gemm_bf16_block(_lib.ptr(a), a.stride(0), _lib.ptr(w), w.stride(0), _lib.ptr(out), out.stride(0), T, N, K, _lib.ptr(bias), _lib.ptr(x),
+                                          0 if x is None else x.stride(0), _lib.ptr(w1), _lib.ptr(b1), a1, _lib.ptr(w2), _lib.ptr(b2), a2,
+                                          _lib.ptr(_lib.status_tensor(a.device)), 0, _lib.stream_ptr(a.device)), "ats_gemm_bf16_block")
+
+
 def linear_residual(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], x: torch.Tensor, c: DytChain) -> torch.Tensor:
     """The residual step after ``y = a @ w^T``: updates ``x`` [T, N] (fp32) in place, returns ``h`` [T, N] in a's dtype."""
     T, N = x.shape
@@ -93,8 +113,11 @@ def linear_residual(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tenso
             y = y + bias
         x += torch.tanh(c.a1 * y) * c.w1 + c.b1
         return (torch.tanh(c.a2 * x) * c.w2 + c.b2).to(a.dtype)
-    part = _product_f32(a, w)
     h = torch.empty(T, N, dtype=a.dtype, device=a.device)
+    if _fused(a, w):
+        _block_gemm(a, w, h, bias, x, c)
+        return h
+    part = _product_f32(a, w)
     _lib.check(_fns().ats_fold_dyt(_lib.ptr(part), part.shape[0], T * N, _lib.ptr(bias), _lib.ptr(x), _lib.ptr(c.w1), _lib.ptr(c.b1), c.a1, _lib.ptr(c.w2),
                                    _lib.ptr(c.b2), c.a2, _lib.ptr(h), int(h.dtype == torch.float32), T, N, _lib.stream_ptr(a.device)), "ats_fold_dyt")
     return h
@@ -105,8 +128,11 @@ def linear_gelu(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor]) 
     T, N = a.shape[0], w.shape[0]
     if not a.is_cuda:
         return gelu_tanh(torch.nn.functional.linear(a.float(), w.float(), bias)).to(a.dtype)
-    part = _product_f32(a, w)
     out = torch.empty(T, N, dtype=a.dtype, device=a.device)
+    if _fused(a, w):
+        _block_gemm(a, w, out, bias, None, None)
+        return out
+    part = _product_f32(a, w)
     _lib.check(_fns().ats_fold_gelu(_lib.ptr(part), part.shape[0], T * N, _lib.ptr(bias), _lib.ptr(out), int(out.dtype == torch.float32), T, N,
                                     _lib.stream_ptr(a.device)), "ats_fold_gelu")
     return out

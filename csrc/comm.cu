@@ -30,11 +30,6 @@ __device__ __forceinline__ void st_release_sys(int* p, int v) {
   asm volatile("st.release.sys.global.s32 [%0], %1;" ::"l"(p), "r"(v) : "memory");
 }
 
-// Wait budget of every peer wait in this library (nanoseconds of %globaltimer).  A host-side value handed to the kernels as
-// an argument, so a test can make a wait give up after a few milliseconds and production runs can allow slow peers more
-// than the one-second default.
-static unsigned long long g_wait_budget_ns = ATS_WAIT_BUDGET_NS;
-
 // flags.p[r] = base of rank r's flag array (int[world]).  The epoch lives in device memory (`epoch_counter`, private to
 // this rank): thread 0 advances it, so a launch that is replayed from a CUDA graph still waits for a NEW arrival of
 // every peer instead of re-using the epoch that was frozen into the captured arguments.  All ranks issue their barriers
@@ -307,6 +302,8 @@ static PeerPtrs to_peers(void* const* host_ptrs, int world) {
 
 using namespace ats;
 
+ATS_API unsigned long long ats_get_wait_budget_ns();  // gemm_tcgen05.cu
+
 // ---- symmetric memory ----------------------------------------------------------------------------------
 ATS_API int ats_ipc_alloc(unsigned long long bytes, void** ptr, unsigned char* handle64) {
   cudaError_t e = cudaMalloc(ptr, bytes);
@@ -337,13 +334,9 @@ ATS_API int ats_peer_barrier(void* const* flags, void* const* payload_dst, const
   PeerPtrs none = {};
   cudaError_t ce = launch_pdl(peer_barrier_kernel, dim3(1), dim3(32), 0, static_cast<cudaStream_t>(stream), to_peers(flags, world),
                               payload_dst ? to_peers(payload_dst, world) : none, payload_src, rank, world, epoch_counter,
-                              (unsigned long long)g_wait_budget_ns, status, wait_ns);
+                              ats_get_wait_budget_ns(), status, wait_ns);
   return int(ce != cudaSuccess ? ce : cudaGetLastError());
 }
-
-// Budget of every peer wait launched after this call (0 restores the default of one second).
-ATS_API void ats_set_wait_budget_ns(unsigned long long ns) { g_wait_budget_ns = ns ? ns : ATS_WAIT_BUDGET_NS; }
-ATS_API unsigned long long ats_get_wait_budget_ns() { return g_wait_budget_ns; }
 
 // Reduce this rank's shard [offset, offset + n) of the gradient buckets of all ranks into out32 and its squared sum
 // into sumsq[0] (added when accumulate).  partial: >= 1184 floats of scratch.

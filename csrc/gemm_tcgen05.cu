@@ -36,7 +36,7 @@ constexpr int GEMM_THREADS = 256;  // TMA, MMA, 4 epilogue warps, 2 copy warps (
 constexpr int MAX_GROUPS = 256;
 constexpr int GEMM_SMEM_BYTES = STAGES * STAGE_BYTES + 1024 /*align*/ + 256 /*barriers*/ + (MAX_GROUPS + 1) * 4;
 
-enum Epilogue : int { kStore = 0, kAddC = 1, kF32 = 2, kSwiGLU = 3, kSwiGLUBwd = 4 };
+enum Epilogue : int { kStore = 0, kAddC = 1, kF32 = 2, kSwiGLU = 3, kSwiGLUBwd = 4, kGelu = 5, kDyt = 6 };
 
 struct GemmArgs {
   int M, N, K;
@@ -60,6 +60,13 @@ struct GemmArgs {
   int k_segs;            // ragged == 2: the reduction of group g runs over k_segs blocks of rows, seg_stride apart,
   int seg_stride;        //              block s holding counts[g * k_segs + s] rows
   void* const* d_table;  // optional per-group output base pointers (e.g. buffers on peer GPUs)
+  // kGelu: D = gelu_tanh(acc + bias).  kDyt: the residual step of a block with Dynamic-Tanh norms, x <- x + tanh(a1 (acc + bias)) w1 + b1,
+  // D = tanh(a2 x) w2 + b2, with x fp32 [M, ldx] (csrc/dyt.cu is the stand-alone form).  All vectors fp32 [N]; bias may be null.
+  const float* bias;
+  float* x;
+  int ldx;
+  const float* w1; const float* b1; const float* w2; const float* b2;
+  float a1, a2;
   // kF32 with scatter_rows > 0: reduce-scatter inside the epilogue.  Row r of the product belongs to rank r / scatter_rows, whose fp32
   // buffer d_table[r / scatter_rows] receives the row at (r % scatter_rows) * ldd with vector atomic adds (`red.add.v4.f32`, which
   // travel over NVLink for rows owned by peers): every rank of a data-parallel group adds its partial weight gradient straight
@@ -302,6 +309,67 @@ __device__ __forceinline__ void epilogue_tile(const GemmArgs& p, const TileCoord
               }
             }
           }
+        }
+      }
+    }
+  } else if (p.epilogue == kGelu || p.epilogue == kDyt) {
+    const bool dyt = p.epilogue == kDyt;
+    __nv_bfloat16* drow = p.D + (long long)row * p.ldd;
+    float* xrow = dyt ? p.x + (long long)row * p.ldx : nullptr;
+#pragma unroll 1
+    for (int c = 0; c < BN / 32; ++c) {
+      const int colbase = t.n0 + c * 32;
+      if (colbase >= p.N) break;
+      uint4 xq[8];  // 32 residual values, requested before the accumulator is read (N is a multiple of 8, x rows are 32-byte aligned)
+      if (dyt && row_ok) {
+#pragma unroll
+        for (int v = 0; v < 4; ++v)
+          if (colbase + v * 8 < p.N) ld_global_32B(xrow + colbase + v * 8, xq[2 * v], xq[2 * v + 1]);
+      }
+      uint32_t r[32];
+      tmem_ld_32x32(taddr + c * 32, r);
+      tmem_ld_wait();
+      if (!row_ok) continue;
+      auto piece = [&](int v, int col) -> uint4 {  // eight columns
+        float f[8];
+#pragma unroll
+        for (int e = 0; e < 8; ++e) f[e] = have_acc ? __uint_as_float(r[v * 8 + e]) * rs : 0.f;
+        if (p.bias) {
+          const float4 b0 = *reinterpret_cast<const float4*>(p.bias + col), b1 = *reinterpret_cast<const float4*>(p.bias + col + 4);
+          f[0] += b0.x; f[1] += b0.y; f[2] += b0.z; f[3] += b0.w;
+          f[4] += b1.x; f[5] += b1.y; f[6] += b1.z; f[7] += b1.w;
+        }
+        if (dyt) {
+          float* xf = reinterpret_cast<float*>(&xq[2 * v]);
+#pragma unroll
+          for (int q = 0; q < 2; ++q) {
+            const float4 w1 = *reinterpret_cast<const float4*>(p.w1 + col + 4 * q), b1 = *reinterpret_cast<const float4*>(p.b1 + col + 4 * q);
+            const float4 w2 = *reinterpret_cast<const float4*>(p.w2 + col + 4 * q), b2 = *reinterpret_cast<const float4*>(p.b2 + col + 4 * q);
+            xf[4 * q] += tanh_fast(p.a1 * f[4 * q]) * w1.x + b1.x;
+            xf[4 * q + 1] += tanh_fast(p.a1 * f[4 * q + 1]) * w1.y + b1.y;
+            xf[4 * q + 2] += tanh_fast(p.a1 * f[4 * q + 2]) * w1.z + b1.z;
+            xf[4 * q + 3] += tanh_fast(p.a1 * f[4 * q + 3]) * w1.w + b1.w;
+            f[4 * q] = tanh_fast(p.a2 * xf[4 * q]) * w2.x + b2.x;
+            f[4 * q + 1] = tanh_fast(p.a2 * xf[4 * q + 1]) * w2.y + b2.y;
+            f[4 * q + 2] = tanh_fast(p.a2 * xf[4 * q + 2]) * w2.z + b2.z;
+            f[4 * q + 3] = tanh_fast(p.a2 * xf[4 * q + 3]) * w2.w + b2.w;
+          }
+          st_global_32B(xrow + col, xq[2 * v], xq[2 * v + 1]);
+        } else {
+#pragma unroll
+          for (int e = 0; e < 8; ++e) f[e] = 0.5f * f[e] * (1.f + tanh_fast(0.7978845608028654f * (f[e] + 0.044715f * f[e] * f[e] * f[e])));
+        }
+        return make_uint4(pack_bf16x2(f[0], f[1]), pack_bf16x2(f[2], f[3]), pack_bf16x2(f[4], f[5]), pack_bf16x2(f[6], f[7]));
+      };
+#pragma unroll
+      for (int v = 0; v < 4; v += 2) {
+        const int col = colbase + v * 8;
+        if (p.wide && col + 16 <= p.N) {
+          const uint4 lo = piece(v, col), hi = piece(v + 1, col + 8);
+          st_global_32B(drow + col, lo, hi);
+        } else {
+          if (col < p.N) *reinterpret_cast<uint4*>(drow + col) = piece(v, col);
+          if (col + 8 < p.N) *reinterpret_cast<uint4*>(drow + col + 8) = piece(v + 1, col + 8);
         }
       }
     }
@@ -1017,7 +1085,14 @@ static int num_sms() {
 
 using namespace ats;
 
-ATS_API unsigned long long ats_get_wait_budget_ns();  // comm.cu
+// Wait budget of every peer wait in this library (nanoseconds of %globaltimer).  A host-side value handed to the kernels as
+// an argument, so a test can make a wait give up after a few milliseconds and production runs can allow slow peers more
+// than the one-second default.  (Here, in the file that every library has, because the gathering products need it.)
+static unsigned long long g_wait_budget_ns = ATS_WAIT_BUDGET_NS;
+// Budget of every peer wait launched after this call (0 restores the default of one second).
+ATS_API void ats_set_wait_budget_ns(unsigned long long ns) { g_wait_budget_ns = ns ? ns : ATS_WAIT_BUDGET_NS; }
+ATS_API unsigned long long ats_get_wait_budget_ns() { return g_wait_budget_ns; }
+
 static int launch_gemm(const CUtensorMap& ma, const CUtensorMap& mb, const GemmArgs& p, int epilogue, int groups, int M, int N,
                        int max_ctas, void* stream, const CUtensorMap* mb_own = nullptr);
 static long long* g_gemm_prof = nullptr;
@@ -1087,6 +1162,7 @@ ATS_API int ats_gemm_bf16(const void* A, long long a_rows, long long a_cols, lon
   p.n_copy = 0; p.n_rot = 0; p.own_row0 = 0; p.own_rows = 0; p.prof = g_gemm_prof;
   p.n_edge = 0; p.edge_chunk[0] = p.edge_chunk[1] = -1;
   p.out2 = nullptr; p.ldout2 = 0; p.out2_gs = 0;
+  if (epilogue == kGelu || epilogue == kDyt) return 1004;  // ats_gemm_bf16_block
   if (epilogue == kSwiGLUBwd) {
     // second output (h) travels in the C slot of this entry point: C / ldc / c_gs
     if (!aux || (up_offset & 7) || (ldaux & 7)) return 1004;
@@ -1094,6 +1170,34 @@ ATS_API int ats_gemm_bf16(const void* A, long long a_rows, long long a_cols, lon
     p.C = nullptr;
   }
   return launch_gemm(ma, mb, p, epilogue, groups, M, N, max_ctas, stream);
+}
+
+// D [M, N] = epilogue(A [M, K] B [N, K]^T), both operands K-major, with the element-wise block steps kGelu (x == nullptr) and kDyt.
+ATS_API int ats_gemm_bf16_block(const void* A, long long lda, const void* B, long long ldb, void* D, int ldd, int M, int N, int K, const void* bias, void* x,
+                                int ldx, const void* w1, const void* b1, float a1, const void* w2, const void* b2, float a2, int* status, int max_ctas,
+                                void* stream) {
+  static thread_local bool ctx_bound = false;
+  if (!ctx_bound) {
+    cudaFree(0);
+    ctx_bound = true;
+  }
+  const bool dyt = x != nullptr;
+  if ((N & 7) || (ldd & 7) || K < 1 || (dyt && ((ldx & 7) || (reinterpret_cast<uintptr_t>(x) & 31) || !w1 || !b1 || !w2 || !b2))) return 1003;
+  CUtensorMap ma, mb;
+  int e;
+  if ((e = make_tmap_2d(&ma, A, M, K, lda, 2, 64, 128))) return e;
+  if ((e = make_tmap_2d(&mb, B, N, K, ldb, 2, 64, 128))) return e;
+  GemmArgs p = {};
+  p.M = M; p.N = N; p.K = K; p.groups = 1; p.b_div = 1; p.k_split = 1; p.k_segs = 1; p.alpha = 1.f;
+  p.b_kblocks = int(K / 64);
+  p.D = static_cast<__nv_bfloat16*>(D); p.ldd = ldd;
+  p.epilogue = dyt ? kDyt : kGelu;
+  p.bias = static_cast<const float*>(bias); p.x = static_cast<float*>(x); p.ldx = ldx;
+  p.w1 = static_cast<const float*>(w1); p.b1 = static_cast<const float*>(b1); p.a1 = a1;
+  p.w2 = static_cast<const float*>(w2); p.b2 = static_cast<const float*>(b2); p.a2 = a2;
+  p.status = status; p.edge_chunk[0] = p.edge_chunk[1] = -1;
+  p.prof = g_gemm_prof;
+  return launch_gemm(ma, mb, p, p.epilogue, 1, M, N, max_ctas, stream);
 }
 
 // Fold of the fp32 partial products that reduction slices leave (k_split > 1, or the dense form with one group per slice):

@@ -951,7 +951,7 @@ ATS_API int ats_serve_plan_dispatch(const void* x, const int* topk_idx, int* slo
 // norm_w / norm_out (both or neither): also write RMSNorm(out) * norm_w, the input of the next block.
 // ready_flags / epoch_counter / experts_per_rank (all or none): the kernel itself waits for the owners of the rows it pulls (see
 // ats_splitk_reduce_signal) instead of relying on a barrier launch before it.
-ATS_API unsigned long long ats_get_wait_budget_ns();  // comm.cu
+ATS_API unsigned long long ats_get_wait_budget_ns();  // gemm_tcgen05.cu
 ATS_API int ats_serve_combine(void* const* src_table, const void* src0, long long src_stride, const int* topk_idx, const int* slot_pos,
                               const float* topk_w, const void* residual, void* out, int tokens, int k, int hidden, const void* norm_w,
                               void* norm_out, float eps, const int* ready_flags, const int* epoch_counter, int experts_per_rank, int* status,
