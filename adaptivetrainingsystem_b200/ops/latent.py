@@ -7,6 +7,7 @@
 from __future__ import annotations
 
 import ctypes
+import os
 from dataclasses import dataclass
 from typing import Optional, Tuple
 
@@ -19,6 +20,10 @@ _vp, _ci, _cll, _cf = ctypes.c_void_p, ctypes.c_int, ctypes.c_longlong, ctypes.c
 
 def pad8(n: int) -> int:
     return (n + 7) // 8 * 8
+
+
+# ATS_WINDOW_TC=0: portions of a prompt use the general window kernel for every shape (for comparison)
+WINDOW_TC = os.environ.get("ATS_WINDOW_TC", "1") == "1"
 
 
 @dataclass(frozen=True)
@@ -182,6 +187,12 @@ def latent_finish(q: torch.Tensor, ctx: torch.Tensor, ring: torch.Tensor, s: Lat
     _call("ats_latent_finish", a, q)
 
 
+def window_tc_ok(q: torch.Tensor, s: LatentShape, L: int) -> bool:
+    """The tensor-core kernel covers these sizes, and the portion is long enough to fill more than a few rows of its query tiles."""
+    return (q.dtype == torch.bfloat16 and WINDOW_TC and L >= 16 and s.dim in (64, 128) and s.rot % 8 == 0 and 8 <= s.rot <= 64 and s.vdim in (64, 128)
+            and s.rank % 8 == 0 and s.scale > 0)
+
+
 def window_attention(q: torch.Tensor, kv: torch.Tensor, ctx: torch.Tensor, gate: Optional[torch.Tensor], s: LatentShape, n_old: int) -> torch.Tensor:
     """q [B * L, q_width] (rotated), kv [B, n_old + L, kv_width], ctx [B, n_old + L, cwp] (its rotated key part is shared by the heads),
     gate [B * L, .] (strided view, heads x vdim) -> sigmoid-gated attention output [B * L, o_pad]."""
@@ -204,6 +215,12 @@ def window_attention(q: torch.Tensor, kv: torch.Tensor, ctx: torch.Tensor, gate:
         return out
     out = torch.empty(B * L, s.o_pad, dtype=q.dtype, device=q.device)
     kr = ctx[..., s.rank:]
+    if window_tc_ok(q, s, L):
+        f = _lib.cuda_lib().ats_window_attn_tc
+        f.restype, f.argtypes = _ci, [_vp, _cll, _vp, _cll, _ci, _vp, _cll, _vp, _cll, _vp, _cll] + [_ci] * 8 + [_cf, _vp, _vp]
+        _lib.check(f(_p(q), q.stride(0), _p(kv), kv.stride(1), s.v_col, _p(kr), ctx.stride(1), _p(gate), 0 if gate is None else gate.stride(0), _p(out), out.stride(0),
+                     B, L, n_old, H, s.dim, s.rot, s.vdim, s.window, s.scale, _p(_lib.status_tensor(q.device)), _lib.stream_ptr(q.device)), "ats_window_attn_tc")
+        return out
     a = _Window(_p(q), q.stride(0), _p(kv), kv.stride(1), s.v_col, _p(kr), ctx.stride(1), _p(gate), 0 if gate is None else gate.stride(0), _p(out), out.stride(0),
                 B, L, n_old, H, s.dim, s.rot, s.vdim, s.window, s.scale)
     _call("ats_window_attn", a, q)

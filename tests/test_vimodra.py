@@ -103,7 +103,8 @@ def _one_layer(layer, **kw):
 
 @pytest.mark.parametrize("device,dtype", PLACES)
 @pytest.mark.parametrize("spec", [dict(), dict(heads=1, dim=32, rot_dim=2, vdim=33, kv_rank=17, q_rank=9, size=1), dict(heads=4, dim=20, rot_dim=12, size=64),
-                                  dict(heads=2, dim=64, rot_dim=64, vdim=64, kv_rank=128, q_rank=64, size=33)])
+                                  dict(heads=2, dim=64, rot_dim=64, vdim=64, kv_rank=128, q_rank=64, size=33),
+                                  dict(heads=3, dim=128, rot_dim=24, vdim=128, kv_rank=56, q_rank=40, size=50)])
 def test_latent_attention_alone(device, dtype, spec):
     cfg, W = _one_layer(O.latent_spec(**spec))
     ids = tokens(70)
@@ -113,6 +114,48 @@ def test_latent_attention_alone(device, dtype, spec):
     close(logits[0], want, dtype)
     close(got[0][0], streams[0], dtype)
     close(run_portions(m, ids, [1] * 30 + [7, 2, 1, 30]), want, dtype)
+
+
+def plain_window_attention(q, kv, kr, gate, s, n_old):
+    """One sequence: q [L, H, dim + rot] rotated, kv / kr of n_old + L rows."""
+    L, H = q.shape[:2]
+    rows = n_old + L
+    out = torch.empty(L, H, s.vdim, dtype=q.dtype)
+    for i in range(L):
+        lo, hi = max(0, n_old + i - s.window + 1), n_old + i + 1
+        for h in range(H):
+            k = torch.cat([kv[lo:hi, h * s.dim:(h + 1) * s.dim], kr[lo:hi]], 1)
+            p = torch.softmax(k @ q[i, h] * s.scale, 0)
+            out[i, h] = p @ kv[lo:hi, s.v_col + h * s.vdim:s.v_col + (h + 1) * s.vdim]
+    assert rows == kv.shape[0]
+    return out.reshape(L, -1) * torch.sigmoid(gate)
+
+
+@gpu
+@pytest.mark.parametrize("dims", [(128, 64, 128), (64, 64, 64), (64, 32, 128), (128, 8, 64)])
+@pytest.mark.parametrize("L,n_old,window", [(300, 0, 1), (300, 0, 97), (513, 100, 101), (256, 255, 256), (128, 0, 1 << 30), (129, 37, 128), (400, 60, 129),
+                                            (17, 500, 501), (640, 0, 384), (257, 0, 127)])
+def test_tensor_core_window_attention(dims, L, n_old, window):
+    """Query tiles of 128 / 256 rows, key blocks of 128: windows at, below and above their sizes, context before the portion, tails;
+    keys at distance window - 1 carry a large score, so that the window's edge shows."""
+    dim, rot, vdim = dims
+    s = latent_ops.LatentShape(2, dim, rot, vdim, 64, 32, window, 0.11, 1e-5)
+    g = torch.Generator().manual_seed(L + window)
+    B = 2
+    q, kv = torch.randn(B, L, s.q_width, generator=g), torch.randn(B, n_old + L, s.kv_width, generator=g)
+    ctx, gate = torch.randn(B, n_old + L, s.cwp, generator=g), torch.randn(B, L, s.o_pad, generator=g)
+    for edge in (window - 1, window):      # just inside and just outside: query i = 1.2 x the key at that distance, for every seventh query
+        for i in range(L):
+            j = n_old + i - edge
+            if i % 7 == (0 if edge == window else 3) and j >= 0:
+                for h in range(2):
+                    q[:, i, h * (dim + rot):h * (dim + rot) + dim] = 1.2 * kv[:, j, h * dim:(h + 1) * dim]
+    q, kv, ctx, gate = (v.to(torch.bfloat16) for v in (q, kv, ctx, gate))
+    assert latent_ops.window_tc_ok(q.cuda(), s, L)
+    out = latent_ops.window_attention(q.cuda().view(B * L, -1), kv.cuda(), ctx.cuda(), gate.cuda().view(B * L, -1), s, n_old).float().cpu().view(B, L, -1)
+    for b in range(B):
+        want = plain_window_attention(q[b].double().view(L, 2, -1), kv[b].double(), ctx[b, :, s.rank:s.cw].double(), gate[b].double(), s, n_old)
+        assert float((out[b] - want).abs().max()) < 3e-2
 
 
 @pytest.mark.parametrize("device,dtype", PLACES)
