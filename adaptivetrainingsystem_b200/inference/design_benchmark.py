@@ -209,7 +209,7 @@ def kernels(size: str, B: int = 8, L: int = 2048, decode_batch: int = 64) -> Lis
     qd = bf(n, s.q_width)
     gd = pd.view(n, -1)[:, s.g_col:]
     t.add("vimodra", "decode latent attention (absorb + ring + expand)",
-          lambda: A.latent_decode(qd, sd["ring"], att.w_ukv[:H * s.dim], att.w_uvt, gd, s, rope.cos, rope.sin, lengths),
+          lambda: att.attend_token(qd, sd["ring"], gd, lengths),
           2.0 * (n * w * s.cw + H * (s.dim + s.vdim) * s.rank), flops=2.0 * n * H * w * (s.cw + s.rank))
     t.add("vimodra", "decode gemm: q / kv latents + gate", lambda: ops.linear(hd, att.w_in), 2.0 * att.w_in.numel())
     ad = bf(n, s.o_pad)

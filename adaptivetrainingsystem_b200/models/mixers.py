@@ -90,12 +90,21 @@ class LatentAttention(_Weights):
         uvt = torch.zeros(s.heads, s.rank, pad8(s.vdim), dtype=dtype, device=device)
         uvt[..., :s.vdim] = uv.to(device=device, dtype=dtype).view(s.heads, s.vdim, s.rank).transpose(1, 2)
         self.put("w_uvt", uvt)
+        self.w_ukt = None   # key expansion transposed per head, for the tensor-core decode kernels
+        if torch.device(device).type == "cuda" and latent_ops.decode_mma_ok(s, dtype):
+            self.put("w_ukt_", uk.to(device=device, dtype=dtype).view(s.heads, s.dim, s.rank).transpose(1, 2).contiguous())
+            self.w_ukt = self.w_ukt_
         self.put("w_o", padded(take("o"), Dp, s.o_pad, dtype, device))
         self.put("q_norm", vector(take("dq.norm"), device))
         self.put("kv_norm", vector(take("dkv.norm"), device))
 
     def state(self, batch: int, max_len: int, dtype, device) -> Dict[str, torch.Tensor]:
         return {"ring": torch.zeros(batch, min(self.s.window, max_len), self.s.cwp, dtype=dtype, device=device)}
+
+    def attend_token(self, q: torch.Tensor, ring: torch.Tensor, gate: torch.Tensor, lengths: torch.Tensor) -> torch.Tensor:
+        s, rope = self.s, self._rope[0]
+        return latent_ops.latent_decode(q, ring, self.w_ukv[:s.heads * s.dim], self.w_uvt, gate, s, rope.cos, rope.sin, lengths, self.w_ukt,
+                                        self.w_ukv[s.v_col:])
 
     def forward(self, h: torch.Tensor, st: Dict[str, torch.Tensor], step: Step) -> torch.Tensor:
         s, rope, ring = self.s, self._rope[0], st["ring"]
@@ -104,7 +113,7 @@ class LatentAttention(_Weights):
         if step.lengths is not None:
             cq, _, _ = latent_ops.latent_context(proj, s, self.q_norm, self.kv_norm, rope.cos, rope.sin, ring, lengths=step.lengths, active=step.active)
             q = ops.linear(cq, self.w_uq)
-            return latent_ops.latent_decode(q, ring, self.w_ukv[:s.heads * s.dim], self.w_uvt, gate, s, rope.cos, rope.sin, step.lengths)
+            return self.attend_token(q, ring, gate, step.lengths)
         cq, ctx, n_old = latent_ops.latent_context(proj, s, self.q_norm, self.kv_norm, rope.cos, rope.sin, ring, pos0=step.pos0)
         q = ops.linear(cq, self.w_uq)
         kv = ops.linear(ctx.view(-1, s.cwp)[:, :s.rank], self.w_ukv[:, :s.rank]).view(step.B, n_old + step.L, -1)

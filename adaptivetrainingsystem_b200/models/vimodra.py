@@ -31,7 +31,7 @@ class Vimodra(nn.Module):
 
     # csrc files a program needs that only runs this model's step function
     KERNEL_SOURCES = ("gemm_tcgen05.cu", "dyt.cu", "latent_attention.cu",
-                      "attention_window_tcgen05.cu", "delta_rule.cu")
+                      "latent_decode.cu", "attention_window_tcgen05.cu", "delta_rule.cu")
     # decode steps over pool rows of different lengths work without a captured graph too
     eager_row_decode = True
 

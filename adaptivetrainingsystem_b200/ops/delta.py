@@ -154,7 +154,7 @@ def delta_scan(mixed: torch.Tensor, rlen: torch.Tensor, gb: torch.Tensor, state:
         return out
     dev = mixed.device
     groups = (L + GROUP - 1) // GROUP
-    coef = torch.empty(B, groups, H, GROUP, 2 * GROUP, dtype=torch.float32, device=dev)
+    coef = torch.empty(B, groups, H, 2 * GROUP * GROUP + 3 * GROUP + 8, dtype=torch.float32, device=dev)   # layout: csrc/delta_rule.cu
     o = torch.empty(B * L, H * s.vdim, dtype=mixed.dtype, device=dev)
     _call("ats_delta_scan", _Scan(_p(mixed), mixed.stride(0), _p(rlen), _p(gb), _p(coef), _p(state), state.stride(0), _p(o), o.stride(0), B, L, H, KH, s.dim, s.vdim,
                                   groups, int(fresh)), mixed)

@@ -24,6 +24,8 @@ def pad8(n: int) -> int:
 
 # ATS_WINDOW_TC=0: portions of a prompt use the general window kernel for every shape (for comparison)
 WINDOW_TC = os.environ.get("ATS_WINDOW_TC", "1") == "1"
+# ATS_LATENT_DECODE_MMA=0: decode steps use the general kernels for every shape (for comparison)
+DECODE_MMA = os.environ.get("ATS_LATENT_DECODE_MMA", "1") == "1"
 
 
 @dataclass(frozen=True)
@@ -227,10 +229,18 @@ def window_attention(q: torch.Tensor, kv: torch.Tensor, ctx: torch.Tensor, gate:
     return out
 
 
+def decode_mma_ok(s: LatentShape, dtype: torch.dtype) -> bool:
+    """The tensor-core decode kernels cover these sizes (the model then keeps the key expansion transposed per head)."""
+    return (dtype == torch.bfloat16 and DECODE_MMA and s.rank in (128, 256, 384, 512) and s.dim % 32 == 0 and s.dim <= 512 and s.rot % 32 == 0 and 32 <= s.rot <= 128
+            and s.vdim % 8 == 0)
+
+
 def latent_decode(q: torch.Tensor, ring: torch.Tensor, w_uk: torch.Tensor, w_uv_t: torch.Tensor, gate: Optional[torch.Tensor], s: LatentShape,
-                  cos: torch.Tensor, sin: torch.Tensor, lengths: torch.Tensor) -> torch.Tensor:
+                  cos: torch.Tensor, sin: torch.Tensor, lengths: torch.Tensor, w_ukt: Optional[torch.Tensor] = None,
+                  w_uv: Optional[torch.Tensor] = None) -> torch.Tensor:
     """One query token per sequence against its ring (which already holds the token's own entry).  q [B, q_width] not yet rotated;
-    w_uk [H * dim, >= rank], w_uv_t [H, rank, >= vdim] -> gated output [B, o_pad]."""
+    w_uk [H * dim, >= rank], w_uv_t [H, rank, >= vdim] -> gated output [B, o_pad].  With w_ukt [H, rank, dim] and w_uv
+    [H * vdim, >= rank] (shapes of :func:`decode_mma_ok`) everything runs on tensor cores."""
     B, R = ring.shape[:2]
     H, dq = s.heads, s.dim + s.rot
     if not q.is_cuda:
@@ -248,6 +258,20 @@ def latent_decode(q: torch.Tensor, ring: torch.Tensor, w_uk: torch.Tensor, w_uv_
             out[b, :H * s.vdim] = o.to(q.dtype)
         return out
     dev = q.device
+    if w_ukt is not None and w_uv is not None and R <= 64 * 4096:
+        # enough chunks to give every SM two, none smaller than a 64-row tile, at most 64 per sequence
+        chunk = max(64, (R * B * ((H + 15) // 16) // 296 + 63) // 64 * 64, (R + 64 * 64 - 1) // (64 * 64) * 64)
+        n_chunks = (R + chunk - 1) // chunk
+        qa = torch.empty(B, H, s.rank, dtype=q.dtype, device=dev)
+        part_o = torch.empty(B, H, n_chunks, s.rank, dtype=torch.float32, device=dev)
+        part_ml = torch.empty(B, H, n_chunks, 2, dtype=torch.float32, device=dev)
+        out = torch.empty(B, s.o_pad, dtype=q.dtype, device=dev)
+        f = _lib.cuda_lib().ats_latent_decode_mma
+        f.restype, f.argtypes = _ci, [_vp, _cll, _vp, _vp, _ci, _vp, _cll, _vp, _vp, _vp, _vp, _cll, _vp, _vp, _vp, _vp, _cll] + [_ci] * 10 + [_cf, _vp]
+        _lib.check(f(_p(q), q.stride(0), _p(w_ukt), _p(w_uv), w_uv.stride(0), _p(ring), ring.stride(0), _p(lengths), _p(cos), _p(sin), _p(gate),
+                     0 if gate is None else gate.stride(0), _p(qa), _p(part_o), _p(part_ml), _p(out), out.stride(0), B, H, s.dim, s.rot, s.rank, s.vdim, s.cwp, R,
+                     chunk, n_chunks, s.scale, _lib.stream_ptr(dev)), "ats_latent_decode_mma")
+        return out
     qa = torch.empty(B, H, s.cwp, dtype=q.dtype, device=dev)
     _call("ats_latent_absorb", _Absorb(_p(q), q.stride(0), _p(w_uk), w_uk.stride(0), _p(cos), _p(sin), _p(lengths), _p(qa), B, H, s.dim, s.rot, s.rank, s.cwp), q)
     chunk = 64

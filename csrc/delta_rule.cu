@@ -96,6 +96,81 @@ __global__ void __launch_bounds__(256) delta_prep_kernel(const DeltaArgs p) {
   }
 }
 
+// The same for portions whose heads are whole 16-byte pieces: a thread owns eight channels and walks PT consecutive tokens with the
+// convolution's inputs in registers; the lanes of a head (dim / 8 of them, a power of two) add up its length with shuffles.
+constexpr int PT = 16;
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(256) delta_prep_vec_kernel(const DeltaArgs p) {
+  pdl_prologue();
+  const int pieces = p.C >> 3, per_block = (pieces + 255) / 256, blocks_t = (p.L + PT - 1) / PT;
+  const int piece = (blockIdx.x % per_block) * 256 + threadIdx.x;
+  const int tb = (blockIdx.x / per_block) % blocks_t, b = blockIdx.x / per_block / blocks_t;
+  const int t0 = tb * PT, t1 = min(p.L, t0 + PT);
+  const bool live = piece < pieces;  // C / 8 need not fill the last block: idle lanes still take part in the shuffles
+  const int c = live ? piece * 8 : 0;
+  const T* in = static_cast<const T*>(p.proj) + (long long)b * p.L * p.ld + c;
+  const T* tail = static_cast<const T*>(p.tail) + (long long)b * p.tail_bs + c;
+  T* out = static_cast<T*>(p.mixed) + (long long)b * p.L * p.ldm + c;
+  float w[TAPS][8], x[TAPS][8];  // x[j]: the input j tokens back (x[0] = current)
+#pragma unroll
+  for (int e = 0; e < 8; ++e)
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) w[j][e] = p.conv[(long long)(c + e) * TAPS + TAPS - 1 - j];
+#pragma unroll
+  for (int j = 1; j < TAPS; ++j) {
+    const int t = t0 - j;
+    if (t >= 0) Typed<T>::load8(in + (long long)t * p.ld, x[j - 1]);
+    else if (p.pos0 > 0) Typed<T>::load8(tail + (long long)(TAPS - 1 + t) * p.C, x[j - 1]);
+    else
+#pragma unroll
+      for (int e = 0; e < 8; ++e) x[j - 1][e] = 0.f;
+  }
+  const int lanes = p.dim >> 3, kd = p.KH * p.dim;
+  const bool qk = live && c < 2 * kd;
+  float nx[8];
+  Typed<T>::load8(in + (long long)t0 * p.ld, nx);
+  for (int t = t0; t < t1; ++t) {
+#pragma unroll
+    for (int j = TAPS - 1; j > 0; --j)
+#pragma unroll
+      for (int e = 0; e < 8; ++e) x[j][e] = x[j - 1][e];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) x[0][e] = nx[e];
+    if (t + 1 < t1) Typed<T>::load8(in + (long long)(t + 1) * p.ld, nx);
+    float y[8], ss = 0.f;
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      float acc = 0.f;
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) acc += x[j][e] * w[j][e];
+      y[e] = acc * Typed<T>::sigmoid_(acc);
+    }
+    Typed<T>::round8(y);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) ss += y[e] * y[e];
+    if (live) Typed<T>::store8(out + (long long)t * p.ldm, y);
+    for (int off = lanes >> 1; off > 0; off >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, off);
+    if (qk && (piece & (lanes - 1)) == 0) {
+      const int head = piece / lanes;
+      p.rlen[((long long)b * p.L + t) * 2 * p.KH + head] = (head < p.KH ? 1.f / sqrtf(float(p.dim)) : 1.f) / sqrtf(ss + 1e-6f);
+    }
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) delta_gates_kernel(const DeltaArgs p) {
+  pdl_prologue();
+  const long long i = blockIdx.x * 256ll + threadIdx.x;
+  if (i >= (long long)p.B * p.L * p.H) return;
+  const long long row = i / p.H;
+  const int h = int(i % p.H);
+  const T* in = static_cast<const T*>(p.proj) + row * p.ld;
+  const float a = Typed<T>::load(in + p.a_col + h) + p.dt_bias[h], bt = Typed<T>::load(in + p.b_col + h);
+  const float sp = a > 20.f ? a : log1pf(expf(a));
+  p.gb[row * 2 * p.H + h] = expf(p.neg_rate[h] * sp);
+  p.gb[row * 2 * p.H + p.H + h] = 1.f / (1.f + expf(-bt));
+}
+
 // After a portion: the last taps - 1 inputs of every channel (one thread per channel, oldest first, in place).
 template <typename T>
 __global__ void __launch_bounds__(256) delta_tail_kernel(const DeltaArgs p) {
@@ -116,13 +191,17 @@ __global__ void __launch_bounds__(256) delta_tail_kernel(const DeltaArgs p) {
 
 // ------------------------------------------------------------------------------------------------ portions
 constexpr int DC = 8;  // tokens per group
+// Per group and head: [DC][2 * DC] inverse of the triangular system (times beta) and read-out coefficients, then per token
+// G_i / |k_i|, G_i dim^-1/2 / |q_i|, D_Ci / |k_i| (G_i = g_1 .. g_i, D_Ci = g_{i+1} .. g_C), then G_C: with the lengths folded in
+// here, the sequential kernel works on the raw q and k.
+constexpr int CO = 2 * DC * DC + 3 * DC + 8;
 
 struct ScanArgs {
   const void* mixed;
   long long ldm;
   const float* rlen;
   const float* gb;
-  float* coef;             // [B, groups, H, DC, 2 * DC]: inverse of the triangular system (times beta), read-out coefficients
+  float* coef;             // [B, groups, H, CO]: see CO
   float* state;            // [B, H, dim, vdim]
   long long state_bs;
   void* o;                 // [B * L, H * vdim]
@@ -190,7 +269,7 @@ __global__ void __launch_bounds__(128) delta_pairs_kernel(const ScanArgs p) {
     // column c of (1 + M)^-1, M_ij = beta_i D_ij kk_ij: forward substitution; the result is multiplied by beta_c (the right-hand
     // side of the system is beta_c (v_c - G_c S^T k_c))
     float y[DC];
-    float* co = p.coef + ((((long long)b * p.groups + grp) * p.H + h) * DC) * 2 * DC;
+    float* co = p.coef + (((long long)b * p.groups + grp) * p.H + h) * CO;
 #pragma unroll
     for (int i = 0; i < DC; ++i) {
       float acc = i == c ? 1.f : 0.f, dec = 1.f;
@@ -209,17 +288,24 @@ __global__ void __launch_bounds__(128) delta_pairs_kernel(const ScanArgs p) {
       if (i > c) dec *= g[i];
       co[i * 2 * DC + DC + c] = i >= c ? dec * s_kq[warp][i][c] : 0.f;
     }
+    float G = 1.f, GC = 1.f;
+#pragma unroll
+    for (int i = 0; i < DC; ++i) {
+      if (i <= c) G *= g[i];
+      GC *= g[i];
+    }
+    const float rk = c < n ? rl[(long long)c * 2 * p.KH + p.KH + kh] : 0.f, rq = c < n ? rl[(long long)c * 2 * p.KH + kh] : 0.f;
+    co += 2 * DC * DC;
+    co[c] = G * rk;
+    co[DC + c] = G * rq;
+    co[2 * DC + c] = dec * rk;  // dec has become g_{c+1} .. g_C
+    if (c == 0) co[3 * DC] = GC;
   }
 }
 
-__device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
-  float2 r;
-  asm("{\n\t.reg .b64 x, y, z, w;\n\tmov.b64 x, {%2, %3};\n\tmov.b64 y, {%4, %5};\n\tmov.b64 z, {%6, %7};\n\t"
-      "fma.rn.f32x2 w, x, y, z;\n\tmov.b64 {%0, %1}, w;\n\t}"
-      : "=f"(r.x), "=f"(r.y)
-      : "f"(a.x), "f"(a.y), "f"(b.x), "f"(b.y), "f"(c.x), "f"(c.y));
-  return r;
-}
+__device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) { return __ffma2_rn(a, b, c); }  // one packed instruction
+// Keeps the compiler from requesting the shared-memory rows of more tokens than registers can hold.
+__device__ __forceinline__ void pace() { asm volatile("" ::: "memory"); }
 
 // Eight per-lane values of which the sum over the eight lanes of a group is wanted: lane l ends up with the sum of value l.
 __device__ __forceinline__ float transpose_sum8(float (&v)[DC], int l) {
@@ -236,15 +322,16 @@ __device__ __forceinline__ float transpose_sum8(float (&v)[DC], int l) {
 }
 
 // EPL: state rows per lane (dim <= 8 * EPL), CPL: value columns per lane group.  CTA = 4 warps of 4 lane groups -> 16 * CPL columns
-// of one head.
-template <typename T, int EPL, int CPL>
-__global__ void __launch_bounds__(128) delta_scan_kernel(const ScanArgs p) {
+// of one head.  The next group's q, k, v and constants are requested before this group's products and stored to the other half of
+// shared memory after them.
+template <typename T, int EPL, int CPL, int OCC>
+__global__ void __launch_bounds__(128, OCC) delta_scan_kernel(const ScanArgs p) {
   pdl_prologue();
   constexpr int DK = 8 * EPL;
-  __shared__ __align__(16) float s_k[2][DC][DK];
-  __shared__ __align__(16) float s_q[2][DC][DK];
-  __shared__ float s_c[2][DC][2 * DC + 1];
-  __shared__ float s_g[2][2][DC];           // G_i = g_1 .. g_i and D_Ci = g_{i+1} .. g_C
+  constexpr int VEC = 16 / int(sizeof(T));             // elements per 16-byte piece
+  constexpr int NP = (2 * DC * DK / VEC + 127) / 128;  // pieces of q and k per thread and group
+  __shared__ __align__(16) float s_kq[2][2][DC][DK];   // [buffer][k, q]
+  __shared__ __align__(16) float s_c[2][CO];
   const int tid = threadIdx.x, lane = tid & 31, l8 = lane & 7;
   const int h = blockIdx.y, b = blockIdx.z, kh = h / (p.H / p.KH);
   const int col0 = (blockIdx.x * 16 + (tid >> 3)) * CPL;
@@ -260,102 +347,126 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const ScanArgs p) {
       S[c][e].y = (ok && d + 1 < p.dim) ? st[(long long)(d + 1) * p.vdim + col0 + c] : 0.f;
     }
   const T* base = static_cast<const T*>(p.mixed) + (long long)b * p.L * p.ldm;
-  auto stage = [&](int grp, int buf) {
+  const T* vbase = base + 2 * p.KH * p.dim + (long long)h * p.vdim + col0;
+  const float* cbase = p.coef + ((long long)b * p.groups * p.H + h) * CO;
+  const bool vec = (p.dim % VEC) == 0;  // rows are whole 16-byte pieces (p.ldm is a multiple of 8)
+  uint4 piece[NP];
+  float4 cpiece;
+  float vnext[CPL];
+  auto request = [&](int grp) {
     const int t0 = grp * DC, n = min(DC, p.L - t0);
-    const long long row0 = (long long)b * p.L + t0;
-    for (int i = tid; i < DC * DK; i += 128) {
-      const int t = i / DK, d = i % DK;
-      float kv = 0.f, qv = 0.f;
-      if (t < n && d < p.dim) {
-        const T* r = base + (t0 + t) * p.ldm + d;
-        kv = Typed<T>::load(r + (long long)(p.KH + kh) * p.dim) * p.rlen[(row0 + t) * 2 * p.KH + p.KH + kh];
-        qv = Typed<T>::load(r + (long long)kh * p.dim) * p.rlen[(row0 + t) * 2 * p.KH + kh];
-      }
-      s_k[buf][t][d] = kv;
-      s_q[buf][t][d] = qv;
-    }
-    const float* co = p.coef + (((long long)b * p.groups + grp) * p.H + h) * DC * 2 * DC;
-    for (int i = tid; i < DC * 2 * DC; i += 128) s_c[buf][i / (2 * DC)][i % (2 * DC)] = co[i];
-    if (tid < DC) {
-      float G = 1.f, D = 1.f;
-      for (int i = 0; i < DC; ++i) {
-        const float g = i < n ? p.gb[(row0 + i) * 2 * p.H + h] : 1.f;
-        if (i <= tid) G *= g;
-        else D *= g;
-      }
-      s_g[buf][0][tid] = G;
-      s_g[buf][1][tid] = D;
-    }
-  };
-  stage(0, 0);
-  __syncthreads();
-  for (int grp = 0; grp < p.groups; ++grp) {
-    const int buf = grp & 1, t0 = grp * DC, n = min(DC, p.L - t0);
-    // value of this lane's token (lane l8 <-> token l8), requested before the products
-    float v[CPL];
 #pragma unroll
-    for (int c = 0; c < CPL; ++c)
-      v[c] = (l8 < n && col0 + c < p.vdim)
-                 ? Typed<T>::load(base + (t0 + l8) * p.ldm + 2 * p.KH * p.dim + (long long)h * p.vdim + col0 + c) : 0.f;
-    if (grp + 1 < p.groups) stage(grp + 1, buf ^ 1);
-    float sk[CPL][DC], sq[CPL][DC];
+    for (int u = 0; u < NP; ++u) {
+      const int i = (u * 128 + tid) * VEC, which = i / (DC * DK), t = (i / DK) % DC, d = i % DK;
+      const T* src = base + (long long)(t0 + t) * p.ldm + (long long)(which ? kh : p.KH + kh) * p.dim + d;
+      piece[u] = make_uint4(0, 0, 0, 0);
+      if (which < 2 && t < n && d < p.dim) {
+        if (vec) piece[u] = *reinterpret_cast<const uint4*>(src);
+        else {
+          T* e = reinterpret_cast<T*>(&piece[u]);
+          for (int x = 0; x < VEC && d + x < p.dim; ++x) e[x] = src[x];
+        }
+      }
+    }
+    if (tid < CO / 4) cpiece = *reinterpret_cast<const float4*>(cbase + (long long)grp * p.H * CO + tid * 4);
+#pragma unroll
+    for (int c = 0; c < CPL; ++c) vnext[c] = (l8 < n && col0 + c < p.vdim) ? Typed<T>::load(vbase + (long long)(t0 + l8) * p.ldm + c) : 0.f;
+  };
+  auto deposit = [&](int buf) {
+#pragma unroll
+    for (int u = 0; u < NP; ++u) {
+      if ((u * 128 + tid) * VEC >= 2 * DC * DK) continue;
+      float* dst = &s_kq[buf][0][0][0] + (u * 128 + tid) * VEC;
+      float f[8];
+      const T* e = reinterpret_cast<const T*>(&piece[u]);
+#pragma unroll
+      for (int x = 0; x < VEC; ++x) f[x] = Typed<T>::load(e + x);
+#pragma unroll
+      for (int x = 0; x < VEC; x += 4) *reinterpret_cast<float4*>(dst + x) = make_float4(f[x], f[x + 1], f[x + 2], f[x + 3]);
+    }
+    if (tid < CO / 4) *reinterpret_cast<float4*>(&s_c[buf][tid * 4]) = cpiece;
+  };
+  // sum over the state rows of S times the eight k (which = 0) or q (1) vectors of the group; lane l8 keeps token l8
+  auto products = [&](int buf, int which, float (&out)[CPL]) {
+    float acc[CPL][DC];
 #pragma unroll
     for (int i = 0; i < DC; ++i) {
-      float2 ak[CPL], aq[CPL];
+      float2 a[CPL];
 #pragma unroll
-      for (int c = 0; c < CPL; ++c) ak[c] = aq[c] = make_float2(0.f, 0.f);
+      for (int c = 0; c < CPL; ++c) a[c] = make_float2(0.f, 0.f);
 #pragma unroll
       for (int e = 0; e < EPL / 4; ++e) {
-        const float4 k4 = *reinterpret_cast<const float4*>(&s_k[buf][i][(e * 8 + l8) * 4]);
-        const float4 q4 = *reinterpret_cast<const float4*>(&s_q[buf][i][(e * 8 + l8) * 4]);
+        const float4 k4 = *reinterpret_cast<const float4*>(&s_kq[buf][which][i][(e * 8 + l8) * 4]);
 #pragma unroll
         for (int c = 0; c < CPL; ++c) {
-          ak[c] = fma2(S[c][2 * e], make_float2(k4.x, k4.y), ak[c]);
-          ak[c] = fma2(S[c][2 * e + 1], make_float2(k4.z, k4.w), ak[c]);
-          aq[c] = fma2(S[c][2 * e], make_float2(q4.x, q4.y), aq[c]);
-          aq[c] = fma2(S[c][2 * e + 1], make_float2(q4.z, q4.w), aq[c]);
+          a[c] = fma2(S[c][2 * e], make_float2(k4.x, k4.y), a[c]);
+          a[c] = fma2(S[c][2 * e + 1], make_float2(k4.z, k4.w), a[c]);
         }
       }
 #pragma unroll
-      for (int c = 0; c < CPL; ++c) {
-        sk[c][i] = ak[c].x + ak[c].y;
-        sq[c][i] = aq[c].x + aq[c].y;
-      }
+      for (int c = 0; c < CPL; ++c) acc[c][i] = a[c].x + a[c].y;
+      if (i & 1) pace();
     }
-    const float G = s_g[buf][0][l8], GC = s_g[buf][0][DC - 1];
-    float w[CPL][DC];  // D_Cj u_j of every token, in every lane
+#pragma unroll
+    for (int c = 0; c < CPL; ++c) out[c] = transpose_sum8(acc[c], l8);
+  };
+  request(0);
+  deposit(0);
+  __syncthreads();
+  for (int grp = 0; grp < p.groups; ++grp) {
+    const int buf = grp & 1, t0 = grp * DC, n = min(DC, p.L - t0);
+    float v[CPL];
+#pragma unroll
+    for (int c = 0; c < CPL; ++c) v[c] = vnext[c];
+    if (grp + 1 < p.groups) request(grp + 1);
+    const float* co = s_c[buf];
+    float sk[CPL], w[CPL][DC];
+    products(buf, 0, sk);
+    const float gk = co[2 * DC * DC + l8], gq = co[2 * DC * DC + DC + l8], GC = co[2 * DC * DC + 3 * DC];
+    __align__(16) float row[2 * DC];
+#pragma unroll
+    for (int j = 0; j < 2 * DC; j += 4) *reinterpret_cast<float4*>(&row[j]) = *reinterpret_cast<const float4*>(&co[l8 * 2 * DC + j]);
+    float o[CPL];
 #pragma unroll
     for (int c = 0; c < CPL; ++c) {
-      const float a = transpose_sum8(sk[c], l8), r = transpose_sum8(sq[c], l8);
-      const float rhs = v[c] - G * a;
-      float u = 0.f, o = G * r;
+      const float rhs = v[c] - gk * sk[c];
+      float u = 0.f;
 #pragma unroll
-      for (int j = 0; j < DC; ++j) u += s_c[buf][l8][j] * __shfl_sync(0xffffffffu, rhs, j, 8);
+      for (int j = 0; j < DC; ++j) u += row[j] * __shfl_sync(0xffffffffu, rhs, j, 8);
+      o[c] = 0.f;
 #pragma unroll
       for (int j = 0; j < DC; ++j) {
-        const float uj = __shfl_sync(0xffffffffu, u, j, 8);
-        o += s_c[buf][l8][DC + j] * uj;
-        w[c][j] = uj * s_g[buf][1][j];
+        w[c][j] = __shfl_sync(0xffffffffu, u, j, 8);
+        o[c] += row[DC + j] * w[c][j];
       }
-      if (l8 < n && col0 + c < p.vdim)
-        Typed<T>::store(static_cast<T*>(p.o) + ((long long)b * p.L + t0 + l8) * p.ldo + (long long)h * p.vdim + col0 + c, o);
     }
+    products(buf, 1, sk);
+#pragma unroll
+    for (int c = 0; c < CPL; ++c)
+      if (l8 < n && col0 + c < p.vdim)
+        Typed<T>::store(static_cast<T*>(p.o) + ((long long)b * p.L + t0 + l8) * p.ldo + (long long)h * p.vdim + col0 + c, o[c] + gq * sk[c]);
 #pragma unroll
     for (int c = 0; c < CPL; ++c)
 #pragma unroll
       for (int e = 0; e < EPL / 2; ++e) S[c][e] = make_float2(S[c][e].x * GC, S[c][e].y * GC);
 #pragma unroll
-    for (int j = 0; j < DC; ++j)
+    for (int j = 0; j < DC; ++j) {
+      const float dk = co[2 * DC * DC + 2 * DC + j];
+      float2 uu[CPL];
+#pragma unroll
+      for (int c = 0; c < CPL; ++c) uu[c] = make_float2(w[c][j] * dk, w[c][j] * dk);
 #pragma unroll
       for (int e = 0; e < EPL / 4; ++e) {
-        const float4 k4 = *reinterpret_cast<const float4*>(&s_k[buf][j][(e * 8 + l8) * 4]);
+        const float4 k4 = *reinterpret_cast<const float4*>(&s_kq[buf][0][j][(e * 8 + l8) * 4]);
 #pragma unroll
         for (int c = 0; c < CPL; ++c) {
-          const float2 uu = make_float2(w[c][j], w[c][j]);
-          S[c][2 * e] = fma2(make_float2(k4.x, k4.y), uu, S[c][2 * e]);
-          S[c][2 * e + 1] = fma2(make_float2(k4.z, k4.w), uu, S[c][2 * e + 1]);
+          S[c][2 * e] = fma2(make_float2(k4.x, k4.y), uu[c], S[c][2 * e]);
+          S[c][2 * e + 1] = fma2(make_float2(k4.z, k4.w), uu[c], S[c][2 * e + 1]);
         }
       }
+      if (j & 1) pace();
+    }
+    if (grp + 1 < p.groups) deposit(buf ^ 1);  // the other half was last read one group ago
     __syncthreads();
   }
 #pragma unroll
@@ -406,6 +517,27 @@ __global__ void __launch_bounds__(256) delta_output_kernel(const DeltaOutArgs p)
   }
   if (h == 0)
     for (int c = p.H * p.vdim + lane; c < p.ldout; c += 32) Typed<T>::store(out + c, 0.f);
+}
+
+// The same with eight values per thread: vdim / 8 lanes (a power of two) per head.
+template <typename T>
+__global__ void __launch_bounds__(256) delta_output_vec_kernel(const DeltaOutArgs p) {
+  pdl_prologue();
+  const int lanes = p.vdim >> 3;
+  const long long i = blockIdx.x * 256ll + threadIdx.x, total = p.rows * p.H * lanes;
+  const bool live = i < total;
+  const long long hr = (live ? i : 0) / lanes, row = hr / p.H;
+  const int h = int(hr % p.H), c = int((live ? i : 0) % lanes) * 8;
+  float v[8], z[8], ss = 0.f;
+  Typed<T>::load8(static_cast<const T*>(p.o) + row * p.ldo + (long long)h * p.vdim + c, v);
+  Typed<T>::load8(static_cast<const T*>(p.gate) + row * p.ldg + (long long)h * p.vdim + c, z);
+#pragma unroll
+  for (int e = 0; e < 8; ++e) ss += v[e] * v[e];
+  for (int off = lanes >> 1; off > 0; off >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, off);
+  const float r = 1.f / sqrtf(ss / float(p.vdim) + p.eps);
+#pragma unroll
+  for (int e = 0; e < 8; ++e) v[e] *= r * p.w[c + e] * z[e] * Typed<T>::sigmoid_(z[e]);
+  if (live) Typed<T>::store8(static_cast<T*>(p.out) + row * p.ldout + (long long)h * p.vdim + c, v);
 }
 
 // ------------------------------------------------------------------------------------------------ decoding
@@ -508,10 +640,10 @@ static int launch_scan(const ScanArgs& p, cudaStream_t s) {
   const long long pw = (long long)p.B * p.groups * p.KH;
   launch_pdl(delta_pairs_kernel<T>, dim3(unsigned((pw + 3) / 4)), dim3(128), 0, s, p);
   auto grid = [&](int cpl) { return dim3((p.vdim + 16 * cpl - 1) / (16 * cpl), p.H, p.B); };
-  if (p.dim <= 32) launch_pdl(delta_scan_kernel<T, 4, 2>, grid(2), dim3(128), 0, s, p);
-  else if (p.dim <= 64) launch_pdl(delta_scan_kernel<T, 8, 2>, grid(2), dim3(128), 0, s, p);
-  else if (p.dim <= 128) launch_pdl(delta_scan_kernel<T, 16, 2>, grid(2), dim3(128), 0, s, p);
-  else if (p.dim <= 256) launch_pdl(delta_scan_kernel<T, 32, 1>, grid(1), dim3(128), 0, s, p);
+  if (p.dim <= 32) launch_pdl(delta_scan_kernel<T, 4, 2, 4>, grid(2), dim3(128), 0, s, p);
+  else if (p.dim <= 64) launch_pdl(delta_scan_kernel<T, 8, 2, 4>, grid(2), dim3(128), 0, s, p);
+  else if (p.dim <= 128) launch_pdl(delta_scan_kernel<T, 16, 2, 4>, grid(2), dim3(128), 0, s, p);
+  else if (p.dim <= 256) launch_pdl(delta_scan_kernel<T, 32, 1, 3>, grid(1), dim3(128), 0, s, p);
   else return 1006;
   return int(cudaGetLastError());
 }
@@ -537,20 +669,41 @@ static int launch_step(const StepArgs& p, cudaStream_t s) {
 using namespace ats;
 
 // Every entry point takes its argument struct by address (the ctypes mirror is in ops/delta.py); `fp32` selects the element type.
-ATS_API int ats_delta_prep(const DeltaArgs* p, int fp32, void* stream) {
-  if (p->taps < 1 || (p->lengths && p->L != 1) || p->KH < 1 || p->H % p->KH) return 1006;
-  const long long warps = (long long)p->B * p->L * (2 * p->KH + p->H + 1);
-  if (warps <= 0) return 0;
-  cudaStream_t s = static_cast<cudaStream_t>(stream);
-  const dim3 grid(unsigned((warps + 7) / 8));
-  if (fp32) launch_pdl(delta_prep_kernel<float>, grid, dim3(256), 0, s, *p);
-  else launch_pdl(delta_prep_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, *p);
-  if (!p->lengths && p->taps > 1) {
-    const dim3 tg((p->C + 255) / 256, p->B);
-    if (fp32) launch_pdl(delta_tail_kernel<float>, tg, dim3(256), 0, s, *p);
-    else launch_pdl(delta_tail_kernel<__nv_bfloat16>, tg, dim3(256), 0, s, *p);
+static bool pow2_lanes(int width) { return (width & 7) == 0 && width <= 256 && ((width >> 3) & ((width >> 3) - 1)) == 0; }
+
+template <typename T>
+static int launch_prep(const DeltaArgs& p, cudaStream_t s) {
+  const bool aligned = (p.ld & 7) == 0 && (p.ldm & 7) == 0 && (p.C & 7) == 0 && (reinterpret_cast<uintptr_t>(p.proj) & 15) == 0 &&
+                       (reinterpret_cast<uintptr_t>(p.tail) & 15) == 0 && (p.tail_bs & 7) == 0;
+  if (!p.lengths && aligned && pow2_lanes(p.dim) && (p.vdim & 7) == 0 && p.taps >= 2 && p.taps <= 4) {
+    const long long blocks = (long long)p.B * ((p.L + PT - 1) / PT) * (((p.C >> 3) + 255) / 256);
+    if (p.taps == 2) launch_pdl(delta_prep_vec_kernel<T, 2>, dim3(unsigned(blocks)), dim3(256), 0, s, p);
+    else if (p.taps == 3) launch_pdl(delta_prep_vec_kernel<T, 3>, dim3(unsigned(blocks)), dim3(256), 0, s, p);
+    else launch_pdl(delta_prep_vec_kernel<T, 4>, dim3(unsigned(blocks)), dim3(256), 0, s, p);
+    launch_pdl(delta_gates_kernel<T>, dim3(unsigned(((long long)p.B * p.L * p.H + 255) / 256)), dim3(256), 0, s, p);
+  } else {
+    const long long warps = (long long)p.B * p.L * (2 * p.KH + p.H + 1);
+    launch_pdl(delta_prep_kernel<T>, dim3(unsigned((warps + 7) / 8)), dim3(256), 0, s, p);
+  }
+  if (!p.lengths && p.taps > 1) launch_pdl(delta_tail_kernel<T>, dim3((p.C + 255) / 256, p.B), dim3(256), 0, s, p);
+  return int(cudaGetLastError());
+}
+
+template <typename T>
+static int launch_output(const DeltaOutArgs& p, cudaStream_t s) {
+  const bool aligned = ((p.ldo | p.ldg | p.ldout) & 7) == 0 && ((reinterpret_cast<uintptr_t>(p.o) | reinterpret_cast<uintptr_t>(p.gate) | reinterpret_cast<uintptr_t>(p.out)) & 15) == 0;
+  if (aligned && pow2_lanes(p.vdim)) {  // heads x vdim is a multiple of 8: no padded columns
+    launch_pdl(delta_output_vec_kernel<T>, dim3(unsigned((p.rows * p.H * (p.vdim >> 3) + 255) / 256)), dim3(256), 0, s, p);
+  } else {
+    launch_pdl(delta_output_kernel<T>, dim3(unsigned((p.rows * p.H + 7) / 8)), dim3(256), 0, s, p);
   }
   return int(cudaGetLastError());
+}
+
+ATS_API int ats_delta_prep(const DeltaArgs* p, int fp32, void* stream) {
+  if (p->taps < 1 || (p->lengths && p->L != 1) || p->KH < 1 || p->H % p->KH) return 1006;
+  if (p->B <= 0 || p->L <= 0) return 0;
+  return fp32 ? launch_prep<float>(*p, static_cast<cudaStream_t>(stream)) : launch_prep<__nv_bfloat16>(*p, static_cast<cudaStream_t>(stream));
 }
 
 ATS_API int ats_delta_scan(const ScanArgs* p, int fp32, void* stream) {
@@ -560,13 +713,8 @@ ATS_API int ats_delta_scan(const ScanArgs* p, int fp32, void* stream) {
 }
 
 ATS_API int ats_delta_output(const DeltaOutArgs* p, int fp32, void* stream) {
-  const long long warps = p->rows * p->H;
-  if (warps <= 0) return 0;
-  cudaStream_t s = static_cast<cudaStream_t>(stream);
-  const dim3 grid(unsigned((warps + 7) / 8));
-  if (fp32) launch_pdl(delta_output_kernel<float>, grid, dim3(256), 0, s, *p);
-  else launch_pdl(delta_output_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, *p);
-  return int(cudaGetLastError());
+  if (p->rows <= 0) return 0;
+  return fp32 ? launch_output<float>(*p, static_cast<cudaStream_t>(stream)) : launch_output<__nv_bfloat16>(*p, static_cast<cudaStream_t>(stream));
 }
 
 ATS_API int ats_delta_step(const StepArgs* p, int fp32, void* stream) {

@@ -85,6 +85,79 @@ __global__ void __launch_bounds__(128) latent_context_kernel(const LatentArgs p)
   }
 }
 
+// The same when every part is whole 16-byte pieces: one warp per row, eight values per access.
+template <typename T>
+__global__ void __launch_bounds__(128) latent_context_vec_kernel(const LatentArgs p) {
+  pdl_prologue();
+  const int rows = p.n_old + p.L, lane = threadIdx.x & 31;
+  const long long r = blockIdx.x * 4ll + (threadIdx.x >> 5);
+  if (r >= (long long)p.B * rows) return;  // whole warp; no CTA barrier below
+  const int b = int(r / rows), j = int(r % rows), half = p.rot >> 1;
+  T* ring = static_cast<T*>(p.ring) + (long long)b * p.ring_bs;
+  float v[8], w[8];
+  if (j < p.n_old) {
+    const T* src = ring + (long long)((p.pos0 - p.n_old + j) % p.R) * p.cwp;
+    T* dst = static_cast<T*>(p.ctx) + r * p.cwp;
+    for (int c = lane * 8; c < p.cwp; c += 256) {
+      Typed<T>::load8(src + c, v);
+      Typed<T>::store8(dst + c, v);
+    }
+    return;
+  }
+  const long long row = (long long)b * p.L + j - p.n_old;
+  const T* in = static_cast<const T*>(p.proj) + row * p.ld;
+  const int pos = p.lengths ? p.lengths[b] : p.pos0 + j - p.n_old;
+  T* dst;
+  if (p.lengths) dst = (p.active && !p.active[b]) ? nullptr : ring + (long long)(pos % p.R) * p.cwp;
+  else dst = static_cast<T*>(p.ctx) + r * p.cwp;
+  float sq = 0.f, sc = 0.f;
+#pragma unroll 4
+  for (int c = lane * 8; c < p.q_rank; c += 256) {
+    Typed<T>::load8(in + p.q_col + c, v);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) sq += v[e] * v[e];
+  }
+#pragma unroll 2
+  for (int c = lane * 8; c < p.rank; c += 256) {
+    Typed<T>::load8(in + p.kv_col + c, v);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) sc += v[e] * v[e];
+  }
+  const float rq = 1.f / sqrtf(warp_sum(sq) / float(p.q_rank) + p.eps), rc = 1.f / sqrtf(warp_sum(sc) / float(p.rank) + p.eps);
+  T* cq = static_cast<T*>(p.cq) + row * p.q_pad;
+#pragma unroll 4
+  for (int c = lane * 8; c < p.q_rank; c += 256) {  // second read: from L1
+    Typed<T>::load8(in + p.q_col + c, v);
+    Typed<float>::load8(p.q_w + c, w);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) v[e] *= rq * w[e];
+    Typed<T>::store8(cq + c, v);
+  }
+  if (dst == nullptr) return;
+#pragma unroll 2
+  for (int c = lane * 8; c < p.rank; c += 256) {
+    Typed<T>::load8(in + p.kv_col + c, v);
+    Typed<float>::load8(p.kv_w + c, w);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) v[e] *= rc * w[e];
+    Typed<T>::store8(dst + c, v);
+  }
+  for (int m = lane * 8; m < half; m += 256) {
+    float u[8], x[8], cs[8], sn[8];
+    Typed<T>::load8(in + p.kv_col + p.rank + m, u);
+    Typed<T>::load8(in + p.kv_col + p.rank + half + m, x);
+    Typed<float>::load8(p.cos + (long long)pos * half + m, cs);
+    Typed<float>::load8(p.sin + (long long)pos * half + m, sn);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      v[e] = u[e] * cs[e] - x[e] * sn[e];
+      w[e] = x[e] * cs[e] + u[e] * sn[e];
+    }
+    Typed<T>::store8(dst + p.rank + m, v);
+    Typed<T>::store8(dst + p.rank + half + m, w);
+  }
+}
+
 struct FinishArgs {
   void* q;               // [B * L, ldq], head h at h * (dim + rot): its last `rot` values are rotated in place
   long long ldq;
@@ -116,6 +189,39 @@ __global__ void __launch_bounds__(128) latent_finish_kernel(const FinishArgs p) 
     const T* src = static_cast<const T*>(p.ctx) + ((long long)b * (p.n_old + p.L) + p.n_old + t) * p.cwp;
     T* dst = static_cast<T*>(p.ring) + (long long)b * p.ring_bs + (pos % p.R) * p.cwp;
     for (int c = threadIdx.x; c < p.cwp; c += blockDim.x) dst[c] = src[c];
+  }
+}
+
+// The same when the halves of the rotated part are whole 16-byte pieces: a thread rotates eight pairs or copies eight values.
+template <typename T>
+__global__ void __launch_bounds__(256) latent_finish_vec_kernel(const FinishArgs p) {
+  pdl_prologue();
+  const int half = p.rot >> 1, per_head = half >> 3, keep = min(p.L, p.R), cp = p.cwp >> 3;
+  const long long rot_n = (long long)p.B * p.L * p.H * per_head, total = rot_n + (long long)p.B * keep * cp;
+  for (long long i = blockIdx.x * 256ll + threadIdx.x; i < total; i += (long long)gridDim.x * 256) {
+    if (i < rot_n) {
+      const int m = int(i % per_head) * 8, h = int((i / per_head) % p.H);
+      const long long row = i / per_head / p.H, pos = p.pos0 + row % p.L;
+      T* d = static_cast<T*>(p.q) + row * p.ldq + (long long)h * (p.dim + p.rot) + p.dim + m;
+      float u[8], x[8], cs[8], sn[8], v[8], w[8];
+      Typed<T>::load8(d, u);
+      Typed<T>::load8(d + half, x);
+      Typed<float>::load8(p.cos + pos * half + m, cs);
+      Typed<float>::load8(p.sin + pos * half + m, sn);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        v[e] = u[e] * cs[e] - x[e] * sn[e];
+        w[e] = x[e] * cs[e] + u[e] * sn[e];
+      }
+      Typed<T>::store8(d, v);
+      Typed<T>::store8(d + half, w);
+    } else {
+      const long long k = i - rot_n;
+      const int c = int(k % cp) * 8, t = p.L - keep + int((k / cp) % keep), b = int(k / cp / keep);
+      float v[8];
+      Typed<T>::load8(static_cast<const T*>(p.ctx) + ((long long)b * (p.n_old + p.L) + p.n_old + t) * p.cwp + c, v);
+      Typed<T>::store8(static_cast<T*>(p.ring) + (long long)b * p.ring_bs + ((p.pos0 + t) % p.R) * (long long)p.cwp + c, v);
+    }
   }
 }
 
@@ -393,25 +499,42 @@ static int big_smem(K kernel, size_t bytes) {
 
 using namespace ats;
 
+static bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
+
+template <typename T>
+static int launch_context(const LatentArgs& p, cudaStream_t s) {
+  const int rows = p.B * (p.n_old + p.L);
+  const bool vec = ((p.q_rank | p.rank | p.q_col | p.kv_col | p.q_pad | p.cwp) & 7) == 0 && (p.rot & 15) == 0 && p.rot > 0 && (p.ld & 7) == 0 && (p.ring_bs & 7) == 0 &&
+                   p.q_pad == p.q_rank && p.cwp == p.rank + p.rot && aligned16(p.proj) && aligned16(p.ring);
+  if (vec) launch_pdl(latent_context_vec_kernel<T>, dim3((rows + 3) / 4), dim3(128), 0, s, p);
+  else launch_pdl(latent_context_kernel<T>, dim3(rows), dim3(128), 0, s, p);
+  return int(cudaGetLastError());
+}
+
+template <typename T>
+static int launch_finish(const FinishArgs& p, cudaStream_t s) {
+  const bool vec = (p.rot & 15) == 0 && p.rot > 0 && (p.dim & 7) == 0 && (p.ldq & 7) == 0 && (p.cwp & 7) == 0 && (p.ring_bs & 7) == 0 && aligned16(p.q) && aligned16(p.ring);
+  if (vec) {
+    const long long n = (long long)p.B * p.L * p.H * (p.rot >> 4) + (long long)p.B * (p.L < p.R ? p.L : p.R) * (p.cwp >> 3);
+    const long long blocks = (n + 255) / 256;
+    launch_pdl(latent_finish_vec_kernel<T>, dim3(unsigned(blocks < 148 * 64 ? blocks : 148 * 64)), dim3(256), 0, s, p);
+  } else {
+    launch_pdl(latent_finish_kernel<T>, dim3(p.B * p.L), dim3(128), 0, s, p);
+  }
+  return int(cudaGetLastError());
+}
+
 // Every entry point takes its argument struct by address (the ctypes mirror is in ops/latent.py); `fp32` selects the element type.
 ATS_API int ats_latent_context(const LatentArgs* p, int fp32, void* stream) {
   if (p->R < 1 || p->rot < 0 || (p->rot & 1) || (p->lengths && p->L != 1) || p->n_old < 0 || p->n_old > p->R) return 1006;
-  const int rows = p->B * (p->n_old + p->L);
-  if (rows <= 0) return 0;
-  cudaStream_t s = static_cast<cudaStream_t>(stream);
-  if (fp32) launch_pdl(latent_context_kernel<float>, dim3(rows), dim3(128), 0, s, *p);
-  else launch_pdl(latent_context_kernel<__nv_bfloat16>, dim3(rows), dim3(128), 0, s, *p);
-  return int(cudaGetLastError());
+  if (p->B <= 0 || p->n_old + p->L <= 0) return 0;
+  return fp32 ? launch_context<float>(*p, static_cast<cudaStream_t>(stream)) : launch_context<__nv_bfloat16>(*p, static_cast<cudaStream_t>(stream));
 }
 
 ATS_API int ats_latent_finish(const FinishArgs* p, int fp32, void* stream) {
   if (p->R < 1 || (p->rot & 1)) return 1006;
-  const int rows = p->B * p->L;
-  if (rows <= 0) return 0;
-  cudaStream_t s = static_cast<cudaStream_t>(stream);
-  if (fp32) launch_pdl(latent_finish_kernel<float>, dim3(rows), dim3(128), 0, s, *p);
-  else launch_pdl(latent_finish_kernel<__nv_bfloat16>, dim3(rows), dim3(128), 0, s, *p);
-  return int(cudaGetLastError());
+  if (p->B <= 0 || p->L <= 0) return 0;
+  return fp32 ? launch_finish<float>(*p, static_cast<cudaStream_t>(stream)) : launch_finish<__nv_bfloat16>(*p, static_cast<cudaStream_t>(stream));
 }
 
 ATS_API int ats_window_attn(const WindowArgs* p, int fp32, void* stream) {

@@ -1,0 +1,361 @@
+// Decoding with latent attention on tensor cores (bf16): one query token per sequence against its ring of latents.  The general
+// form for any sizes and for fp32, and the layout of the ring, are in latent_attention.cu.
+//
+//   latent_head_mm<absorb>   qa[b, h, :] = W_uk[h]^T q_u[b, h, :]               per head: [16 sequences x dim] x [dim x rank]
+//   latent_ring              scores of 16 heads against the ring rows (one shared row serves all heads, so the heads are the 16 rows of
+//                            the MMA), soft-max, weighted sum of the latents; chunks of the ring are merged by the next kernel
+//   latent_head_mm<expand>   out[b, h, :] = sigmoid(gate) * W_uv[h] (merged latent)   [16 sequences x rank] x [rank x vdim]
+//
+// A decode step is bound by the bytes of the ring, so warp-level MMAs are enough; a 64-row tile of the ring is fetched once with
+// cp.async and serves both products (plain and transposing ldmatrix; rows are padded by 16 bytes against bank conflicts).  Weights
+// stream straight from global memory into B fragments: the order of the reduction index is permuted so that the 16-byte piece a lane
+// loads is its fragment for two consecutive steps, and the A fragments are read with the same permutation.
+#include "common.cuh"
+
+namespace ats {
+
+__device__ __forceinline__ void mma_bf16_16816(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+               : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void ldmatrix_x4(uint32_t addr, uint32_t (&r)[4]) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void ldmatrix_x4_trans(uint32_t addr, uint32_t (&r)[4]) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+// 16 bytes global -> shared; zeros when `ok` is false
+__device__ __forceinline__ void cp_async_16(uint32_t dst, const void* src, bool ok) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(ok ? 16 : 0) : "memory");
+}
+__device__ __forceinline__ void cp_async_wait_all() {
+  asm volatile("cp.async.commit_group;" ::: "memory");
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
+}
+
+struct HeadMmArgs {
+  const __nv_bfloat16* x;   // absorb: q, head h at h * x_hs, rows x_ld apart
+  long long x_ld;
+  int x_hs;
+  const float* part_o;      // expand: [B, H, n_chunks, K] partial latents and [B, H, n_chunks, 2] (max, sum)
+  const float* part_ml;
+  int n_chunks;
+  const __nv_bfloat16* w;   // [H, N, ldw], reduction index contiguous
+  long long w_hs;
+  int ldw;
+  __nv_bfloat16* out;       // row b, head h, column n at b * out_ld + h * out_hs + n
+  long long out_ld;
+  int out_hs;
+  const __nv_bfloat16* gate;  // same columns as out, rows ldg apart (expand; may be null)
+  long long ldg;
+  int B, H, N, K;
+};
+constexpr int HM_MAX_CHUNKS = 64;
+
+// CTA: 16 sequences x (WARPS * NT * 8) output columns of one head.
+template <int WARPS, int NT, bool EXPAND>
+__global__ void __launch_bounds__(WARPS * 32) latent_head_mm_kernel(const HeadMmArgs p) {
+  pdl_prologue();
+  extern __shared__ __align__(16) uint8_t smem_raw[];
+  __nv_bfloat16* sx = reinterpret_cast<__nv_bfloat16*>(smem_raw);  // [16][K + 32]
+  __shared__ float s_f[EXPAND ? 16 : 1][EXPAND ? HM_MAX_CHUNKS : 1];
+  const int ldx = p.K + 32, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
+  const int h = blockIdx.y, b0 = blockIdx.z * 16, nb = min(16, p.B - b0);
+  const int n0 = (blockIdx.x * WARPS + warp) * NT * 8;
+  if (EXPAND) {
+    if (tid < 16 && tid < nb) {
+      const float* ml = p.part_ml + ((long long)(b0 + tid) * p.H + h) * p.n_chunks * 2;
+      float m = -INFINITY, l = 0.f;
+      for (int c = 0; c < p.n_chunks; ++c) m = fmaxf(m, ml[2 * c]);
+      for (int c = 0; c < p.n_chunks; ++c) {
+        const float f = ml[2 * c + 1] > 0.f ? __expf(ml[2 * c] - m) : 0.f;
+        s_f[tid][c] = f;
+        l += f * ml[2 * c + 1];
+      }
+      const float inv = 1.f / l;
+      for (int c = 0; c < p.n_chunks; ++c) s_f[tid][c] *= inv;
+    }
+    __syncthreads();
+    const int quads = p.K >> 2;
+    for (int i = tid; i < 16 * quads; i += WARPS * 32) {
+      const int j = i / quads, r = (i % quads) * 4;
+      float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (j < nb) {
+        const float* po = p.part_o + (((long long)(b0 + j) * p.H + h) * p.n_chunks) * p.K + r;
+        for (int c = 0; c < p.n_chunks; ++c) {
+          const float f = s_f[j][c];
+          if (f > 0.f) {  // chunks beyond a short sequence were not written
+            const float4 v = *reinterpret_cast<const float4*>(po + (long long)c * p.K);
+            a.x += f * v.x; a.y += f * v.y; a.z += f * v.z; a.w += f * v.w;
+          }
+        }
+      }
+      *reinterpret_cast<uint2*>(sx + j * ldx + r) = make_uint2(pack_bf16x2(a.x, a.y), pack_bf16x2(a.z, a.w));
+    }
+  } else {
+    const int pieces = p.K >> 3;
+    for (int i = tid; i < 16 * pieces; i += WARPS * 32) {
+      const int j = i / pieces, c = (i % pieces) * 8;
+      *reinterpret_cast<uint4*>(sx + j * ldx + c) =
+          j < nb ? *reinterpret_cast<const uint4*>(p.x + (b0 + j) * p.x_ld + (long long)h * p.x_hs + c) : make_uint4(0, 0, 0, 0);
+    }
+  }
+  __syncthreads();
+  if (n0 >= p.N) return;
+  float acc[NT][4];
+#pragma unroll
+  for (int i = 0; i < NT; ++i)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) acc[i][e] = 0.f;
+  const __nv_bfloat16* w = p.w + h * p.w_hs + 8 * t;
+#pragma unroll 4
+  for (int k = 0; k < p.K; k += 32) {
+    const uint4 lo = *reinterpret_cast<const uint4*>(sx + g * ldx + k + 8 * t), hi = *reinterpret_cast<const uint4*>(sx + (g + 8) * ldx + k + 8 * t);
+#pragma unroll
+    for (int i = 0; i < NT; ++i) {
+      const int n = n0 + i * 8 + g;
+      const uint4 b = n < p.N ? *reinterpret_cast<const uint4*>(w + (long long)n * p.ldw + k) : make_uint4(0, 0, 0, 0);
+      mma_bf16_16816(acc[i], lo.x, hi.x, lo.y, hi.y, b.x, b.y);
+      mma_bf16_16816(acc[i], lo.z, hi.z, lo.w, hi.w, b.z, b.w);
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < NT; ++i) {
+    const int n = n0 + i * 8 + 2 * t;
+    if (n >= p.N) continue;
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int j = g + 8 * e;
+      if (j >= nb) continue;
+      float v0 = acc[i][2 * e], v1 = acc[i][2 * e + 1];
+      const long long at = (long long)h * p.out_hs + n;
+      if (EXPAND && p.gate) {
+        const float2 gt = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(p.gate + (b0 + j) * p.ldg + at));
+        v0 = __fdividef(v0, 1.f + __expf(-gt.x));
+        v1 = __fdividef(v1, 1.f + __expf(-gt.y));
+      }
+      *reinterpret_cast<uint32_t*>(p.out + (b0 + j) * p.out_ld + at) = pack_bf16x2(v0, v1);
+    }
+  }
+}
+
+struct RingArgs {
+  const __nv_bfloat16* qa;    // [B, H, rank] absorbed queries
+  const __nv_bfloat16* q;     // [B, ldq]: rotated part of head h at h * dq + dim (not yet rotated)
+  long long ldq;
+  int dim, dq;
+  const float* cos;           // [positions, rot / 2]
+  const float* sin;
+  const __nv_bfloat16* ring;  // [B, R, cwp]
+  long long ring_bs;
+  const int* lengths;
+  int H, R, rank, rot, cwp, chunk, n_chunks;
+  float scale;
+  float* part_o;              // [B, H, n_chunks, rank]
+  float* part_ml;             // [B, H, n_chunks, 2]
+};
+constexpr int LR_KEYS = 64, LR_THREADS = 256;
+
+struct RingSmem {
+  int ldt, qa, s, pr, al, total;  // row pitch of tile and queries (elements), byte offsets
+  __host__ __device__ explicit RingSmem(int cw) {
+    ldt = cw + 8;
+    qa = LR_KEYS * ldt * 2;
+    s = qa + 16 * ldt * 2;
+    pr = s + 16 * (LR_KEYS + 4) * 4;
+    al = pr + 16 * (LR_KEYS + 8) * 2;
+    total = al + 16 * 4;
+  }
+};
+
+// NTW: 8-column tiles of the latent per warp (rank = 64 * NTW).
+template <int NTW>
+__global__ void __launch_bounds__(LR_THREADS, 2) latent_ring_kernel(const RingArgs p) {
+  pdl_prologue();
+  extern __shared__ __align__(16) uint8_t smem_raw[];
+  const int cw = p.rank + p.rot;
+  const RingSmem L(cw);
+  __nv_bfloat16* tile = reinterpret_cast<__nv_bfloat16*>(smem_raw);
+  __nv_bfloat16* sq = reinterpret_cast<__nv_bfloat16*>(smem_raw + L.qa);
+  float* ss = reinterpret_cast<float*>(smem_raw + L.s);                  // [16][LR_KEYS + 4]
+  __nv_bfloat16* sp = reinterpret_cast<__nv_bfloat16*>(smem_raw + L.pr);  // [16][LR_KEYS + 8]
+  float* sal = reinterpret_cast<float*>(smem_raw + L.al);                // [16]
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
+  const int chunk = blockIdx.x, h0 = blockIdx.y * 16, b = blockIdx.z, nh = min(16, p.H - h0);
+  const int pos = p.lengths[b], n = min(pos + 1, p.R), k0 = chunk * p.chunk, k1 = min(n, k0 + p.chunk);
+  float* ml = p.part_ml + (((long long)b * p.H + h0) * p.n_chunks + chunk) * 2;
+  if (k0 >= k1) {
+    if (tid < nh) {
+      ml[(long long)tid * p.n_chunks * 2] = -INFINITY;
+      ml[(long long)tid * p.n_chunks * 2 + 1] = 0.f;
+    }
+    return;
+  }
+  const __nv_bfloat16* ring = p.ring + (long long)b * p.ring_bs;
+  auto fetch = [&](int first) {
+    const int pieces = cw >> 3;
+    for (int i = tid; i < LR_KEYS * pieces; i += LR_THREADS) {
+      const int r = i / pieces, c = (i % pieces) * 8;
+      const bool ok = first + r < k1;
+      cp_async_16(smem_u32(tile + r * L.ldt + c), ring + (long long)(ok ? first + r : k0) * p.cwp + c, ok);
+    }
+  };
+  fetch(k0);
+  // absorbed queries (rows of heads that do not exist are zero), rotated parts
+  for (int i = tid; i < 16 * (p.rank >> 3); i += LR_THREADS) {
+    const int r = i / (p.rank >> 3), c = (i % (p.rank >> 3)) * 8;
+    *reinterpret_cast<uint4*>(sq + r * L.ldt + c) =
+        r < nh ? *reinterpret_cast<const uint4*>(p.qa + ((long long)b * p.H + h0 + r) * p.rank + c) : make_uint4(0, 0, 0, 0);
+  }
+  const int half = p.rot >> 1;
+  for (int i = tid; i < 16 * half; i += LR_THREADS) {
+    const int r = i / half, m = i % half;
+    float u = 0.f, v = 0.f;
+    if (r < nh) {
+      const __nv_bfloat16* qr = p.q + b * p.ldq + (long long)(h0 + r) * p.dq + p.dim + m;
+      const float x = __bfloat162float(qr[0]), y = __bfloat162float(qr[half]);
+      const float cs = p.cos[(long long)pos * half + m], sn = p.sin[(long long)pos * half + m];
+      u = x * cs - y * sn;
+      v = y * cs + x * sn;
+    }
+    sq[r * L.ldt + p.rank + m] = __float2bfloat16(u);
+    sq[r * L.ldt + p.rank + half + m] = __float2bfloat16(v);
+  }
+  float acc[NTW][4];
+#pragma unroll
+  for (int i = 0; i < NTW; ++i)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) acc[i][e] = 0.f;
+  float m_[2] = {-INFINITY, -INFINITY}, l_[2] = {0.f, 0.f};  // soft-max state of heads 2 * warp, + 1
+  const uint32_t a_addr = smem_u32(sq + (lane & 15) * L.ldt + (lane >> 4) * 8);
+  const uint32_t b_addr = smem_u32(tile + (warp * 8 + (lane & 7)) * L.ldt + (lane >> 3) * 8);
+  const uint32_t p_addr = smem_u32(sp + (lane & 15) * (LR_KEYS + 8) + (lane >> 4) * 8);
+  const uint32_t v_addr = smem_u32(tile + (lane & 15) * L.ldt + warp * NTW * 8 + (lane >> 4) * 8);
+  for (int first = k0; first < k1; first += LR_KEYS) {
+    cp_async_wait_all();
+    __syncthreads();
+    // ---- scores: warp w, keys 8 w .. 8 w + 7 of the tile
+    {
+      float c0[4] = {0.f, 0.f, 0.f, 0.f}, c1[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll 2
+      for (int k = 0; k < cw; k += 32) {
+        uint32_t bb[4], a0[4], a1[4];
+        ldmatrix_x4(b_addr + k * 2, bb);
+        ldmatrix_x4(a_addr + k * 2, a0);
+        ldmatrix_x4(a_addr + k * 2 + 32, a1);
+        mma_bf16_16816(c0, a0[0], a0[1], a0[2], a0[3], bb[0], bb[1]);
+        mma_bf16_16816(c1, a1[0], a1[1], a1[2], a1[3], bb[2], bb[3]);
+      }
+      const int key = warp * 8 + 2 * t;
+      const bool ok0 = first + key < k1, ok1 = first + key + 1 < k1;
+      float* s0 = ss + g * (LR_KEYS + 4) + key;
+      float* s1 = ss + (g + 8) * (LR_KEYS + 4) + key;
+      s0[0] = ok0 ? (c0[0] + c1[0]) * p.scale : -INFINITY;
+      s0[1] = ok1 ? (c0[1] + c1[1]) * p.scale : -INFINITY;
+      s1[0] = ok0 ? (c0[2] + c1[2]) * p.scale : -INFINITY;
+      s1[1] = ok1 ? (c0[3] + c1[3]) * p.scale : -INFINITY;
+    }
+    __syncthreads();
+    // ---- soft-max: two heads per warp
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int r = warp * 2 + e;
+      const float x0 = ss[r * (LR_KEYS + 4) + lane], x1 = ss[r * (LR_KEYS + 4) + lane + 32];
+      const float mn = fmaxf(m_[e], warp_max(fmaxf(x0, x1)));  // the tile has at least one key: finite
+      const float al = __expf(m_[e] - mn), p0 = __expf(x0 - mn), p1 = __expf(x1 - mn);
+      m_[e] = mn;
+      l_[e] = l_[e] * al + warp_sum(p0 + p1);
+      sp[r * (LR_KEYS + 8) + lane] = __float2bfloat16(p0);
+      sp[r * (LR_KEYS + 8) + lane + 32] = __float2bfloat16(p1);
+      if (lane == 0) sal[r] = al;
+    }
+    __syncthreads();
+    // ---- weighted sum of the latents: warp w, columns w * NTW * 8 ..
+    const float al0 = sal[g], al1 = sal[g + 8];
+#pragma unroll
+    for (int i = 0; i < NTW; ++i) {
+      acc[i][0] *= al0; acc[i][1] *= al0;
+      acc[i][2] *= al1; acc[i][3] *= al1;
+    }
+#pragma unroll
+    for (int k = 0; k < LR_KEYS; k += 16) {
+      uint32_t a[4];
+      ldmatrix_x4(p_addr + k * 2, a);
+#pragma unroll
+      for (int i = 0; i < NTW; i += 2) {
+        uint32_t v[4];
+        ldmatrix_x4_trans(v_addr + (k * L.ldt + i * 8) * 2, v);
+        mma_bf16_16816(acc[i], a[0], a[1], a[2], a[3], v[0], v[1]);
+        mma_bf16_16816(acc[i + 1], a[0], a[1], a[2], a[3], v[2], v[3]);
+      }
+    }
+    __syncthreads();
+    if (first + LR_KEYS < k1) fetch(first + LR_KEYS);
+  }
+#pragma unroll
+  for (int i = 0; i < NTW; ++i) {
+    const int c = (warp * NTW + i) * 8 + 2 * t;
+    float* o = p.part_o + (((long long)b * p.H + h0 + g) * p.n_chunks + chunk) * p.rank + c;
+    if (g < nh) *reinterpret_cast<float2*>(o) = make_float2(acc[i][0], acc[i][1]);
+    if (g + 8 < nh) *reinterpret_cast<float2*>(o + 8ll * p.n_chunks * p.rank) = make_float2(acc[i][2], acc[i][3]);
+  }
+  if (lane == 0)
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int r = warp * 2 + e;
+      if (r < nh) {
+        ml[(long long)r * p.n_chunks * 2] = m_[e];
+        ml[(long long)r * p.n_chunks * 2 + 1] = l_[e];
+      }
+    }
+}
+
+template <int NTW>
+static cudaError_t launch_ring(const RingArgs& p, int B, cudaStream_t s) {
+  const RingSmem L(p.rank + p.rot);
+  cudaError_t e = cudaFuncSetAttribute(latent_ring_kernel<NTW>, cudaFuncAttributeMaxDynamicSharedMemorySize, L.total);
+  if (e != cudaSuccess) return e;
+  return launch_pdl(latent_ring_kernel<NTW>, dim3(p.n_chunks, (p.H + 15) / 16, B), dim3(LR_THREADS), size_t(L.total), s, p);
+}
+
+}  // namespace ats
+
+using namespace ats;
+
+// One decoded token per sequence (see the head of the file).  q [B, ldq] head h at h * (dim + rot), not rotated; w_ukt [H, rank, dim],
+// w_uv [H, vdim, ldv], ring [B, R, cwp].  qa [B, H, rank], part_o, part_ml: scratch.  Returns 1003 for shapes this form does not cover.
+ATS_API int ats_latent_decode_mma(const void* q, long long ldq, const void* w_ukt, const void* w_uv, int ldv, const void* ring, long long ring_bs,
+                                  const int* lengths, const float* cos, const float* sin, const void* gate, long long ldg, void* qa, float* part_o,
+                                  float* part_ml, void* out, long long ldo, int B, int H, int dim, int rot, int rank, int vdim, int cwp, int R, int chunk,
+                                  int n_chunks, float scale, void* stream) {
+  if (B < 1) return 0;
+  const bool rank_ok = rank == 128 || rank == 256 || rank == 384 || rank == 512;
+  if (!rank_ok || (dim & 31) || dim > 512 || (rot & 31) || rot < 32 || rot > 128 || (vdim & 7) || (ldq & 7) || (ldv & 7) || (cwp & 7) || (ring_bs & 7) || (ldo & 1) ||
+      (gate && (ldg & 1)) || chunk < LR_KEYS || (chunk % LR_KEYS) || n_chunks < 1 || n_chunks > HM_MAX_CHUNKS || (long long)chunk * n_chunks < R)
+    return 1003;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  HeadMmArgs a = {};
+  a.x = static_cast<const __nv_bfloat16*>(q); a.x_ld = ldq; a.x_hs = dim + rot;
+  a.w = static_cast<const __nv_bfloat16*>(w_ukt); a.w_hs = (long long)rank * dim; a.ldw = dim;
+  a.out = static_cast<__nv_bfloat16*>(qa); a.out_ld = (long long)H * rank; a.out_hs = rank;
+  a.B = B; a.H = H; a.N = rank; a.K = dim;
+  const int bt = (B + 15) / 16;
+  cudaError_t e = launch_pdl(latent_head_mm_kernel<4, 4, false>, dim3(rank / 128, H, bt), dim3(128), size_t(16) * (dim + 32) * 2, s, a);
+  if (e != cudaSuccess) return int(e);
+  RingArgs r;
+  r.qa = static_cast<const __nv_bfloat16*>(qa); r.q = static_cast<const __nv_bfloat16*>(q); r.ldq = ldq; r.dim = dim; r.dq = dim + rot;
+  r.cos = cos; r.sin = sin; r.ring = static_cast<const __nv_bfloat16*>(ring); r.ring_bs = ring_bs; r.lengths = lengths;
+  r.H = H; r.R = R; r.rank = rank; r.rot = rot; r.cwp = cwp; r.chunk = chunk; r.n_chunks = n_chunks; r.scale = scale;
+  r.part_o = part_o; r.part_ml = part_ml;
+  e = rank == 128 ? launch_ring<2>(r, B, s) : rank == 256 ? launch_ring<4>(r, B, s) : rank == 384 ? launch_ring<6>(r, B, s) : launch_ring<8>(r, B, s);
+  if (e != cudaSuccess) return int(e);
+  HeadMmArgs x = {};
+  x.part_o = part_o; x.part_ml = part_ml; x.n_chunks = n_chunks;
+  x.w = static_cast<const __nv_bfloat16*>(w_uv); x.w_hs = (long long)vdim * ldv; x.ldw = ldv;
+  x.out = static_cast<__nv_bfloat16*>(out); x.out_ld = ldo; x.out_hs = vdim;
+  x.gate = static_cast<const __nv_bfloat16*>(gate); x.ldg = ldg;
+  x.B = B; x.H = H; x.N = vdim; x.K = rank;
+  e = launch_pdl(latent_head_mm_kernel<8, 2, true>, dim3((vdim + 127) / 128, H, bt), dim3(256), size_t(16) * (rank + 32) * 2, s, x);
+  return int(e != cudaSuccess ? e : cudaGetLastError());
+}
