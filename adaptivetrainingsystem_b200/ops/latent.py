@@ -259,8 +259,9 @@ def latent_decode(q: torch.Tensor, ring: torch.Tensor, w_uk: torch.Tensor, w_uv_
         return out
     dev = q.device
     if w_ukt is not None and w_uv is not None and R <= 64 * 4096:
-        # enough chunks to give every SM two, none smaller than a 64-row tile, at most 64 per sequence
-        chunk = max(64, (R * B * ((H + 15) // 16) // 296 + 63) // 64 * 64, (R + 64 * 64 - 1) // (64 * 64) * 64)
+        # two CTAs per SM share the ring's chunks: as many chunks per sequence as fit one wave, of whole 64-row tiles, at most 64
+        n_chunks = max(1, min(64, (R + 63) // 64, 296 // (B * ((H + 15) // 16))))
+        chunk = ((R + n_chunks - 1) // n_chunks + 63) // 64 * 64
         n_chunks = (R + chunk - 1) // chunk
         qa = torch.empty(B, H, s.rank, dtype=q.dtype, device=dev)
         part_o = torch.empty(B, H, n_chunks, s.rank, dtype=torch.float32, device=dev)

@@ -11,7 +11,7 @@
 //   group, u_i = beta_i (v_i - G_i S^T k_i - sum_{j < i} D_ij (k_j . k_i) u_j), D_ij = g_{j+1} .. g_i, G_i = g_1 .. g_i, a unit lower
 //   triangular system whose 8 x 8 inverse does not depend on the value column; delta_pairs computes it (and the read-out
 //   coefficients) for all groups in parallel, so that the sequential kernel only does three products with the state per token.
-//   Columns of S are independent: eight lanes share a column (or two), everything in fp32 with packed fma.f32x2.
+//   Columns of S are independent: sixteen lanes share eight columns, everything in fp32 with packed fma.f32x2.
 // * delta_output: output norm over vdim, weight, silu gate.
 // * delta_step: one decoded token per sequence: state read once and written once, output norm and gate in the same launch.
 //
@@ -98,12 +98,12 @@ __global__ void __launch_bounds__(256) delta_prep_kernel(const DeltaArgs p) {
 
 // The same for portions whose heads are whole 16-byte pieces: a thread owns eight channels and walks PT consecutive tokens with the
 // convolution's inputs in registers; the lanes of a head (dim / 8 of them, a power of two) add up its length with shuffles.
-constexpr int PT = 16;
+constexpr int PT = 16, PV_THREADS = 128;
 template <typename T, int TAPS>
-__global__ void __launch_bounds__(256) delta_prep_vec_kernel(const DeltaArgs p) {
+__global__ void __launch_bounds__(PV_THREADS, 4) delta_prep_vec_kernel(const DeltaArgs p) {
   pdl_prologue();
-  const int pieces = p.C >> 3, per_block = (pieces + 255) / 256, blocks_t = (p.L + PT - 1) / PT;
-  const int piece = (blockIdx.x % per_block) * 256 + threadIdx.x;
+  const int pieces = p.C >> 3, per_block = (pieces + PV_THREADS - 1) / PV_THREADS, blocks_t = (p.L + PT - 1) / PT;
+  const int piece = (blockIdx.x % per_block) * PV_THREADS + threadIdx.x;
   const int tb = (blockIdx.x / per_block) % blocks_t, b = blockIdx.x / per_block / blocks_t;
   const int t0 = tb * PT, t1 = min(p.L, t0 + PT);
   const bool live = piece < pieces;  // C / 8 need not fill the last block: idle lanes still take part in the shuffles
@@ -126,33 +126,47 @@ __global__ void __launch_bounds__(256) delta_prep_vec_kernel(const DeltaArgs p) 
       for (int e = 0; e < 8; ++e) x[j - 1][e] = 0.f;
   }
   const int lanes = p.dim >> 3, kd = p.KH * p.dim;
-  const bool qk = live && c < 2 * kd;
-  float nx[8];
-  Typed<T>::load8(in + (long long)t0 * p.ld, nx);
-  for (int t = t0; t < t1; ++t) {
+  const bool qk = live && c < 2 * kd, warp_qk = __any_sync(0xffffffffu, qk);
+  // tokens come in batches of PB whose loads are issued one batch ahead
+  constexpr int PB = 4;
+  typename Typed<T>::Raw8 nx[PB];
 #pragma unroll
-    for (int j = TAPS - 1; j > 0; --j)
+  for (int u = 0; u < PB; ++u) nx[u] = Typed<T>::raw8(in + (long long)min(t0 + u, t1 - 1) * p.ld);
+  for (int tb0 = t0; tb0 < t1; tb0 += PB) {
+    typename Typed<T>::Raw8 cur[PB];
 #pragma unroll
-      for (int e = 0; e < 8; ++e) x[j][e] = x[j - 1][e];
+    for (int u = 0; u < PB; ++u) cur[u] = nx[u];
+    if (tb0 + PB < t1)
 #pragma unroll
-    for (int e = 0; e < 8; ++e) x[0][e] = nx[e];
-    if (t + 1 < t1) Typed<T>::load8(in + (long long)(t + 1) * p.ld, nx);
-    float y[8], ss = 0.f;
+      for (int u = 0; u < PB; ++u) nx[u] = Typed<T>::raw8(in + (long long)min(tb0 + PB + u, t1 - 1) * p.ld);
 #pragma unroll
-    for (int e = 0; e < 8; ++e) {
-      float acc = 0.f;
+    for (int u = 0; u < PB; ++u) {
+      const int t = tb0 + u;
+      if (t >= t1) break;
 #pragma unroll
-      for (int j = 0; j < TAPS; ++j) acc += x[j][e] * w[j][e];
-      y[e] = acc * Typed<T>::sigmoid_(acc);
-    }
-    Typed<T>::round8(y);
+      for (int j = TAPS - 1; j > 0; --j)
 #pragma unroll
-    for (int e = 0; e < 8; ++e) ss += y[e] * y[e];
-    if (live) Typed<T>::store8(out + (long long)t * p.ldm, y);
-    for (int off = lanes >> 1; off > 0; off >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, off);
-    if (qk && (piece & (lanes - 1)) == 0) {
-      const int head = piece / lanes;
-      p.rlen[((long long)b * p.L + t) * 2 * p.KH + head] = (head < p.KH ? 1.f / sqrtf(float(p.dim)) : 1.f) / sqrtf(ss + 1e-6f);
+        for (int e = 0; e < 8; ++e) x[j][e] = x[j - 1][e];
+      Typed<T>::unpack8(cur[u], x[0]);
+      float y[8], ss = 0.f;
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        float acc = 0.f;
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) acc += x[j][e] * w[j][e];
+        y[e] = acc * Typed<T>::sigmoid_(acc);
+      }
+      Typed<T>::round8(y);
+      if (live) Typed<T>::store8(out + (long long)t * p.ldm, y);
+      if (warp_qk) {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) ss += y[e] * y[e];
+        for (int off = lanes >> 1; off > 0; off >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, off);
+        if (qk && (piece & (lanes - 1)) == 0) {
+          const int head = piece / lanes;
+          p.rlen[((long long)b * p.L + t) * 2 * p.KH + head] = (head < p.KH ? 1.f / sqrtf(float(p.dim)) : 1.f) / sqrtf(ss + 1e-6f);
+        }
+      }
     }
   }
 }
@@ -307,52 +321,48 @@ __device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) { return __
 // Keeps the compiler from requesting the shared-memory rows of more tokens than registers can hold.
 __device__ __forceinline__ void pace() { asm volatile("" ::: "memory"); }
 
-// Eight per-lane values of which the sum over the eight lanes of a group is wanted: lane l ends up with the sum of value l.
-__device__ __forceinline__ float transpose_sum8(float (&v)[DC], int l) {
-#pragma unroll
-  for (int s = 4; s > 0; s >>= 1) {
-    const bool up = (l & s) != 0;
-#pragma unroll
-    for (int i = 0; i < s; ++i) {
-      const float send = up ? v[i] : v[i + s], have = up ? v[i + s] : v[i];
-      v[i] = have + __shfl_xor_sync(0xffffffffu, send, s);
-    }
-  }
-  return v[0];
+// One step of a transposing reduction over lanes: of the pair (lo, hi) this lane keeps hi when its bit `s` is set, else lo, and adds
+// what the lane across sends.
+__device__ __forceinline__ float keep_add(float lo, float hi, int lane, int s) {
+  const bool up = (lane & s) != 0;
+  return (up ? hi : lo) + __shfl_xor_sync(0xffffffffu, up ? lo : hi, s);
 }
 
-// EPL: state rows per lane (dim <= 8 * EPL), CPL: value columns per lane group.  CTA = 4 warps of 4 lane groups -> 16 * CPL columns
-// of one head.  The next group's q, k, v and constants are requested before this group's products and stored to the other half of
-// shared memory after them.
-template <typename T, int EPL, int CPL, int OCC>
-__global__ void __launch_bounds__(128, OCC) delta_scan_kernel(const ScanArgs p) {
+// Sixteen lanes share CPL value columns: lane l holds EPL state rows (dim <= 16 * EPL) of each.  CTA = 4 warps of 2 lane groups ->
+// 8 * CPL columns of one head.  With the state spread over sixteen lanes, a row of k or q read from shared memory serves CPL columns,
+// which keeps the load pipe below the FMA pipe.  The next group's q, k, v and constants are requested before this group's products
+// and stored to the other half of shared memory after them.  After a product, lane l holds token l % 8, columns (l / 8) * CPL / 2 ...
+template <typename T, int EPL, int CPL>
+__global__ void __launch_bounds__(128, 2) delta_scan_kernel(const ScanArgs p) {
   pdl_prologue();
-  constexpr int DK = 8 * EPL;
+  constexpr int DK = 16 * EPL, HC = CPL / 2;
   constexpr int VEC = 16 / int(sizeof(T));             // elements per 16-byte piece
   constexpr int NP = (2 * DC * DK / VEC + 127) / 128;  // pieces of q and k per thread and group
   __shared__ __align__(16) float s_kq[2][2][DC][DK];   // [buffer][k, q]
   __shared__ __align__(16) float s_c[2][CO];
-  const int tid = threadIdx.x, lane = tid & 31, l8 = lane & 7;
+  __shared__ __align__(16) float s_u[8][3][DC][CPL];   // [lane group][right-hand side, u, D_Cj u_j / |k_j|]
+  const int tid = threadIdx.x, lane = tid & 31, l16 = lane & 15, grp16 = tid >> 4, tok = l16 & 7, half = l16 >> 3;
   const int h = blockIdx.y, b = blockIdx.z, kh = h / (p.H / p.KH);
-  const int col0 = (blockIdx.x * 16 + (tid >> 3)) * CPL;
+  const int col0 = (blockIdx.x * 8 + grp16) * CPL, colh = col0 + half * HC;
   float2 S[CPL][EPL / 2];
   float* st = p.state + (long long)b * p.state_bs + (long long)h * p.dim * p.vdim;
 #pragma unroll
   for (int c = 0; c < CPL; ++c)
 #pragma unroll
     for (int e = 0; e < EPL / 2; ++e) {
-      const int d = ((e >> 1) * 8 + l8) * 4 + (e & 1) * 2;
+      const int d = ((e >> 1) * 16 + l16) * 4 + (e & 1) * 2;
       const bool ok = !p.fresh && col0 + c < p.vdim;
       S[c][e].x = (ok && d < p.dim) ? st[(long long)d * p.vdim + col0 + c] : 0.f;
       S[c][e].y = (ok && d + 1 < p.dim) ? st[(long long)(d + 1) * p.vdim + col0 + c] : 0.f;
     }
   const T* base = static_cast<const T*>(p.mixed) + (long long)b * p.L * p.ldm;
-  const T* vbase = base + 2 * p.KH * p.dim + (long long)h * p.vdim + col0;
+  const T* vbase = base + 2 * p.KH * p.dim + (long long)h * p.vdim + colh;
+  T* obase = static_cast<T*>(p.o) + (long long)b * p.L * p.ldo + (long long)h * p.vdim + colh;
   const float* cbase = p.coef + ((long long)b * p.groups * p.H + h) * CO;
   const bool vec = (p.dim % VEC) == 0;  // rows are whole 16-byte pieces (p.ldm is a multiple of 8)
   uint4 piece[NP];
   float4 cpiece;
-  float vnext[CPL];
+  float vnext[HC];
   auto request = [&](int grp) {
     const int t0 = grp * DC, n = min(DC, p.L - t0);
 #pragma unroll
@@ -370,7 +380,7 @@ __global__ void __launch_bounds__(128, OCC) delta_scan_kernel(const ScanArgs p) 
     }
     if (tid < CO / 4) cpiece = *reinterpret_cast<const float4*>(cbase + (long long)grp * p.H * CO + tid * 4);
 #pragma unroll
-    for (int c = 0; c < CPL; ++c) vnext[c] = (l8 < n && col0 + c < p.vdim) ? Typed<T>::load(vbase + (long long)(t0 + l8) * p.ldm + c) : 0.f;
+    for (int c = 0; c < HC; ++c) vnext[c] = (tok < n && colh + c < p.vdim) ? Typed<T>::load(vbase + (long long)(t0 + tok) * p.ldm + c) : 0.f;
   };
   auto deposit = [&](int buf) {
 #pragma unroll
@@ -386,82 +396,115 @@ __global__ void __launch_bounds__(128, OCC) delta_scan_kernel(const ScanArgs p) 
     }
     if (tid < CO / 4) *reinterpret_cast<float4*>(&s_c[buf][tid * 4]) = cpiece;
   };
-  // sum over the state rows of S times the eight k (which = 0) or q (1) vectors of the group; lane l8 keeps token l8
-  auto products = [&](int buf, int which, float (&out)[CPL]) {
-    float acc[CPL][DC];
+  // sums over the state rows of S times the eight k (which = 0) or q (1) vectors of the group
+  auto products = [&](int buf, int which, float (&out)[HC]) {
+    float r2[2][CPL];
 #pragma unroll
-    for (int i = 0; i < DC; ++i) {
-      float2 a[CPL];
+    for (int y = 0; y < 2; ++y) {      // tokens y, y + 4, y + 2, y + 6
+      float r4[2][CPL];
 #pragma unroll
-      for (int c = 0; c < CPL; ++c) a[c] = make_float2(0.f, 0.f);
+      for (int z = 0; z < 2; ++z) {
+        float r8[2][CPL];
 #pragma unroll
-      for (int e = 0; e < EPL / 4; ++e) {
-        const float4 k4 = *reinterpret_cast<const float4*>(&s_kq[buf][which][i][(e * 8 + l8) * 4]);
+        for (int x = 0; x < 2; ++x) {
+          const int i = y + 2 * z + 4 * x;
+          float2 a[CPL];
 #pragma unroll
-        for (int c = 0; c < CPL; ++c) {
-          a[c] = fma2(S[c][2 * e], make_float2(k4.x, k4.y), a[c]);
-          a[c] = fma2(S[c][2 * e + 1], make_float2(k4.z, k4.w), a[c]);
+          for (int c = 0; c < CPL; ++c) a[c] = make_float2(0.f, 0.f);
+#pragma unroll
+          for (int e = 0; e < EPL / 4; ++e) {
+            const float4 k4 = *reinterpret_cast<const float4*>(&s_kq[buf][which][i][(e * 16 + l16) * 4]);
+#pragma unroll
+            for (int c = 0; c < CPL; ++c) {
+              a[c] = fma2(S[c][2 * e], make_float2(k4.x, k4.y), a[c]);
+              a[c] = fma2(S[c][2 * e + 1], make_float2(k4.z, k4.w), a[c]);
+            }
+          }
+#pragma unroll
+          for (int c = 0; c < CPL; ++c) r8[x][c] = a[c].x + a[c].y;
         }
+#pragma unroll
+        for (int c = 0; c < CPL; ++c) r4[z][c] = keep_add(r8[0][c], r8[1][c], lane, 4);
+        pace();
       }
 #pragma unroll
-      for (int c = 0; c < CPL; ++c) acc[c][i] = a[c].x + a[c].y;
-      if (i & 1) pace();
+      for (int c = 0; c < CPL; ++c) r2[y][c] = keep_add(r4[0][c], r4[1][c], lane, 2);
     }
 #pragma unroll
-    for (int c = 0; c < CPL; ++c) out[c] = transpose_sum8(acc[c], l8);
+    for (int c = 0; c < CPL; ++c) r2[0][c] = keep_add(r2[0][c], r2[1][c], lane, 1);
+#pragma unroll
+    for (int c = 0; c < HC; ++c) out[c] = keep_add(r2[0][c], r2[0][c + HC], lane, 8);
   };
   request(0);
   deposit(0);
   __syncthreads();
   for (int grp = 0; grp < p.groups; ++grp) {
     const int buf = grp & 1, t0 = grp * DC, n = min(DC, p.L - t0);
-    float v[CPL];
-#pragma unroll
-    for (int c = 0; c < CPL; ++c) v[c] = vnext[c];
-    if (grp + 1 < p.groups) request(grp + 1);
     const float* co = s_c[buf];
-    float sk[CPL], w[CPL][DC];
-    products(buf, 0, sk);
-    const float gk = co[2 * DC * DC + l8], gq = co[2 * DC * DC + DC + l8], GC = co[2 * DC * DC + 3 * DC];
-    __align__(16) float row[2 * DC];
+    float sk[HC], o[HC];
+    {
+      float v[HC];
 #pragma unroll
-    for (int j = 0; j < 2 * DC; j += 4) *reinterpret_cast<float4*>(&row[j]) = *reinterpret_cast<const float4*>(&co[l8 * 2 * DC + j]);
-    float o[CPL];
+      for (int c = 0; c < HC; ++c) v[c] = vnext[c];
+      if (grp + 1 < p.groups) request(grp + 1);
+      products(buf, 0, sk);
+      const float gk = co[2 * DC * DC + tok];
 #pragma unroll
-    for (int c = 0; c < CPL; ++c) {
-      const float rhs = v[c] - gk * sk[c];
-      float u = 0.f;
+      for (int c = 0; c < HC; ++c) s_u[grp16][0][tok][half * HC + c] = v[c] - gk * sk[c];
+    }
+    __syncwarp();
+    {
+      const float dk = co[2 * DC * DC + 2 * DC + tok];
+      float u[HC];
 #pragma unroll
-      for (int j = 0; j < DC; ++j) u += row[j] * __shfl_sync(0xffffffffu, rhs, j, 8);
-      o[c] = 0.f;
+      for (int c = 0; c < HC; ++c) u[c] = 0.f;
 #pragma unroll
       for (int j = 0; j < DC; ++j) {
-        w[c][j] = __shfl_sync(0xffffffffu, u, j, 8);
-        o[c] += row[DC + j] * w[c][j];
+        const float m = co[tok * 2 * DC + j];
+#pragma unroll
+        for (int c = 0; c < HC; ++c) u[c] += m * s_u[grp16][0][j][half * HC + c];
+      }
+#pragma unroll
+      for (int c = 0; c < HC; ++c) {
+        s_u[grp16][1][tok][half * HC + c] = u[c];
+        s_u[grp16][2][tok][half * HC + c] = u[c] * dk;
       }
     }
-    products(buf, 1, sk);
+    __syncwarp();
 #pragma unroll
-    for (int c = 0; c < CPL; ++c)
-      if (l8 < n && col0 + c < p.vdim)
-        Typed<T>::store(static_cast<T*>(p.o) + ((long long)b * p.L + t0 + l8) * p.ldo + (long long)h * p.vdim + col0 + c, o[c] + gq * sk[c]);
+    for (int c = 0; c < HC; ++c) o[c] = 0.f;
+#pragma unroll
+    for (int j = 0; j < DC; ++j) {
+      const float m = co[tok * 2 * DC + DC + j];
+#pragma unroll
+      for (int c = 0; c < HC; ++c) o[c] += m * s_u[grp16][1][j][half * HC + c];
+    }
+    products(buf, 1, sk);
+    const float gq = co[2 * DC * DC + DC + tok], GC = co[2 * DC * DC + 3 * DC];
+    if (tok < n)
+#pragma unroll
+      for (int c = 0; c < HC; ++c)
+        if (colh + c < p.vdim) Typed<T>::store(obase + (long long)(t0 + tok) * p.ldo + c, o[c] + gq * sk[c]);
 #pragma unroll
     for (int c = 0; c < CPL; ++c)
 #pragma unroll
       for (int e = 0; e < EPL / 2; ++e) S[c][e] = make_float2(S[c][e].x * GC, S[c][e].y * GC);
 #pragma unroll
     for (int j = 0; j < DC; ++j) {
-      const float dk = co[2 * DC * DC + 2 * DC + j];
-      float2 uu[CPL];
+      float w[CPL];
 #pragma unroll
-      for (int c = 0; c < CPL; ++c) uu[c] = make_float2(w[c][j] * dk, w[c][j] * dk);
+      for (int c = 0; c < CPL; c += 4) {
+        const float4 q = *reinterpret_cast<const float4*>(&s_u[grp16][2][j][c]);
+        w[c] = q.x; w[c + 1] = q.y; w[c + 2] = q.z; w[c + 3] = q.w;
+      }
 #pragma unroll
       for (int e = 0; e < EPL / 4; ++e) {
-        const float4 k4 = *reinterpret_cast<const float4*>(&s_kq[buf][0][j][(e * 8 + l8) * 4]);
+        const float4 k4 = *reinterpret_cast<const float4*>(&s_kq[buf][0][j][(e * 16 + l16) * 4]);
 #pragma unroll
         for (int c = 0; c < CPL; ++c) {
-          S[c][2 * e] = fma2(make_float2(k4.x, k4.y), uu[c], S[c][2 * e]);
-          S[c][2 * e + 1] = fma2(make_float2(k4.z, k4.w), uu[c], S[c][2 * e + 1]);
+          const float2 uu = make_float2(w[c], w[c]);
+          S[c][2 * e] = fma2(make_float2(k4.x, k4.y), uu, S[c][2 * e]);
+          S[c][2 * e + 1] = fma2(make_float2(k4.z, k4.w), uu, S[c][2 * e + 1]);
         }
       }
       if (j & 1) pace();
@@ -474,7 +517,7 @@ __global__ void __launch_bounds__(128, OCC) delta_scan_kernel(const ScanArgs p) 
     if (col0 + c >= p.vdim) continue;
 #pragma unroll
     for (int e = 0; e < EPL / 2; ++e) {
-      const int d = ((e >> 1) * 8 + l8) * 4 + (e & 1) * 2;
+      const int d = ((e >> 1) * 16 + l16) * 4 + (e & 1) * 2;
       if (d < p.dim) st[(long long)d * p.vdim + col0 + c] = S[c][e].x;
       if (d + 1 < p.dim) st[(long long)(d + 1) * p.vdim + col0 + c] = S[c][e].y;
     }
@@ -635,21 +678,125 @@ __global__ void __launch_bounds__(ST_THREADS) delta_step_kernel(const StepArgs p
     for (int v = p.H * p.vdim + tid; v < p.ldout; v += ST_THREADS) Typed<T>::store(out + v, 0.f);
 }
 
+// The same with four columns per access (vdim a multiple of 4, up to 128 per pass): 32 column quads x 8 row groups, RPT rows per thread.
+constexpr int SV_THREADS = 256;
+template <typename T, int RPT>
+__global__ void __launch_bounds__(SV_THREADS, RPT <= 8 ? 4 : RPT <= 16 ? 2 : 1) delta_step_vec_kernel(const StepArgs p) {
+  pdl_prologue();
+  extern __shared__ __align__(16) float smv[];
+  const int tid = threadIdx.x, c = tid & 31, rg = tid >> 5, h = blockIdx.x, b = blockIdx.y;
+  float4* s_r = reinterpret_cast<float4*>(smv);                   // [8][32]
+  float* s_k = smv + 8 * 32 * 4;                                  // [dim]
+  float* s_q = s_k + p.dim;                                       // [dim]
+  float* s_o = s_q + p.dim;                                       // [vdim]
+  float* s_red = s_o + p.vdim;                                    // [40]
+  const int kh = h / (p.H / p.KH);
+  const bool fresh = p.lengths[b] == 0, keep = !(p.active && !p.active[b]);
+  const T* mixed = static_cast<const T*>(p.mixed) + (long long)b * p.ldm;
+  float* st = p.state + (long long)b * p.state_bs + (long long)h * p.dim * p.vdim;
+  const float rq = p.rlen[(long long)b * 2 * p.KH + kh], rk = p.rlen[(long long)b * 2 * p.KH + p.KH + kh];
+  const float g = p.gb[(long long)b * 2 * p.H + h], beta = p.gb[(long long)b * 2 * p.H + p.H + h];
+  float ss = 0.f;
+  for (int v0 = 0; v0 < p.vdim; v0 += 128) {
+    const int v = v0 + c * 4;
+    const bool ok = v < p.vdim;
+    float4 S[RPT];
+#pragma unroll
+    for (int i = 0; i < RPT; ++i) {
+      const int d = rg + i * 8;
+      S[i] = (ok && d < p.dim && !fresh) ? __ldcs(reinterpret_cast<const float4*>(st + (long long)d * p.vdim + v)) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    if (v0 == 0) {
+      for (int d = tid; d < p.dim; d += SV_THREADS) {
+        s_k[d] = Typed<T>::load(mixed + (long long)(p.KH + kh) * p.dim + d) * rk;
+        s_q[d] = Typed<T>::load(mixed + (long long)kh * p.dim + d) * rq;
+      }
+      __syncthreads();
+    }
+    float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int i = 0; i < RPT; ++i) {
+      const int d = rg + i * 8;
+      S[i].x *= g; S[i].y *= g; S[i].z *= g; S[i].w *= g;
+      const float k = d < p.dim ? s_k[d] : 0.f;
+      a.x += S[i].x * k; a.y += S[i].y * k; a.z += S[i].z * k; a.w += S[i].w * k;
+    }
+    s_r[rg * 32 + c] = a;
+    __syncthreads();
+    float4 t = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int r = 0; r < 8; ++r) {
+      const float4 x = s_r[r * 32 + c];
+      t.x += x.x; t.y += x.y; t.z += x.z; t.w += x.w;
+    }
+    __syncthreads();
+    float4 u = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (ok) {
+      const T* vp = mixed + 2ll * p.KH * p.dim + (long long)h * p.vdim + v;
+      u = make_float4(beta * (Typed<T>::load(vp) - t.x), beta * (Typed<T>::load(vp + 1) - t.y), beta * (Typed<T>::load(vp + 2) - t.z),
+                      beta * (Typed<T>::load(vp + 3) - t.w));
+    }
+    a = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int i = 0; i < RPT; ++i) {
+      const int d = rg + i * 8;
+      if (d < p.dim) {
+        const float k = s_k[d], q = s_q[d];
+        S[i].x += k * u.x; S[i].y += k * u.y; S[i].z += k * u.z; S[i].w += k * u.w;
+        a.x += S[i].x * q; a.y += S[i].y * q; a.z += S[i].z * q; a.w += S[i].w * q;
+        if (ok && keep) __stcs(reinterpret_cast<float4*>(st + (long long)d * p.vdim + v), S[i]);
+      }
+    }
+    s_r[rg * 32 + c] = a;
+    __syncthreads();
+    if (rg == 0 && ok) {
+      t = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+      for (int r = 0; r < 8; ++r) {
+        const float4 x = s_r[r * 32 + c];
+        t.x += x.x; t.y += x.y; t.z += x.z; t.w += x.w;
+      }
+      s_o[v] = t.x; s_o[v + 1] = t.y; s_o[v + 2] = t.z; s_o[v + 3] = t.w;
+      ss += t.x * t.x + t.y * t.y + t.z * t.z + t.w * t.w;
+    }
+    __syncthreads();
+  }
+  ss = block_sum(ss, s_red);
+  const float r = 1.f / sqrtf(ss / float(p.vdim) + p.eps);
+  T* out = static_cast<T*>(p.out) + (long long)b * p.ldout;
+  const T* gt = static_cast<const T*>(p.gate) + (long long)b * p.ldg + (long long)h * p.vdim;
+  for (int v = tid; v < p.vdim; v += SV_THREADS) {
+    const float z = Typed<T>::load(gt + v);
+    Typed<T>::store(out + (long long)h * p.vdim + v, s_o[v] * r * p.w[v] * z * Typed<T>::sigmoid_(z));
+  }
+  if (h == 0)
+    for (int v = p.H * p.vdim + tid; v < p.ldout; v += SV_THREADS) Typed<T>::store(out + v, 0.f);
+}
+
 template <typename T>
 static int launch_scan(const ScanArgs& p, cudaStream_t s) {
   const long long pw = (long long)p.B * p.groups * p.KH;
   launch_pdl(delta_pairs_kernel<T>, dim3(unsigned((pw + 3) / 4)), dim3(128), 0, s, p);
-  auto grid = [&](int cpl) { return dim3((p.vdim + 16 * cpl - 1) / (16 * cpl), p.H, p.B); };
-  if (p.dim <= 32) launch_pdl(delta_scan_kernel<T, 4, 2, 4>, grid(2), dim3(128), 0, s, p);
-  else if (p.dim <= 64) launch_pdl(delta_scan_kernel<T, 8, 2, 4>, grid(2), dim3(128), 0, s, p);
-  else if (p.dim <= 128) launch_pdl(delta_scan_kernel<T, 16, 2, 4>, grid(2), dim3(128), 0, s, p);
-  else if (p.dim <= 256) launch_pdl(delta_scan_kernel<T, 32, 1, 3>, grid(1), dim3(128), 0, s, p);
+  auto grid = [&](int cpl) { return dim3((p.vdim + 8 * cpl - 1) / (8 * cpl), p.H, p.B); };
+  if (p.dim <= 64) launch_pdl(delta_scan_kernel<T, 4, 8>, grid(8), dim3(128), 0, s, p);
+  else if (p.dim <= 128) launch_pdl(delta_scan_kernel<T, 8, 8>, grid(8), dim3(128), 0, s, p);
+  else if (p.dim <= 256) launch_pdl(delta_scan_kernel<T, 16, 4>, grid(4), dim3(128), 0, s, p);
   else return 1006;
   return int(cudaGetLastError());
 }
 
 template <typename T>
 static int launch_step(const StepArgs& p, cudaStream_t s) {
+  if ((p.vdim & 3) == 0 && p.dim <= 256 && (p.state_bs & 3) == 0 && (reinterpret_cast<uintptr_t>(p.state) & 15) == 0) {
+    const size_t sm = size_t(8 * 32 * 4 + 2 * p.dim + p.vdim + 40) * sizeof(float);
+    if (sm <= 48 * 1024) {
+      const dim3 vgrid(p.H, p.B);
+      if (p.dim <= 64) launch_pdl(delta_step_vec_kernel<T, 8>, vgrid, dim3(SV_THREADS), sm, s, p);
+      else if (p.dim <= 128) launch_pdl(delta_step_vec_kernel<T, 16>, vgrid, dim3(SV_THREADS), sm, s, p);
+      else launch_pdl(delta_step_vec_kernel<T, 32>, vgrid, dim3(SV_THREADS), sm, s, p);
+      return int(cudaGetLastError());
+    }
+  }
   int CW = 32;
   while (CW < p.vdim && CW < 128) CW *= 2;
   const int rg = ST_THREADS / CW, rows = (p.dim + rg - 1) / rg;
@@ -676,10 +823,10 @@ static int launch_prep(const DeltaArgs& p, cudaStream_t s) {
   const bool aligned = (p.ld & 7) == 0 && (p.ldm & 7) == 0 && (p.C & 7) == 0 && (reinterpret_cast<uintptr_t>(p.proj) & 15) == 0 &&
                        (reinterpret_cast<uintptr_t>(p.tail) & 15) == 0 && (p.tail_bs & 7) == 0;
   if (!p.lengths && aligned && pow2_lanes(p.dim) && (p.vdim & 7) == 0 && p.taps >= 2 && p.taps <= 4) {
-    const long long blocks = (long long)p.B * ((p.L + PT - 1) / PT) * (((p.C >> 3) + 255) / 256);
-    if (p.taps == 2) launch_pdl(delta_prep_vec_kernel<T, 2>, dim3(unsigned(blocks)), dim3(256), 0, s, p);
-    else if (p.taps == 3) launch_pdl(delta_prep_vec_kernel<T, 3>, dim3(unsigned(blocks)), dim3(256), 0, s, p);
-    else launch_pdl(delta_prep_vec_kernel<T, 4>, dim3(unsigned(blocks)), dim3(256), 0, s, p);
+    const long long blocks = (long long)p.B * ((p.L + PT - 1) / PT) * (((p.C >> 3) + PV_THREADS - 1) / PV_THREADS);
+    if (p.taps == 2) launch_pdl(delta_prep_vec_kernel<T, 2>, dim3(unsigned(blocks)), dim3(PV_THREADS), 0, s, p);
+    else if (p.taps == 3) launch_pdl(delta_prep_vec_kernel<T, 3>, dim3(unsigned(blocks)), dim3(PV_THREADS), 0, s, p);
+    else launch_pdl(delta_prep_vec_kernel<T, 4>, dim3(unsigned(blocks)), dim3(PV_THREADS), 0, s, p);
     launch_pdl(delta_gates_kernel<T>, dim3(unsigned(((long long)p.B * p.L * p.H + 255) / 256)), dim3(256), 0, s, p);
   } else {
     const long long warps = (long long)p.B * p.L * (2 * p.KH + p.H + 1);

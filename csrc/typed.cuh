@@ -17,6 +17,12 @@ template <> struct Typed<float> {
     *reinterpret_cast<float4*>(v) = *reinterpret_cast<const float4*>(p);
     *reinterpret_cast<float4*>(v + 4) = *reinterpret_cast<const float4*>(p + 4);
   }
+  struct Raw8 { float4 a, b; };
+  static __device__ __forceinline__ Raw8 raw8(const float* p) { return {*reinterpret_cast<const float4*>(p), *reinterpret_cast<const float4*>(p + 4)}; }
+  static __device__ __forceinline__ void unpack8(const Raw8& r, float (&v)[8]) {
+    v[0] = r.a.x; v[1] = r.a.y; v[2] = r.a.z; v[3] = r.a.w;
+    v[4] = r.b.x; v[5] = r.b.y; v[6] = r.b.z; v[7] = r.b.w;
+  }
   static __device__ __forceinline__ void store8(float* p, const float (&v)[8]) {
     *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
     *reinterpret_cast<float4*>(p + 4) = make_float4(v[4], v[5], v[6], v[7]);
@@ -37,8 +43,10 @@ template <> struct Typed<__nv_bfloat16> {
   static __device__ __forceinline__ void store4(__nv_bfloat16* p, float4 v) {
     *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(v.x, v.y), pack_bf16x2(v.z, v.w));
   }
-  static __device__ __forceinline__ void load8(const __nv_bfloat16* p, float (&v)[8]) {
-    const uint4 u = *reinterpret_cast<const uint4*>(p);
+  using Raw8 = uint4;
+  static __device__ __forceinline__ Raw8 raw8(const __nv_bfloat16* p) { return *reinterpret_cast<const uint4*>(p); }
+  static __device__ __forceinline__ void load8(const __nv_bfloat16* p, float (&v)[8]) { unpack8(raw8(p), v); }
+  static __device__ __forceinline__ void unpack8(const Raw8& u, float (&v)[8]) {
     const float2 a = unpack_bf16x2(u.x), b = unpack_bf16x2(u.y), c = unpack_bf16x2(u.z), d = unpack_bf16x2(u.w);
     v[0] = a.x; v[1] = a.y; v[2] = b.x; v[3] = b.y; v[4] = c.x; v[5] = c.y; v[6] = d.x; v[7] = d.y;
   }
