@@ -141,7 +141,7 @@ class GatedDelta(_Weights):
         self.put("w_in", stacked([(take("q"), 0), (take("k"), kd), (take("v"), 2 * kd), (take("g"), s.g_col), (take("a"), s.a_col), (take("b"), s.b_col)], Dp,
                                  dtype, device))
         self.put("w_o", padded(take("o"), Dp, s.o_pad, dtype, device))
-        self.put("conv", torch.cat([take(n + ".conv") for n in "qkv"]).to(device=device, dtype=torch.float32).contiguous())
+        self.put("conv", torch.cat([take(n + ".conv") for n in "qkv"]).T.to(device=device, dtype=torch.float32).contiguous())
         self.put("neg_rate", -torch.exp(vector(take("A_log"), device)))
         self.put("dt_bias", vector(take("dt_bias"), device))
         self.put("norm", vector(take("norm"), device))

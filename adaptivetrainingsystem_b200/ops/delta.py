@@ -107,7 +107,7 @@ def _norm_gate(o: torch.Tensor, gate: torch.Tensor, w: torch.Tensor, s: DeltaSha
 # ----------------------------------------------------------------------------------------------------------
 def delta_prep(proj: torch.Tensor, s: DeltaShape, conv: torch.Tensor, neg_rate: torch.Tensor, dt_bias: torch.Tensor, tail: torch.Tensor, pos0: int = 0,
                lengths: Optional[torch.Tensor] = None, active: Optional[torch.Tensor] = None) -> Tuple[torch.Tensor, torch.Tensor, torch.Tensor]:
-    """proj [B, L, proj_width]; conv [channels, taps], neg_rate = -exp(A_log), dt_bias [H] in fp32; tail [B, taps - 1, channels] ->
+    """proj [B, L, proj_width]; conv [taps, channels] (last row: current token), neg_rate = -exp(A_log), dt_bias [H] in fp32; tail [B, taps - 1, channels] ->
     (mixed [B * L, .], reciprocal lengths [B * L, 2 kv_heads], [decay, step size] [B * L, 2 H]); the tail moves on by the portion."""
     B, L, _ = proj.shape
     H, KH, C, n = s.heads, s.kv_heads, s.channels, s.taps - 1
@@ -116,7 +116,7 @@ def delta_prep(proj: torch.Tensor, s: DeltaShape, conv: torch.Tensor, neg_rate: 
         fresh = [(int(lengths[b]) if lengths is not None else pos0) == 0 for b in range(B)]
         old = torch.stack([torch.zeros_like(tail[b]) if fresh[b] else tail[b] for b in range(B)])
         full = torch.cat([old, x], dim=1)
-        y = sum(full[:, j:j + L].float() * conv[:, j] for j in range(s.taps))
+        y = sum(full[:, j:j + L].float() * conv[j] for j in range(s.taps))
         mixed = torch.nn.functional.silu(y).to(proj.dtype).view(B * L, C)
         for b in range(B):
             if active is None or int(active[b]):

@@ -25,7 +25,7 @@ struct DeltaArgs {
   long long ld;
   int g_col, a_col, b_col;
   int B, L, H, KH, dim, vdim, taps, C;   // C = 2 * KH * dim + H * vdim convolved channels
-  const float* conv;       // [C, taps]
+  const float* conv;       // [taps, C], last row = current token
   const float* neg_rate;   // [H] -exp(A_log)
   const float* dt_bias;    // [H]
   void* tail;              // [B, taps - 1, C] last inputs of the convolutions (oldest first)
@@ -40,6 +40,15 @@ struct DeltaArgs {
 };
 
 template <typename T>
+__device__ __forceinline__ void delta_gate(const DeltaArgs& p, long long row, int h) {
+  const T* in = static_cast<const T*>(p.proj) + row * p.ld;
+  const float a = Typed<T>::load(in + p.a_col + h) + p.dt_bias[h], bt = Typed<T>::load(in + p.b_col + h);
+  const float sp = a > 20.f ? a : log1pf(expf(a));
+  p.gb[row * 2 * p.H + h] = expf(p.neg_rate[h] * sp);
+  p.gb[row * 2 * p.H + p.H + h] = 1.f / (1.f + expf(-bt));
+}
+
+template <typename T>
 __global__ void __launch_bounds__(256) delta_prep_kernel(const DeltaArgs p) {
   pdl_prologue();
   const int units = 2 * p.KH + p.H + 1, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -50,12 +59,7 @@ __global__ void __launch_bounds__(256) delta_prep_kernel(const DeltaArgs p) {
   const int pos0 = p.lengths ? p.lengths[b] : p.pos0;
   const T* in = static_cast<const T*>(p.proj) + row * p.ld;
   if (unit == units - 1) {  // decay and step size of every head
-    for (int h = lane; h < p.H; h += 32) {
-      const float a = Typed<T>::load(in + p.a_col + h) + p.dt_bias[h], bt = Typed<T>::load(in + p.b_col + h);
-      const float sp = a > 20.f ? a : log1pf(expf(a));
-      p.gb[row * 2 * p.H + h] = expf(p.neg_rate[h] * sp);
-      p.gb[row * 2 * p.H + p.H + h] = 1.f / (1.f + expf(-bt));
-    }
+    for (int h = lane; h < p.H; h += 32) delta_gate<T>(p, row, h);
     return;
   }
   const int width = unit < 2 * p.KH ? p.dim : p.vdim;
@@ -66,14 +70,14 @@ __global__ void __launch_bounds__(256) delta_prep_kernel(const DeltaArgs p) {
   float ss = 0.f;
   for (int i = lane; i < width; i += 32) {
     const int c = c0 + i;
-    const float* cw = p.conv + (long long)c * p.taps;
+    const float* cw = p.conv + c;
     const T cur = in[c];
-    float acc = Typed<T>::load(&cur) * cw[p.taps - 1];
+    float acc = Typed<T>::load(&cur) * cw[(long long)(p.taps - 1) * p.C];
     for (int j = 1; j < p.taps; ++j) {  // j tokens back
       float x = 0.f;
       if (t - j >= 0) x = Typed<T>::load(in - j * p.ld + c);
       else if (pos0 > 0) x = Typed<T>::load(tail + (long long)(p.taps - 1 + t - j) * p.C + c);
-      acc += x * cw[p.taps - 1 - j];
+      acc += x * cw[(long long)(p.taps - 1 - j) * p.C];
     }
     if (keep) {  // decoding: shift the channel's inputs (this thread is the only one that touches them)
       for (int j = 0; j < p.taps - 2; ++j) {
@@ -96,12 +100,18 @@ __global__ void __launch_bounds__(256) delta_prep_kernel(const DeltaArgs p) {
   }
 }
 
-// The same for portions whose heads are whole 16-byte pieces: a thread owns eight channels and walks PT consecutive tokens with the
-// convolution's inputs in registers; the lanes of a head (dim / 8 of them, a power of two) add up its length with shuffles.
-constexpr int PT = 16, PV_THREADS = 128;
+// The same when heads are whole 16-byte pieces: a thread owns eight channels and walks PT consecutive tokens with the convolution's
+// inputs in registers; the lanes of a head (dim / 8 of them, a power of two) add up its length with shuffles.  The blocks after
+// `conv_blocks` compute decays and step sizes.
+constexpr int PT = 32, PV_THREADS = 128;
 template <typename T, int TAPS>
-__global__ void __launch_bounds__(PV_THREADS, 4) delta_prep_vec_kernel(const DeltaArgs p) {
+__global__ void __launch_bounds__(PV_THREADS, 4) delta_prep_vec_kernel(const DeltaArgs p, int conv_blocks) {
   pdl_prologue();
+  if (int(blockIdx.x) >= conv_blocks) {
+    const long long i = (blockIdx.x - conv_blocks) * (long long)PV_THREADS + threadIdx.x;
+    if (i < (long long)p.B * p.L * p.H) delta_gate<T>(p, i / p.H, int(i % p.H));
+    return;
+  }
   const int pieces = p.C >> 3, per_block = (pieces + PV_THREADS - 1) / PV_THREADS, blocks_t = (p.L + PT - 1) / PT;
   const int piece = (blockIdx.x % per_block) * PV_THREADS + threadIdx.x;
   const int tb = (blockIdx.x / per_block) % blocks_t, b = blockIdx.x / per_block / blocks_t;
@@ -113,14 +123,13 @@ __global__ void __launch_bounds__(PV_THREADS, 4) delta_prep_vec_kernel(const Del
   T* out = static_cast<T*>(p.mixed) + (long long)b * p.L * p.ldm + c;
   float w[TAPS][8], x[TAPS][8];  // x[j]: the input j tokens back (x[0] = current)
 #pragma unroll
-  for (int e = 0; e < 8; ++e)
-#pragma unroll
-    for (int j = 0; j < TAPS; ++j) w[j][e] = p.conv[(long long)(c + e) * TAPS + TAPS - 1 - j];
+  for (int j = 0; j < TAPS; ++j) Typed<float>::load8(p.conv + (long long)(TAPS - 1 - j) * p.C + c, w[j]);
+  const int pos0 = p.lengths ? p.lengths[b] : p.pos0;
 #pragma unroll
   for (int j = 1; j < TAPS; ++j) {
     const int t = t0 - j;
     if (t >= 0) Typed<T>::load8(in + (long long)t * p.ld, x[j - 1]);
-    else if (p.pos0 > 0) Typed<T>::load8(tail + (long long)(TAPS - 1 + t) * p.C, x[j - 1]);
+    else if (pos0 > 0) Typed<T>::load8(tail + (long long)(TAPS - 1 + t) * p.C, x[j - 1]);
     else
 #pragma unroll
       for (int e = 0; e < 8; ++e) x[j - 1][e] = 0.f;
@@ -169,20 +178,11 @@ __global__ void __launch_bounds__(PV_THREADS, 4) delta_prep_vec_kernel(const Del
       }
     }
   }
-}
-
-template <typename T>
-__global__ void __launch_bounds__(256) delta_gates_kernel(const DeltaArgs p) {
-  pdl_prologue();
-  const long long i = blockIdx.x * 256ll + threadIdx.x;
-  if (i >= (long long)p.B * p.L * p.H) return;
-  const long long row = i / p.H;
-  const int h = int(i % p.H);
-  const T* in = static_cast<const T*>(p.proj) + row * p.ld;
-  const float a = Typed<T>::load(in + p.a_col + h) + p.dt_bias[h], bt = Typed<T>::load(in + p.b_col + h);
-  const float sp = a > 20.f ? a : log1pf(expf(a));
-  p.gb[row * 2 * p.H + h] = expf(p.neg_rate[h] * sp);
-  p.gb[row * 2 * p.H + p.H + h] = 1.f / (1.f + expf(-bt));
+  if (p.lengths && live && !(p.active && !p.active[b])) {  // decoding: this thread's channels move on by the token
+    T* tw = static_cast<T*>(p.tail) + (long long)b * p.tail_bs + c;
+#pragma unroll
+    for (int j = 0; j < TAPS - 1; ++j) Typed<T>::store8(tw + (long long)(TAPS - 2 - j) * p.C, x[j]);
+  }
 }
 
 // After a portion: the last taps - 1 inputs of every channel (one thread per channel, oldest first, in place).
@@ -223,8 +223,27 @@ struct ScanArgs {
   int B, L, H, KH, dim, vdim, groups, fresh;
 };
 
+// 16 x 8 products of one group: rows 0..7 k_i . k_j, rows 8..15 q_i . k_j, sums over dim.  bf16 values: exact products accumulated in
+// fp32 by a warp-level MMA, whose B fragment is the same registers as the upper half of A (the order of the reduction is
+// permuted so that a lane's 16-byte piece serves two steps).
+__device__ __forceinline__ void group_products_mma(const __nv_bfloat16* q, const __nv_bfloat16* k, long long ldm, int dim, int n, int lane, float (&c)[4]) {
+  const int g = lane >> 2, t = lane & 3;
+  c[0] = c[1] = c[2] = c[3] = 0.f;
+  for (int d = 8 * t; d < ((dim + 31) & ~31); d += 32) {
+    uint4 kv = make_uint4(0, 0, 0, 0), qv = make_uint4(0, 0, 0, 0);
+    if (g < n && d < dim) {
+      kv = *reinterpret_cast<const uint4*>(k + g * ldm + d);
+      qv = *reinterpret_cast<const uint4*>(q + g * ldm + d);
+    }
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(kv.x), "r"(qv.x), "r"(kv.y), "r"(qv.y), "r"(kv.x), "r"(kv.y));
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(kv.z), "r"(qv.z), "r"(kv.w), "r"(qv.w), "r"(kv.z), "r"(kv.w));
+  }
+}
+
 // One warp per (group, kv head, sequence): 8 x 8 products of the keys with keys and queries, then per value head the inverse.
-template <typename T>
+template <typename T, bool MMA>
 __global__ void __launch_bounds__(128) delta_pairs_kernel(const ScanArgs p) {
   pdl_prologue();
   __shared__ float s_kk[4][DC][DC + 1], s_kq[4][DC][DC + 1];
@@ -237,6 +256,19 @@ __global__ void __launch_bounds__(128) delta_pairs_kernel(const ScanArgs p) {
   const T* base = static_cast<const T*>(p.mixed) + row0 * p.ldm;
   const T* q = base + (long long)kh * p.dim;
   const T* k = base + (long long)(p.KH + kh) * p.dim;
+  const float* rl = p.rlen + row0 * 2 * p.KH;
+  if constexpr (MMA) {
+    float c[4];
+    group_products_mma(q, k, p.ldm, p.dim, n, lane, c);
+    const int i = lane >> 2, j = 2 * (lane & 3);
+    const float rki = i < n ? rl[(long long)i * 2 * p.KH + p.KH + kh] : 0.f, rqi = i < n ? rl[(long long)i * 2 * p.KH + kh] : 0.f;
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const float rkj = j + e < n ? rl[(long long)(j + e) * 2 * p.KH + p.KH + kh] : 0.f;
+      s_kk[warp][i][j + e] = c[e] * rki * rkj;
+      s_kq[warp][i][j + e] = c[2 + e] * rqi * rkj;
+    }
+  } else {
   float kk[DC][DC], kq[DC][DC];
 #pragma unroll
   for (int i = 0; i < DC; ++i)
@@ -257,7 +289,6 @@ __global__ void __launch_bounds__(128) delta_pairs_kernel(const ScanArgs p) {
         kq[i][j] += qv[i] * kv[j];
       }
   }
-  const float* rl = p.rlen + row0 * 2 * p.KH;
 #pragma unroll
   for (int i = 0; i < DC; ++i)
 #pragma unroll
@@ -270,6 +301,7 @@ __global__ void __launch_bounds__(128) delta_pairs_kernel(const ScanArgs p) {
         s_kq[warp][i][j] = c * rqi * rkj;
       }
     }
+  }
   __syncwarp();
   // lane = (value head of the group r, column c of the 8 x 8 inverse)
   for (int x = lane; x < rep * DC; x += 32) {
@@ -776,7 +808,13 @@ __global__ void __launch_bounds__(SV_THREADS, RPT <= 8 ? 4 : RPT <= 16 ? 2 : 1) 
 template <typename T>
 static int launch_scan(const ScanArgs& p, cudaStream_t s) {
   const long long pw = (long long)p.B * p.groups * p.KH;
-  launch_pdl(delta_pairs_kernel<T>, dim3(unsigned((pw + 3) / 4)), dim3(128), 0, s, p);
+  const dim3 pgrid(unsigned((pw + 3) / 4));
+  if constexpr (sizeof(T) == 2) {
+    if ((p.dim & 7) == 0 && (p.ldm & 7) == 0) launch_pdl(delta_pairs_kernel<T, true>, pgrid, dim3(128), 0, s, p);
+    else launch_pdl(delta_pairs_kernel<T, false>, pgrid, dim3(128), 0, s, p);
+  } else {
+    launch_pdl(delta_pairs_kernel<T, false>, pgrid, dim3(128), 0, s, p);
+  }
   auto grid = [&](int cpl) { return dim3((p.vdim + 8 * cpl - 1) / (8 * cpl), p.H, p.B); };
   if (p.dim <= 64) launch_pdl(delta_scan_kernel<T, 4, 8>, grid(8), dim3(128), 0, s, p);
   else if (p.dim <= 128) launch_pdl(delta_scan_kernel<T, 8, 8>, grid(8), dim3(128), 0, s, p);
@@ -822,12 +860,12 @@ template <typename T>
 static int launch_prep(const DeltaArgs& p, cudaStream_t s) {
   const bool aligned = (p.ld & 7) == 0 && (p.ldm & 7) == 0 && (p.C & 7) == 0 && (reinterpret_cast<uintptr_t>(p.proj) & 15) == 0 &&
                        (reinterpret_cast<uintptr_t>(p.tail) & 15) == 0 && (p.tail_bs & 7) == 0;
-  if (!p.lengths && aligned && pow2_lanes(p.dim) && (p.vdim & 7) == 0 && p.taps >= 2 && p.taps <= 4) {
-    const long long blocks = (long long)p.B * ((p.L + PT - 1) / PT) * (((p.C >> 3) + PV_THREADS - 1) / PV_THREADS);
-    if (p.taps == 2) launch_pdl(delta_prep_vec_kernel<T, 2>, dim3(unsigned(blocks)), dim3(PV_THREADS), 0, s, p);
-    else if (p.taps == 3) launch_pdl(delta_prep_vec_kernel<T, 3>, dim3(unsigned(blocks)), dim3(PV_THREADS), 0, s, p);
-    else launch_pdl(delta_prep_vec_kernel<T, 4>, dim3(unsigned(blocks)), dim3(PV_THREADS), 0, s, p);
-    launch_pdl(delta_gates_kernel<T>, dim3(unsigned(((long long)p.B * p.L * p.H + 255) / 256)), dim3(256), 0, s, p);
+  if (aligned && pow2_lanes(p.dim) && (p.vdim & 7) == 0 && p.taps >= 2 && p.taps <= 4) {
+    const int conv = p.B * ((p.L + PT - 1) / PT) * (((p.C >> 3) + PV_THREADS - 1) / PV_THREADS);
+    const dim3 grid(unsigned(conv + ((long long)p.B * p.L * p.H + PV_THREADS - 1) / PV_THREADS));
+    if (p.taps == 2) launch_pdl(delta_prep_vec_kernel<T, 2>, grid, dim3(PV_THREADS), 0, s, p, conv);
+    else if (p.taps == 3) launch_pdl(delta_prep_vec_kernel<T, 3>, grid, dim3(PV_THREADS), 0, s, p, conv);
+    else launch_pdl(delta_prep_vec_kernel<T, 4>, grid, dim3(PV_THREADS), 0, s, p, conv);
   } else {
     const long long warps = (long long)p.B * p.L * (2 * p.KH + p.H + 1);
     launch_pdl(delta_prep_kernel<T>, dim3(unsigned((warps + 7) / 8)), dim3(256), 0, s, p);

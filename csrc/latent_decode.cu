@@ -6,8 +6,8 @@
 //                            the MMA), soft-max, weighted sum of the latents; chunks of the ring are merged by the next kernel
 //   latent_head_mm<expand>   out[b, h, :] = sigmoid(gate) * W_uv[h] (merged latent)   [16 sequences x rank] x [rank x vdim]
 //
-// A decode step is bound by the bytes of the ring, so warp-level MMAs are enough; a 64-row tile of the ring is fetched once with
-// cp.async and serves both products (plain and transposing ldmatrix; rows are padded by 16 bytes against bank conflicts).  Weights
+// A decode step is bound by the bytes of the ring, so warp-level MMAs are enough; a 32-row tile of the ring is fetched once with
+// cp.async (the next one while this one is used) and serves both products (plain and transposing ldmatrix; rows are padded by 16 bytes against bank conflicts).  Weights
 // stream straight from global memory into B fragments: the order of the reduction index is permuted so that the 16-byte piece a lane
 // loads is its fragment for two consecutive steps, and the A fragments are read with the same permutation.
 #include "common.cuh"
@@ -29,10 +29,9 @@ __device__ __forceinline__ void ldmatrix_x4_trans(uint32_t addr, uint32_t (&r)[4
 __device__ __forceinline__ void cp_async_16(uint32_t dst, const void* src, bool ok) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(ok ? 16 : 0) : "memory");
 }
-__device__ __forceinline__ void cp_async_wait_all() {
-  asm volatile("cp.async.commit_group;" ::: "memory");
-  asm volatile("cp.async.wait_group 0;" ::: "memory");
-}
+__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N>
+__device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
 struct HeadMmArgs {
   const __nv_bfloat16* x;   // absorb: q, head h at h * x_hs, rows x_ld apart
@@ -51,7 +50,7 @@ struct HeadMmArgs {
   long long ldg;
   int B, H, N, K;
 };
-constexpr int HM_MAX_CHUNKS = 64;
+constexpr int HM_MAX_CHUNKS = 64;  // two per lane in the merge
 
 // CTA: 16 sequences x (WARPS * NT * 8) output columns of one head.
 template <int WARPS, int NT, bool EXPAND>
@@ -63,18 +62,26 @@ __global__ void __launch_bounds__(WARPS * 32) latent_head_mm_kernel(const HeadMm
   const int ldx = p.K + 32, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
   const int h = blockIdx.y, b0 = blockIdx.z * 16, nb = min(16, p.B - b0);
   const int n0 = (blockIdx.x * WARPS + warp) * NT * 8;
+  // the first PRE steps of this lane's weights, requested before the inputs are gathered
+  constexpr int PRE = 4;
+  const __nv_bfloat16* w = p.w + h * p.w_hs + 8 * t;
+  uint4 pre[PRE][NT];
+#pragma unroll
+  for (int u = 0; u < PRE; ++u)
+#pragma unroll
+    for (int i = 0; i < NT; ++i) {
+      const int n = n0 + i * 8 + g;
+      pre[u][i] = (n < p.N && u * 32 < p.K) ? *reinterpret_cast<const uint4*>(w + (long long)n * p.ldw + u * 32) : make_uint4(0, 0, 0, 0);
+    }
   if (EXPAND) {
-    if (tid < 16 && tid < nb) {
-      const float* ml = p.part_ml + ((long long)(b0 + tid) * p.H + h) * p.n_chunks * 2;
-      float m = -INFINITY, l = 0.f;
-      for (int c = 0; c < p.n_chunks; ++c) m = fmaxf(m, ml[2 * c]);
-      for (int c = 0; c < p.n_chunks; ++c) {
-        const float f = ml[2 * c + 1] > 0.f ? __expf(ml[2 * c] - m) : 0.f;
-        s_f[tid][c] = f;
-        l += f * ml[2 * c + 1];
-      }
-      const float inv = 1.f / l;
-      for (int c = 0; c < p.n_chunks; ++c) s_f[tid][c] *= inv;
+    for (int j = warp; j < nb; j += WARPS) {  // merge factors of the chunks: one warp per sequence, lanes over chunks
+      const float2* ml = reinterpret_cast<const float2*>(p.part_ml) + ((long long)(b0 + j) * p.H + h) * p.n_chunks;
+      const float2 x0 = lane < p.n_chunks ? ml[lane] : make_float2(-INFINITY, 0.f), x1 = lane + 32 < p.n_chunks ? ml[lane + 32] : make_float2(-INFINITY, 0.f);
+      const float m = warp_max(fmaxf(x0.x, x1.x));
+      const float f0 = x0.y > 0.f ? __expf(x0.x - m) : 0.f, f1 = x1.y > 0.f ? __expf(x1.x - m) : 0.f;
+      const float inv = 1.f / warp_sum(f0 * x0.y + f1 * x1.y);
+      s_f[j][lane] = f0 * inv;
+      s_f[j][lane + 32] = f1 * inv;
     }
     __syncthreads();
     const int quads = p.K >> 2;
@@ -83,12 +90,12 @@ __global__ void __launch_bounds__(WARPS * 32) latent_head_mm_kernel(const HeadMm
       float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
       if (j < nb) {
         const float* po = p.part_o + (((long long)(b0 + j) * p.H + h) * p.n_chunks) * p.K + r;
+#pragma unroll 4
         for (int c = 0; c < p.n_chunks; ++c) {
           const float f = s_f[j][c];
-          if (f > 0.f) {  // chunks beyond a short sequence were not written
-            const float4 v = *reinterpret_cast<const float4*>(po + (long long)c * p.K);
-            a.x += f * v.x; a.y += f * v.y; a.z += f * v.z; a.w += f * v.w;
-          }
+          // (a chunk beyond a short sequence was not written: its factor is zero and its values are not used)
+          const float4 v = f > 0.f ? *reinterpret_cast<const float4*>(po + (long long)c * p.K) : make_float4(0.f, 0.f, 0.f, 0.f);
+          a.x += f * v.x; a.y += f * v.y; a.z += f * v.z; a.w += f * v.w;
         }
       }
       *reinterpret_cast<uint2*>(sx + j * ldx + r) = make_uint2(pack_bf16x2(a.x, a.y), pack_bf16x2(a.z, a.w));
@@ -108,16 +115,27 @@ __global__ void __launch_bounds__(WARPS * 32) latent_head_mm_kernel(const HeadMm
   for (int i = 0; i < NT; ++i)
 #pragma unroll
     for (int e = 0; e < 4; ++e) acc[i][e] = 0.f;
-  const __nv_bfloat16* w = p.w + h * p.w_hs + 8 * t;
-#pragma unroll 4
-  for (int k = 0; k < p.K; k += 32) {
-    const uint4 lo = *reinterpret_cast<const uint4*>(sx + g * ldx + k + 8 * t), hi = *reinterpret_cast<const uint4*>(sx + (g + 8) * ldx + k + 8 * t);
+  // blocks of PRE steps: the next block's weights are in flight while this one is multiplied
+  for (int k0 = 0; k0 < p.K; k0 += 32 * PRE) {
+    uint4 cur[PRE][NT];
 #pragma unroll
-    for (int i = 0; i < NT; ++i) {
-      const int n = n0 + i * 8 + g;
-      const uint4 b = n < p.N ? *reinterpret_cast<const uint4*>(w + (long long)n * p.ldw + k) : make_uint4(0, 0, 0, 0);
-      mma_bf16_16816(acc[i], lo.x, hi.x, lo.y, hi.y, b.x, b.y);
-      mma_bf16_16816(acc[i], lo.z, hi.z, lo.w, hi.w, b.z, b.w);
+    for (int u = 0; u < PRE; ++u)
+#pragma unroll
+      for (int i = 0; i < NT; ++i) {
+        cur[u][i] = pre[u][i];
+        const int n = n0 + i * 8 + g, k = k0 + 32 * (PRE + u);
+        pre[u][i] = (n < p.N && k < p.K) ? *reinterpret_cast<const uint4*>(w + (long long)n * p.ldw + k) : make_uint4(0, 0, 0, 0);
+      }
+#pragma unroll
+    for (int u = 0; u < PRE; ++u) {
+      const int k = k0 + 32 * u;
+      if (k >= p.K) break;
+      const uint4 lo = *reinterpret_cast<const uint4*>(sx + g * ldx + k + 8 * t), hi = *reinterpret_cast<const uint4*>(sx + (g + 8) * ldx + k + 8 * t);
+#pragma unroll
+      for (int i = 0; i < NT; ++i) {
+        mma_bf16_16816(acc[i], lo.x, hi.x, lo.y, hi.y, cur[u][i].x, cur[u][i].y);
+        mma_bf16_16816(acc[i], lo.z, hi.z, lo.w, hi.w, cur[u][i].z, cur[u][i].w);
+      }
     }
   }
 #pragma unroll
@@ -155,15 +173,15 @@ struct RingArgs {
   float* part_o;              // [B, H, n_chunks, rank]
   float* part_ml;             // [B, H, n_chunks, 2]
 };
-constexpr int LR_KEYS = 64, LR_THREADS = 256;
+constexpr int LR_KEYS = 32, LR_THREADS = 256;
 
 struct RingSmem {
   int ldt, qa, s, pr, al, total;  // row pitch of tile and queries (elements), byte offsets
   __host__ __device__ explicit RingSmem(int cw) {
     ldt = cw + 8;
-    qa = LR_KEYS * ldt * 2;
+    qa = 2 * LR_KEYS * ldt * 2;
     s = qa + 16 * ldt * 2;
-    pr = s + 16 * (LR_KEYS + 4) * 4;
+    pr = s + 2 * 16 * (LR_KEYS + 4) * 4;
     al = pr + 16 * (LR_KEYS + 8) * 2;
     total = al + 16 * 4;
   }
@@ -178,7 +196,7 @@ __global__ void __launch_bounds__(LR_THREADS, 2) latent_ring_kernel(const RingAr
   const RingSmem L(cw);
   __nv_bfloat16* tile = reinterpret_cast<__nv_bfloat16*>(smem_raw);
   __nv_bfloat16* sq = reinterpret_cast<__nv_bfloat16*>(smem_raw + L.qa);
-  float* ss = reinterpret_cast<float*>(smem_raw + L.s);                  // [16][LR_KEYS + 4]
+  float* ss = reinterpret_cast<float*>(smem_raw + L.s);                  // [half of the reduction][16][LR_KEYS + 4]
   __nv_bfloat16* sp = reinterpret_cast<__nv_bfloat16*>(smem_raw + L.pr);  // [16][LR_KEYS + 8]
   float* sal = reinterpret_cast<float*>(smem_raw + L.al);                // [16]
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
@@ -193,15 +211,19 @@ __global__ void __launch_bounds__(LR_THREADS, 2) latent_ring_kernel(const RingAr
     return;
   }
   const __nv_bfloat16* ring = p.ring + (long long)b * p.ring_bs;
-  auto fetch = [&](int first) {
-    const int pieces = cw >> 3;
-    for (int i = tid; i < LR_KEYS * pieces; i += LR_THREADS) {
-      const int r = i / pieces, c = (i % pieces) * 8;
+  // rows 4 w .. 4 w + 3 of a tile belong to warp w: no divisions in the copy loop
+  auto fetch = [&](int first, int buf) {
+#pragma unroll
+    for (int x = 0; x < LR_KEYS / 8; ++x) {
+      const int r = warp * (LR_KEYS / 8) + x;
       const bool ok = first + r < k1;
-      cp_async_16(smem_u32(tile + r * L.ldt + c), ring + (long long)(ok ? first + r : k0) * p.cwp + c, ok);
+      const __nv_bfloat16* src = ring + (long long)(ok ? first + r : k0) * p.cwp;
+      __nv_bfloat16* dst = tile + (buf * LR_KEYS + r) * L.ldt;
+      for (int c = lane * 8; c < cw; c += 256) cp_async_16(smem_u32(dst + c), src + c, ok);
     }
+    cp_async_commit();
   };
-  fetch(k0);
+  fetch(k0, 0);
   // absorbed queries (rows of heads that do not exist are zero), rotated parts
   for (int i = tid; i < 16 * (p.rank >> 3); i += LR_THREADS) {
     const int r = i / (p.rank >> 3), c = (i % (p.rank >> 3)) * 8;
@@ -229,45 +251,47 @@ __global__ void __launch_bounds__(LR_THREADS, 2) latent_ring_kernel(const RingAr
     for (int e = 0; e < 4; ++e) acc[i][e] = 0.f;
   float m_[2] = {-INFINITY, -INFINITY}, l_[2] = {0.f, 0.f};  // soft-max state of heads 2 * warp, + 1
   const uint32_t a_addr = smem_u32(sq + (lane & 15) * L.ldt + (lane >> 4) * 8);
-  const uint32_t b_addr = smem_u32(tile + (warp * 8 + (lane & 7)) * L.ldt + (lane >> 3) * 8);
+  const uint32_t b_addr = smem_u32(tile + ((warp & 3) * 8 + (lane & 7)) * L.ldt + (lane >> 3) * 8);
   const uint32_t p_addr = smem_u32(sp + (lane & 15) * (LR_KEYS + 8) + (lane >> 4) * 8);
   const uint32_t v_addr = smem_u32(tile + (lane & 15) * L.ldt + warp * NTW * 8 + (lane >> 4) * 8);
-  for (int first = k0; first < k1; first += LR_KEYS) {
-    cp_async_wait_all();
+  const int steps = cw >> 5, k_mid = ((steps + 1) >> 1) * 32, k_lo = warp < 4 ? 0 : k_mid, k_hi = warp < 4 ? k_mid : cw;
+  int buf = 0;
+  for (int first = k0; first < k1; first += LR_KEYS, buf ^= 1) {
+    if (first + LR_KEYS < k1) {
+      fetch(first + LR_KEYS, buf ^ 1);
+      cp_async_wait<1>();
+    } else {
+      cp_async_wait<0>();
+    }
     __syncthreads();
-    // ---- scores: warp w, keys 8 w .. 8 w + 7 of the tile
+    const uint32_t stage = uint32_t(buf * LR_KEYS * L.ldt * 2);
+    // ---- scores: warps w and w + 4 take keys 8 w .. 8 w + 7 of the tile, each half of the reduction
     {
       float c0[4] = {0.f, 0.f, 0.f, 0.f}, c1[4] = {0.f, 0.f, 0.f, 0.f};
-#pragma unroll 2
-      for (int k = 0; k < cw; k += 32) {
+#pragma unroll 3
+      for (int k = k_lo; k < k_hi; k += 32) {
         uint32_t bb[4], a0[4], a1[4];
-        ldmatrix_x4(b_addr + k * 2, bb);
+        ldmatrix_x4(b_addr + stage + k * 2, bb);
         ldmatrix_x4(a_addr + k * 2, a0);
         ldmatrix_x4(a_addr + k * 2 + 32, a1);
         mma_bf16_16816(c0, a0[0], a0[1], a0[2], a0[3], bb[0], bb[1]);
         mma_bf16_16816(c1, a1[0], a1[1], a1[2], a1[3], bb[2], bb[3]);
       }
-      const int key = warp * 8 + 2 * t;
-      const bool ok0 = first + key < k1, ok1 = first + key + 1 < k1;
-      float* s0 = ss + g * (LR_KEYS + 4) + key;
-      float* s1 = ss + (g + 8) * (LR_KEYS + 4) + key;
-      s0[0] = ok0 ? (c0[0] + c1[0]) * p.scale : -INFINITY;
-      s0[1] = ok1 ? (c0[1] + c1[1]) * p.scale : -INFINITY;
-      s1[0] = ok0 ? (c0[2] + c1[2]) * p.scale : -INFINITY;
-      s1[1] = ok1 ? (c0[3] + c1[3]) * p.scale : -INFINITY;
+      float* s0 = ss + ((warp >> 2) * 16 + g) * (LR_KEYS + 4) + (warp & 3) * 8 + 2 * t;
+      *reinterpret_cast<float2*>(s0) = make_float2(c0[0] + c1[0], c0[1] + c1[1]);
+      *reinterpret_cast<float2*>(s0 + 8 * (LR_KEYS + 4)) = make_float2(c0[2] + c1[2], c0[3] + c1[3]);
     }
     __syncthreads();
-    // ---- soft-max: two heads per warp
+    // ---- soft-max: two heads per warp, one key per lane
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
       const int r = warp * 2 + e;
-      const float x0 = ss[r * (LR_KEYS + 4) + lane], x1 = ss[r * (LR_KEYS + 4) + lane + 32];
-      const float mn = fmaxf(m_[e], warp_max(fmaxf(x0, x1)));  // the tile has at least one key: finite
-      const float al = __expf(m_[e] - mn), p0 = __expf(x0 - mn), p1 = __expf(x1 - mn);
+      const float x = first + lane < k1 ? (ss[r * (LR_KEYS + 4) + lane] + ss[(16 + r) * (LR_KEYS + 4) + lane]) * p.scale : -INFINITY;
+      const float mn = fmaxf(m_[e], warp_max(x));  // the tile has at least one key: finite
+      const float al = __expf(m_[e] - mn), pr = __expf(x - mn);
       m_[e] = mn;
-      l_[e] = l_[e] * al + warp_sum(p0 + p1);
-      sp[r * (LR_KEYS + 8) + lane] = __float2bfloat16(p0);
-      sp[r * (LR_KEYS + 8) + lane + 32] = __float2bfloat16(p1);
+      l_[e] = l_[e] * al + warp_sum(pr);
+      sp[r * (LR_KEYS + 8) + lane] = __float2bfloat16(pr);
       if (lane == 0) sal[r] = al;
     }
     __syncthreads();
@@ -285,13 +309,12 @@ __global__ void __launch_bounds__(LR_THREADS, 2) latent_ring_kernel(const RingAr
 #pragma unroll
       for (int i = 0; i < NTW; i += 2) {
         uint32_t v[4];
-        ldmatrix_x4_trans(v_addr + (k * L.ldt + i * 8) * 2, v);
+        ldmatrix_x4_trans(v_addr + stage + (k * L.ldt + i * 8) * 2, v);
         mma_bf16_16816(acc[i], a[0], a[1], a[2], a[3], v[0], v[1]);
         mma_bf16_16816(acc[i + 1], a[0], a[1], a[2], a[3], v[2], v[3]);
       }
     }
-    __syncthreads();
-    if (first + LR_KEYS < k1) fetch(first + LR_KEYS);
+    __syncthreads();  // the next fetch overwrites this stage's partner, and the scores are written again
   }
 #pragma unroll
   for (int i = 0; i < NTW; ++i) {

@@ -229,7 +229,7 @@ def test_delta_state_and_tail_after_portions(device, dtype):
     for L in (2, 11, 1, 1, 16, 6):
         part = proj[:, at:at + L].contiguous().to(device)
         lengths = torch.full((B,), at, dtype=torch.int32, device=device) if L == 1 else None
-        mixed, rlen, gb = delta_ops.delta_prep(part, s, conv.to(device), rate.to(device), dt.to(device), tail, at, lengths)
+        mixed, rlen, gb = delta_ops.delta_prep(part, s, conv.T.contiguous().to(device), rate.to(device), dt.to(device), tail, at, lengths)
         if L == 1:
             delta_ops.delta_step(mixed, rlen, gb, state, part.view(B, -1)[:, s.g_col:], torch.ones(20, device=device), s, lengths)
         else:
