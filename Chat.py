@@ -2,10 +2,13 @@
 """Interactive chat / batch generation from a checkpoint.
 
     python Chat.py --checkpoint experiments/run/checkpoints/checkpoint_final.pt [--mode standard] [--prompt "..."]
+    python Chat.py --model FOLDER [--token-ids "5 17 3"] [--new-tokens 32]
 
 Loads single-file checkpoints under any of the keys ``model_state_dict | module | state_dict | model`` and infers the
 architecture from the tensor names when no config is stored (reference ``Chat.py:132-298``); generation uses the KV-cache
-engine.  Slash commands: /mode <name>, /temp <x>, /tokens <n>, /reset, /stats, /quit (reference ``Chat.py:671-707``)."""
+engine.  ``--model`` takes a folder with ``config.json`` and ``model.safetensors``; its ``architecture`` selects the model class
+(``models/registry.py``).  ``--token-ids`` continues a sequence of token ids and prints the new ids (models without a tokenizer).
+Slash commands: /mode <name>, /temp <x>, /tokens <n>, /reset, /stats, /quit (reference ``Chat.py:671-707``)."""
 from __future__ import annotations
 
 import argparse
@@ -19,7 +22,7 @@ import torch  # noqa: E402
 from adaptivetrainingsystem_b200.config import ModelConfig  # noqa: E402
 from adaptivetrainingsystem_b200.data.tokenizer import ConversationTokenizer  # noqa: E402
 from adaptivetrainingsystem_b200.inference import GENERATION_MODES, GenerationEngine, SamplingParams  # noqa: E402
-from adaptivetrainingsystem_b200.models import DeepSeekTransformer  # noqa: E402
+from adaptivetrainingsystem_b200.models import DeepSeekTransformer, load_model  # noqa: E402
 from adaptivetrainingsystem_b200.training.checkpoint import MODEL_KEYS  # noqa: E402
 
 
@@ -53,14 +56,21 @@ def load_checkpoint_smart(path: str):
 
 
 class ChatInterface:
-    def __init__(self, checkpoint: str, device: str = "auto", mode: str = "standard", quantize: str = None, quantized_file: str = None):
+    def __init__(self, checkpoint: str = None, device: str = "auto", mode: str = "standard", quantize: str = None, quantized_file: str = None,
+                 model_folder: str = None):
         self.device = torch.device("cuda" if (device == "auto" and torch.cuda.is_available()) else ("cpu" if device == "auto" else device))
-        sd, cfg = load_checkpoint_smart(checkpoint)
-        cfg.gradient_checkpointing = False
         dtype = torch.bfloat16 if self.device.type == "cuda" else torch.float32
-        self.model = DeepSeekTransformer(cfg)
-        self.model.load_state_dict({k: v for k, v in sd.items()}, strict=False)
-        self.model = self.model.to(self.device, dtype).eval()
+        if model_folder:
+            self.model = load_model(model_folder, dtype, self.device)
+            cfg = self.model.config
+        else:
+            sd, cfg = load_checkpoint_smart(checkpoint)
+            cfg.gradient_checkpointing = False
+            self.model = DeepSeekTransformer(cfg)
+            self.model.load_state_dict({k: v for k, v in sd.items()}, strict=False)
+            self.model = self.model.to(self.device, dtype).eval()
+        if quantize and not isinstance(self.model, DeepSeekTransformer):
+            raise SystemExit(f"--quantize: not built for {type(self.model).__name__}")
         if quantize:
             if self.device.type != "cuda" and quantize != "int4":
                 raise SystemExit("--quantize fp8 / int8 needs a GPU: those paths run on the tensor-core GEMM")
@@ -105,6 +115,13 @@ class ChatInterface:
         batcher = ContinuousBatcher(self.engine, max_batch=min(max_batch, len(prompts)), max_len=rows, params=self.params)
         return [self.tokenizer.decode(t) for t in batcher.run(prompts)]
 
+    def continue_ids(self, ids, new_tokens: int):
+        """The ids that follow ``ids`` under the current sampling parameters (stop tokens of the tokenizer do not apply)."""
+        from dataclasses import replace
+        prompt = torch.tensor([list(ids)], dtype=torch.long, device=self.device)
+        res = self.engine.generate(prompt, replace(self.params, max_new_tokens=new_tokens, stop_token_ids=()))
+        return res["tokens"][0].tolist()
+
     def command(self, line: str) -> bool:
         cmd, *rest = line[1:].split()
         if cmd in ("quit", "exit"):
@@ -142,7 +159,11 @@ class ChatInterface:
 
 if __name__ == "__main__":
     ap = argparse.ArgumentParser()
-    ap.add_argument("--checkpoint", required=True)
+    src = ap.add_mutually_exclusive_group(required=True)
+    src.add_argument("--checkpoint", default=None)
+    src.add_argument("--model", default=None, help="folder with config.json and model.safetensors")
+    ap.add_argument("--token-ids", default=None, help="continue these token ids (separated by blanks or commas) and print the new ids")
+    ap.add_argument("--new-tokens", type=int, default=32, help="with --token-ids: how many")
     ap.add_argument("--mode", default="standard", choices=list(GENERATION_MODES))
     ap.add_argument("--prompt", default=None)
     ap.add_argument("--device", default="auto")
@@ -152,8 +173,10 @@ if __name__ == "__main__":
     ap.add_argument("--prompts-file", default=None, help="one prompt per line, answered together by continuous batching")
     ap.add_argument("--max-batch", type=int, default=16)
     a = ap.parse_args()
-    chat = ChatInterface(a.checkpoint, a.device, a.mode, a.quantize, a.quantized_file)
-    if a.prompts_file:
+    chat = ChatInterface(a.checkpoint, a.device, a.mode, a.quantize, a.quantized_file, a.model)
+    if a.token_ids:
+        print(" ".join(map(str, chat.continue_ids([int(t) for t in a.token_ids.replace(",", " ").split()], a.new_tokens))))
+    elif a.prompts_file:
         with open(a.prompts_file) as f:
             lines = [l.strip() for l in f if l.strip()]
         for q, ans in zip(lines, chat.respond_many(lines, a.max_batch)):

@@ -11,7 +11,7 @@
 //   group, u_i = beta_i (v_i - G_i S^T k_i - sum_{j < i} D_ij (k_j . k_i) u_j), D_ij = g_{j+1} .. g_i, G_i = g_1 .. g_i, a unit lower
 //   triangular system whose 8 x 8 inverse does not depend on the value column; delta_pairs computes it (and the read-out
 //   coefficients) for all groups in parallel, so that the sequential kernel only does three products with the state per token.
-//   Columns of S are independent: sixteen lanes share eight columns, everything in fp32 with packed fma.f32x2.
+//   Columns of S are independent: sixteen lanes share four columns, everything in fp32 with packed fma.f32x2.
 // * delta_output: output norm over vdim, weight, silu gate.
 // * delta_step: one decoded token per sequence: state read once and written once, output norm and gate in the same launch.
 //
@@ -121,67 +121,66 @@ __global__ void __launch_bounds__(PV_THREADS, 4) delta_prep_vec_kernel(const Del
   const T* in = static_cast<const T*>(p.proj) + (long long)b * p.L * p.ld + c;
   const T* tail = static_cast<const T*>(p.tail) + (long long)b * p.tail_bs + c;
   T* out = static_cast<T*>(p.mixed) + (long long)b * p.L * p.ldm + c;
-  float w[TAPS][8], x[TAPS][8];  // x[j]: the input j tokens back (x[0] = current)
+  constexpr int PB = 4;
+  float w[TAPS][8], x[TAPS - 1 + PB][8];
 #pragma unroll
-  for (int j = 0; j < TAPS; ++j) Typed<float>::load8(p.conv + (long long)(TAPS - 1 - j) * p.C + c, w[j]);
+  for (int j = 0; j < TAPS; ++j) Typed<float>::load8(p.conv + (long long)j * p.C + c, w[j]);
   const int pos0 = p.lengths ? p.lengths[b] : p.pos0;
 #pragma unroll
-  for (int j = 1; j < TAPS; ++j) {
-    const int t = t0 - j;
-    if (t >= 0) Typed<T>::load8(in + (long long)t * p.ld, x[j - 1]);
-    else if (pos0 > 0) Typed<T>::load8(tail + (long long)(TAPS - 1 + t) * p.C, x[j - 1]);
+  for (int j = 0; j < TAPS - 1; ++j) {
+    const int t = t0 - (TAPS - 1) + j;
+    if (t >= 0) Typed<T>::load8(in + (long long)t * p.ld, x[j]);
+    else if (pos0 > 0) Typed<T>::load8(tail + (long long)(TAPS - 1 + t) * p.C, x[j]);
     else
 #pragma unroll
-      for (int e = 0; e < 8; ++e) x[j - 1][e] = 0.f;
+      for (int e = 0; e < 8; ++e) x[j][e] = 0.f;
   }
   const int lanes = p.dim >> 3, kd = p.KH * p.dim;
   const bool qk = live && c < 2 * kd, warp_qk = __any_sync(0xffffffffu, qk);
-  // tokens come in batches of PB whose loads are issued one batch ahead
-  constexpr int PB = 4;
+  const int head = piece / lanes;
+  // tokens come in batches of PB whose loads are issued one batch ahead; x[0 .. TAPS - 2] is the history, oldest first
   typename Typed<T>::Raw8 nx[PB];
 #pragma unroll
   for (int u = 0; u < PB; ++u) nx[u] = Typed<T>::raw8(in + (long long)min(t0 + u, t1 - 1) * p.ld);
   for (int tb0 = t0; tb0 < t1; tb0 += PB) {
-    typename Typed<T>::Raw8 cur[PB];
 #pragma unroll
-    for (int u = 0; u < PB; ++u) cur[u] = nx[u];
+    for (int u = 0; u < PB; ++u) Typed<T>::unpack8(nx[u], x[TAPS - 1 + u]);
     if (tb0 + PB < t1)
 #pragma unroll
       for (int u = 0; u < PB; ++u) nx[u] = Typed<T>::raw8(in + (long long)min(tb0 + PB + u, t1 - 1) * p.ld);
 #pragma unroll
     for (int u = 0; u < PB; ++u) {
       const int t = tb0 + u;
-      if (t >= t1) break;
-#pragma unroll
-      for (int j = TAPS - 1; j > 0; --j)
-#pragma unroll
-        for (int e = 0; e < 8; ++e) x[j][e] = x[j - 1][e];
-      Typed<T>::unpack8(cur[u], x[0]);
       float y[8], ss = 0.f;
 #pragma unroll
       for (int e = 0; e < 8; ++e) {
-        float acc = 0.f;
+        float acc = x[u][e] * w[0][e];
 #pragma unroll
-        for (int j = 0; j < TAPS; ++j) acc += x[j][e] * w[j][e];
+        for (int j = 1; j < TAPS; ++j) acc += x[u + j][e] * w[j][e];
         y[e] = acc * Typed<T>::sigmoid_(acc);
       }
-      Typed<T>::round8(y);
-      if (live) Typed<T>::store8(out + (long long)t * p.ldm, y);
+      const typename Typed<T>::Raw8 packed = Typed<T>::pack8(y);
+      if (live && t < t1) Typed<T>::store_raw8(out + (long long)t * p.ldm, packed);
       if (warp_qk) {
+        Typed<T>::unpack8(packed, y);
 #pragma unroll
         for (int e = 0; e < 8; ++e) ss += y[e] * y[e];
         for (int off = lanes >> 1; off > 0; off >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, off);
-        if (qk && (piece & (lanes - 1)) == 0) {
-          const int head = piece / lanes;
+        if (qk && t < t1 && (piece & (lanes - 1)) == 0)
           p.rlen[((long long)b * p.L + t) * 2 * p.KH + head] = (head < p.KH ? 1.f / sqrtf(float(p.dim)) : 1.f) / sqrtf(ss + 1e-6f);
-        }
       }
     }
+    // the batch's last tokens are the next history (in decoding, the one token of the batch sits at x[TAPS - 1])
+    if (tb0 + PB < t1)
+#pragma unroll
+      for (int j = 0; j < TAPS - 1; ++j)
+#pragma unroll
+        for (int e = 0; e < 8; ++e) x[j][e] = x[PB + j][e];
   }
   if (p.lengths && live && !(p.active && !p.active[b])) {  // decoding: this thread's channels move on by the token
     T* tw = static_cast<T*>(p.tail) + (long long)b * p.tail_bs + c;
 #pragma unroll
-    for (int j = 0; j < TAPS - 1; ++j) Typed<T>::store8(tw + (long long)(TAPS - 2 - j) * p.C, x[j]);
+    for (int j = 0; j < TAPS - 1; ++j) Typed<T>::store8(tw + (long long)j * p.C, x[j + 1]);
   }
 }
 
@@ -360,17 +359,47 @@ __device__ __forceinline__ float keep_add(float lo, float hi, int lane, int s) {
   return (up ? hi : lo) + __shfl_xor_sync(0xffffffffu, up ? lo : hi, s);
 }
 
+// A lane's EPL values of a k or q row in shared memory: pieces of up to eight consecutive elements, sixteen lanes side by side.
+template <typename T, int EPL>
+struct RowPiece {
+  static constexpr int W = EPL < 8 ? EPL : 8;
+  static __device__ __forceinline__ int index(int pair, int l16) {  // first state row of pair `pair` (two rows) of lane l16
+    return ((2 * pair) / W * 16 + l16) * W + (2 * pair) % W;
+  }
+  static __device__ __forceinline__ void load(const T* row, int l16, float2 (&k)[EPL / 2]) {
+#pragma unroll
+    for (int c = 0; c < EPL / W; ++c) {
+      const T* p = row + (c * 16 + l16) * W;
+      if constexpr (sizeof(T) == 2) {
+        uint32_t u[W / 2];
+        if constexpr (W == 8) *reinterpret_cast<uint4*>(u) = *reinterpret_cast<const uint4*>(p);
+        else *reinterpret_cast<uint2*>(u) = *reinterpret_cast<const uint2*>(p);
+#pragma unroll
+        for (int x = 0; x < W / 2; ++x) k[c * W / 2 + x] = unpack_bf16x2(u[x]);
+      } else {
+#pragma unroll
+        for (int x = 0; x < W / 4; ++x) {
+          const float4 v = *reinterpret_cast<const float4*>(p + 4 * x);
+          k[c * W / 2 + 2 * x] = make_float2(v.x, v.y);
+          k[c * W / 2 + 2 * x + 1] = make_float2(v.z, v.w);
+        }
+      }
+    }
+  }
+};
+
 // Sixteen lanes share CPL value columns: lane l holds EPL state rows (dim <= 16 * EPL) of each.  CTA = 4 warps of 2 lane groups ->
-// 8 * CPL columns of one head.  With the state spread over sixteen lanes, a row of k or q read from shared memory serves CPL columns,
-// which keeps the load pipe below the FMA pipe.  The next group's q, k, v and constants are requested before this group's products
+// 8 * CPL columns of one head.  k and q rows stay in the element type in shared memory: with the state spread over sixteen lanes and
+// 16-byte reads of eight bf16 values the load pipe stays below the FMA pipe.  The next group's q, k, v and constants are requested before this group's products
 // and stored to the other half of shared memory after them.  After a product, lane l holds token l % 8, columns (l / 8) * CPL / 2 ...
-template <typename T, int EPL, int CPL>
-__global__ void __launch_bounds__(128, 2) delta_scan_kernel(const ScanArgs p) {
+template <typename T, int EPL, int CPL, int OCC>
+__global__ void __launch_bounds__(128, OCC) delta_scan_kernel(const ScanArgs p) {
   pdl_prologue();
   constexpr int DK = 16 * EPL, HC = CPL / 2;
   constexpr int VEC = 16 / int(sizeof(T));             // elements per 16-byte piece
   constexpr int NP = (2 * DC * DK / VEC + 127) / 128;  // pieces of q and k per thread and group
-  __shared__ __align__(16) float s_kq[2][2][DC][DK];   // [buffer][k, q]
+  using Row = RowPiece<T, EPL>;
+  __shared__ __align__(16) T s_kq[2][2][DC][DK];       // [buffer][k, q]
   __shared__ __align__(16) float s_c[2][CO];
   __shared__ __align__(16) float s_u[8][3][DC][CPL];   // [lane group][right-hand side, u, D_Cj u_j / |k_j|]
   const int tid = threadIdx.x, lane = tid & 31, l16 = lane & 15, grp16 = tid >> 4, tok = l16 & 7, half = l16 >> 3;
@@ -382,7 +411,7 @@ __global__ void __launch_bounds__(128, 2) delta_scan_kernel(const ScanArgs p) {
   for (int c = 0; c < CPL; ++c)
 #pragma unroll
     for (int e = 0; e < EPL / 2; ++e) {
-      const int d = ((e >> 1) * 16 + l16) * 4 + (e & 1) * 2;
+      const int d = Row::index(e, l16);
       const bool ok = !p.fresh && col0 + c < p.vdim;
       S[c][e].x = (ok && d < p.dim) ? st[(long long)d * p.vdim + col0 + c] : 0.f;
       S[c][e].y = (ok && d + 1 < p.dim) ? st[(long long)(d + 1) * p.vdim + col0 + c] : 0.f;
@@ -418,13 +447,7 @@ __global__ void __launch_bounds__(128, 2) delta_scan_kernel(const ScanArgs p) {
 #pragma unroll
     for (int u = 0; u < NP; ++u) {
       if ((u * 128 + tid) * VEC >= 2 * DC * DK) continue;
-      float* dst = &s_kq[buf][0][0][0] + (u * 128 + tid) * VEC;
-      float f[8];
-      const T* e = reinterpret_cast<const T*>(&piece[u]);
-#pragma unroll
-      for (int x = 0; x < VEC; ++x) f[x] = Typed<T>::load(e + x);
-#pragma unroll
-      for (int x = 0; x < VEC; x += 4) *reinterpret_cast<float4*>(dst + x) = make_float4(f[x], f[x + 1], f[x + 2], f[x + 3]);
+      *reinterpret_cast<uint4*>(&s_kq[buf][0][0][0] + (u * 128 + tid) * VEC) = piece[u];
     }
     if (tid < CO / 4) *reinterpret_cast<float4*>(&s_c[buf][tid * 4]) = cpiece;
   };
@@ -443,15 +466,12 @@ __global__ void __launch_bounds__(128, 2) delta_scan_kernel(const ScanArgs p) {
           float2 a[CPL];
 #pragma unroll
           for (int c = 0; c < CPL; ++c) a[c] = make_float2(0.f, 0.f);
+          float2 k[EPL / 2];
+          Row::load(s_kq[buf][which][i], l16, k);
 #pragma unroll
-          for (int e = 0; e < EPL / 4; ++e) {
-            const float4 k4 = *reinterpret_cast<const float4*>(&s_kq[buf][which][i][(e * 16 + l16) * 4]);
+          for (int e = 0; e < EPL / 2; ++e)
 #pragma unroll
-            for (int c = 0; c < CPL; ++c) {
-              a[c] = fma2(S[c][2 * e], make_float2(k4.x, k4.y), a[c]);
-              a[c] = fma2(S[c][2 * e + 1], make_float2(k4.z, k4.w), a[c]);
-            }
-          }
+            for (int c = 0; c < CPL; ++c) a[c] = fma2(S[c][e], k[e], a[c]);
 #pragma unroll
           for (int c = 0; c < CPL; ++c) r8[x][c] = a[c].x + a[c].y;
         }
@@ -529,16 +549,12 @@ __global__ void __launch_bounds__(128, 2) delta_scan_kernel(const ScanArgs p) {
         const float4 q = *reinterpret_cast<const float4*>(&s_u[grp16][2][j][c]);
         w[c] = q.x; w[c + 1] = q.y; w[c + 2] = q.z; w[c + 3] = q.w;
       }
+      float2 k[EPL / 2];
+      Row::load(s_kq[buf][0][j], l16, k);
 #pragma unroll
-      for (int e = 0; e < EPL / 4; ++e) {
-        const float4 k4 = *reinterpret_cast<const float4*>(&s_kq[buf][0][j][(e * 16 + l16) * 4]);
+      for (int e = 0; e < EPL / 2; ++e)
 #pragma unroll
-        for (int c = 0; c < CPL; ++c) {
-          const float2 uu = make_float2(w[c], w[c]);
-          S[c][2 * e] = fma2(make_float2(k4.x, k4.y), uu, S[c][2 * e]);
-          S[c][2 * e + 1] = fma2(make_float2(k4.z, k4.w), uu, S[c][2 * e + 1]);
-        }
-      }
+        for (int c = 0; c < CPL; ++c) S[c][e] = fma2(k[e], make_float2(w[c], w[c]), S[c][e]);
       if (j & 1) pace();
     }
     if (grp + 1 < p.groups) deposit(buf ^ 1);  // the other half was last read one group ago
@@ -549,7 +565,7 @@ __global__ void __launch_bounds__(128, 2) delta_scan_kernel(const ScanArgs p) {
     if (col0 + c >= p.vdim) continue;
 #pragma unroll
     for (int e = 0; e < EPL / 2; ++e) {
-      const int d = ((e >> 1) * 16 + l16) * 4 + (e & 1) * 2;
+      const int d = Row::index(e, l16);
       if (d < p.dim) st[(long long)d * p.vdim + col0 + c] = S[c][e].x;
       if (d + 1 < p.dim) st[(long long)(d + 1) * p.vdim + col0 + c] = S[c][e].y;
     }
@@ -816,9 +832,9 @@ static int launch_scan(const ScanArgs& p, cudaStream_t s) {
     launch_pdl(delta_pairs_kernel<T, false>, pgrid, dim3(128), 0, s, p);
   }
   auto grid = [&](int cpl) { return dim3((p.vdim + 8 * cpl - 1) / (8 * cpl), p.H, p.B); };
-  if (p.dim <= 64) launch_pdl(delta_scan_kernel<T, 4, 8>, grid(8), dim3(128), 0, s, p);
-  else if (p.dim <= 128) launch_pdl(delta_scan_kernel<T, 8, 8>, grid(8), dim3(128), 0, s, p);
-  else if (p.dim <= 256) launch_pdl(delta_scan_kernel<T, 16, 4>, grid(4), dim3(128), 0, s, p);
+  if (p.dim <= 64) launch_pdl(delta_scan_kernel<T, 4, 4, 5>, grid(4), dim3(128), 0, s, p);
+  else if (p.dim <= 128) launch_pdl(delta_scan_kernel<T, 8, 4, 5>, grid(4), dim3(128), 0, s, p);
+  else if (p.dim <= 256) launch_pdl(delta_scan_kernel<T, 16, 4, 3>, grid(4), dim3(128), 0, s, p);
   else return 1006;
   return int(cudaGetLastError());
 }

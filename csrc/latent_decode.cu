@@ -63,7 +63,7 @@ __global__ void __launch_bounds__(WARPS * 32) latent_head_mm_kernel(const HeadMm
   const int h = blockIdx.y, b0 = blockIdx.z * 16, nb = min(16, p.B - b0);
   const int n0 = (blockIdx.x * WARPS + warp) * NT * 8;
   // the first PRE steps of this lane's weights, requested before the inputs are gathered
-  constexpr int PRE = 4;
+  constexpr int PRE = 16 / NT;
   const __nv_bfloat16* w = p.w + h * p.w_hs + 8 * t;
   uint4 pre[PRE][NT];
 #pragma unroll
@@ -84,21 +84,29 @@ __global__ void __launch_bounds__(WARPS * 32) latent_head_mm_kernel(const HeadMm
       s_f[j][lane + 32] = f1 * inv;
     }
     __syncthreads();
+    // four rows of a column quad at a time: with the chunk loop unrolled, up to eight loads are in flight per thread
     const int quads = p.K >> 2;
-    for (int i = tid; i < 16 * quads; i += WARPS * 32) {
-      const int j = i / quads, r = (i % quads) * 4;
-      float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+    const long long row = (long long)p.H * p.n_chunks * p.K;  // elements between sequences
+    for (int i = tid; i < 4 * quads; i += WARPS * 32) {
+      const int j = (i / quads) * 4, r = (i % quads) * 4;
+      float4 a[4];
+#pragma unroll
+      for (int u = 0; u < 4; ++u) a[u] = make_float4(0.f, 0.f, 0.f, 0.f);
       if (j < nb) {
-        const float* po = p.part_o + (((long long)(b0 + j) * p.H + h) * p.n_chunks) * p.K + r;
-#pragma unroll 4
-        for (int c = 0; c < p.n_chunks; ++c) {
-          const float f = s_f[j][c];
-          // (a chunk beyond a short sequence was not written: its factor is zero and its values are not used)
-          const float4 v = f > 0.f ? *reinterpret_cast<const float4*>(po + (long long)c * p.K) : make_float4(0.f, 0.f, 0.f, 0.f);
-          a.x += f * v.x; a.y += f * v.y; a.z += f * v.z; a.w += f * v.w;
-        }
+        const float* po = p.part_o + ((long long)(b0 + j) * p.H + h) * p.n_chunks * p.K + r;
+#pragma unroll 2
+        for (int c = 0; c < p.n_chunks; ++c)
+#pragma unroll
+          for (int u = 0; u < 4; ++u) {
+            const float f = j + u < nb ? s_f[j + u][c] : 0.f;
+            // (a chunk beyond a short sequence was not written: its factor is zero and its values are not used)
+            const float4 v = f > 0.f ? *reinterpret_cast<const float4*>(po + u * row + (long long)c * p.K) : make_float4(0.f, 0.f, 0.f, 0.f);
+            a[u].x += f * v.x; a[u].y += f * v.y; a[u].z += f * v.z; a[u].w += f * v.w;
+          }
       }
-      *reinterpret_cast<uint2*>(sx + j * ldx + r) = make_uint2(pack_bf16x2(a.x, a.y), pack_bf16x2(a.z, a.w));
+#pragma unroll
+      for (int u = 0; u < 4; ++u)
+        *reinterpret_cast<uint2*>(sx + (j + u) * ldx + r) = make_uint2(pack_bf16x2(a[u].x, a[u].y), pack_bf16x2(a[u].z, a[u].w));
     }
   } else {
     const int pieces = p.K >> 3;
@@ -181,7 +189,7 @@ struct RingSmem {
     ldt = cw + 8;
     qa = 2 * LR_KEYS * ldt * 2;
     s = qa + 16 * ldt * 2;
-    pr = s + 2 * 16 * (LR_KEYS + 4) * 4;
+    pr = s + 4 * 16 * (LR_KEYS + 4) * 4;
     al = pr + 16 * (LR_KEYS + 8) * 2;
     total = al + 16 * 4;
   }
@@ -196,7 +204,7 @@ __global__ void __launch_bounds__(LR_THREADS, 2) latent_ring_kernel(const RingAr
   const RingSmem L(cw);
   __nv_bfloat16* tile = reinterpret_cast<__nv_bfloat16*>(smem_raw);
   __nv_bfloat16* sq = reinterpret_cast<__nv_bfloat16*>(smem_raw + L.qa);
-  float* ss = reinterpret_cast<float*>(smem_raw + L.s);                  // [half of the reduction][16][LR_KEYS + 4]
+  float* ss = reinterpret_cast<float*>(smem_raw + L.s);                  // [quarter of the reduction][16][LR_KEYS + 4]
   __nv_bfloat16* sp = reinterpret_cast<__nv_bfloat16*>(smem_raw + L.pr);  // [16][LR_KEYS + 8]
   float* sal = reinterpret_cast<float*>(smem_raw + L.al);                // [16]
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
@@ -250,11 +258,17 @@ __global__ void __launch_bounds__(LR_THREADS, 2) latent_ring_kernel(const RingAr
 #pragma unroll
     for (int e = 0; e < 4; ++e) acc[i][e] = 0.f;
   float m_[2] = {-INFINITY, -INFINITY}, l_[2] = {0.f, 0.f};  // soft-max state of heads 2 * warp, + 1
-  const uint32_t a_addr = smem_u32(sq + (lane & 15) * L.ldt + (lane >> 4) * 8);
-  const uint32_t b_addr = smem_u32(tile + ((warp & 3) * 8 + (lane & 7)) * L.ldt + (lane >> 3) * 8);
+  // score phase: warp w takes keys 16 (w & 1) .. + 15 of a tile and a quarter of the reduction, whose query fragments stay in registers
+  const int steps = cw >> 4, per = (steps + 3) >> 2, q_lo = (warp >> 1) * per, q_n = max(0, min(per, steps - q_lo));
+  __syncthreads();  // queries are complete
+  uint32_t aq[NTW + 2][4];
+#pragma unroll
+  for (int x = 0; x < NTW + 2; ++x)
+    if (x < q_n) ldmatrix_x4(smem_u32(sq + (lane & 15) * L.ldt + (q_lo + x) * 16 + (lane >> 4) * 8), aq[x]);
+  // (matrices: keys 0..7 and 8..15, each with the two halves of the 16 reduction columns)
+  const uint32_t b_addr = smem_u32(tile + ((warp & 1) * 16 + (lane >> 4) * 8 + (lane & 7)) * L.ldt + q_lo * 16 + ((lane >> 3) & 1) * 8);
   const uint32_t p_addr = smem_u32(sp + (lane & 15) * (LR_KEYS + 8) + (lane >> 4) * 8);
   const uint32_t v_addr = smem_u32(tile + (lane & 15) * L.ldt + warp * NTW * 8 + (lane >> 4) * 8);
-  const int steps = cw >> 5, k_mid = ((steps + 1) >> 1) * 32, k_lo = warp < 4 ? 0 : k_mid, k_hi = warp < 4 ? k_mid : cw;
   int buf = 0;
   for (int first = k0; first < k1; first += LR_KEYS, buf ^= 1) {
     if (first + LR_KEYS < k1) {
@@ -265,28 +279,30 @@ __global__ void __launch_bounds__(LR_THREADS, 2) latent_ring_kernel(const RingAr
     }
     __syncthreads();
     const uint32_t stage = uint32_t(buf * LR_KEYS * L.ldt * 2);
-    // ---- scores: warps w and w + 4 take keys 8 w .. 8 w + 7 of the tile, each half of the reduction
+    // ---- scores
     {
-      float c0[4] = {0.f, 0.f, 0.f, 0.f}, c1[4] = {0.f, 0.f, 0.f, 0.f};
-#pragma unroll 3
-      for (int k = k_lo; k < k_hi; k += 32) {
-        uint32_t bb[4], a0[4], a1[4];
-        ldmatrix_x4(b_addr + stage + k * 2, bb);
-        ldmatrix_x4(a_addr + k * 2, a0);
-        ldmatrix_x4(a_addr + k * 2 + 32, a1);
-        mma_bf16_16816(c0, a0[0], a0[1], a0[2], a0[3], bb[0], bb[1]);
-        mma_bf16_16816(c1, a1[0], a1[1], a1[2], a1[3], bb[2], bb[3]);
-      }
-      float* s0 = ss + ((warp >> 2) * 16 + g) * (LR_KEYS + 4) + (warp & 3) * 8 + 2 * t;
-      *reinterpret_cast<float2*>(s0) = make_float2(c0[0] + c1[0], c0[1] + c1[1]);
-      *reinterpret_cast<float2*>(s0 + 8 * (LR_KEYS + 4)) = make_float2(c0[2] + c1[2], c0[3] + c1[3]);
+      float c0[4] = {0.f, 0.f, 0.f, 0.f}, c1[4] = {0.f, 0.f, 0.f, 0.f};  // keys 0..7 / 8..15 of the warp's sixteen
+#pragma unroll
+      for (int x = 0; x < NTW + 2; ++x)
+        if (x < q_n) {
+          uint32_t bb[4];
+          ldmatrix_x4(b_addr + stage + x * 32, bb);
+          mma_bf16_16816(c0, aq[x][0], aq[x][1], aq[x][2], aq[x][3], bb[0], bb[1]);
+          mma_bf16_16816(c1, aq[x][0], aq[x][1], aq[x][2], aq[x][3], bb[2], bb[3]);
+        }
+      float* s0 = ss + ((warp >> 1) * 16 + g) * (LR_KEYS + 4) + (warp & 1) * 16 + 2 * t;
+      *reinterpret_cast<float2*>(s0) = make_float2(c0[0], c0[1]);
+      *reinterpret_cast<float2*>(s0 + 8) = make_float2(c1[0], c1[1]);
+      *reinterpret_cast<float2*>(s0 + 8 * (LR_KEYS + 4)) = make_float2(c0[2], c0[3]);
+      *reinterpret_cast<float2*>(s0 + 8 * (LR_KEYS + 4) + 8) = make_float2(c1[2], c1[3]);
     }
     __syncthreads();
     // ---- soft-max: two heads per warp, one key per lane
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
       const int r = warp * 2 + e;
-      const float x = first + lane < k1 ? (ss[r * (LR_KEYS + 4) + lane] + ss[(16 + r) * (LR_KEYS + 4) + lane]) * p.scale : -INFINITY;
+      const float x = first + lane < k1 ? ((ss[r * (LR_KEYS + 4) + lane] + ss[(16 + r) * (LR_KEYS + 4) + lane]) +
+                                             (ss[(32 + r) * (LR_KEYS + 4) + lane] + ss[(48 + r) * (LR_KEYS + 4) + lane])) * p.scale : -INFINITY;
       const float mn = fmaxf(m_[e], warp_max(x));  // the tile has at least one key: finite
       const float al = __expf(m_[e] - mn), pr = __expf(x - mn);
       m_[e] = mn;

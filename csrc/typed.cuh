@@ -12,7 +12,7 @@ template <> struct Typed<float> {
   static __device__ __forceinline__ void store(float* p, float v) { *p = v; }
   static __device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
   static __device__ __forceinline__ void store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
-  // eight values, 16-byte aligned; round8: to what the type can hold
+  // eight values, 16-byte aligned; Raw8: as they lie in memory
   static __device__ __forceinline__ void load8(const float* p, float (&v)[8]) {
     *reinterpret_cast<float4*>(v) = *reinterpret_cast<const float4*>(p);
     *reinterpret_cast<float4*>(v + 4) = *reinterpret_cast<const float4*>(p + 4);
@@ -23,11 +23,15 @@ template <> struct Typed<float> {
     v[0] = r.a.x; v[1] = r.a.y; v[2] = r.a.z; v[3] = r.a.w;
     v[4] = r.b.x; v[5] = r.b.y; v[6] = r.b.z; v[7] = r.b.w;
   }
+  static __device__ __forceinline__ Raw8 pack8(const float (&v)[8]) { return {make_float4(v[0], v[1], v[2], v[3]), make_float4(v[4], v[5], v[6], v[7])}; }
+  static __device__ __forceinline__ void store_raw8(float* p, const Raw8& r) {
+    *reinterpret_cast<float4*>(p) = r.a;
+    *reinterpret_cast<float4*>(p + 4) = r.b;
+  }
   static __device__ __forceinline__ void store8(float* p, const float (&v)[8]) {
     *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
     *reinterpret_cast<float4*>(p + 4) = make_float4(v[4], v[5], v[6], v[7]);
   }
-  static __device__ __forceinline__ void round8(float (&)[8]) {}
   static __device__ __forceinline__ float exp_(float x) { return expf(x); }
   static __device__ __forceinline__ float tanh_(float x) { return tanhf(x); }
   static __device__ __forceinline__ float sigmoid_(float x) { return 1.f / (1.f + expf(-x)); }
@@ -50,13 +54,11 @@ template <> struct Typed<__nv_bfloat16> {
     const float2 a = unpack_bf16x2(u.x), b = unpack_bf16x2(u.y), c = unpack_bf16x2(u.z), d = unpack_bf16x2(u.w);
     v[0] = a.x; v[1] = a.y; v[2] = b.x; v[3] = b.y; v[4] = c.x; v[5] = c.y; v[6] = d.x; v[7] = d.y;
   }
-  static __device__ __forceinline__ void store8(__nv_bfloat16* p, const float (&v)[8]) {
-    *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]), pack_bf16x2(v[4], v[5]), pack_bf16x2(v[6], v[7]));
+  static __device__ __forceinline__ Raw8 pack8(const float (&v)[8]) {
+    return make_uint4(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]), pack_bf16x2(v[4], v[5]), pack_bf16x2(v[6], v[7]));
   }
-  static __device__ __forceinline__ void round8(float (&v)[8]) {
-#pragma unroll
-    for (int e = 0; e < 8; ++e) v[e] = __bfloat162float(__float2bfloat16(v[e]));
-  }
+  static __device__ __forceinline__ void store_raw8(__nv_bfloat16* p, const Raw8& r) { *reinterpret_cast<uint4*>(p) = r; }
+  static __device__ __forceinline__ void store8(__nv_bfloat16* p, const float (&v)[8]) { store_raw8(p, pack8(v)); }
   static __device__ __forceinline__ float exp_(float x) { return __expf(x); }
   static __device__ __forceinline__ float tanh_(float x) { return tanh_fast(x); }
   static __device__ __forceinline__ float sigmoid_(float x) { return __fdividef(1.f, 1.f + __expf(-x)); }

@@ -448,6 +448,20 @@ def test_trace_program(tmp_path):
     assert not (tmp_path / "1.f32").exists()
 
 
+@pytest.mark.parametrize("device", ["cpu", pytest.param("cuda", marks=gpu)])
+def test_command_line_continues_token_ids(device, tmp_path):
+    import Chat
+    cfg = mixed_config()
+    W = O.random_weights(cfg, seed=2)
+    O.save_model(str(tmp_path), cfg, W)
+    chat = Chat.ChatInterface(model_folder=str(tmp_path), device=device, mode="greedy")
+    prompt = tokens(9)
+    got, want = chat.continue_ids(prompt, 6), greedy_oracle(cfg, W, prompt, 6)
+    assert len(got) == 6 and (device != "cpu" or got == want)
+    with pytest.raises(SystemExit, match="quantize"):
+        Chat.ChatInterface(model_folder=str(tmp_path), device=device, quantize="int4")
+
+
 # ------------------------------------------------------------------------------------------------ configuration, folders
 def test_configuration_round_trip_and_errors(tmp_path):
     d = mixed_config()
