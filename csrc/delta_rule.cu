@@ -11,7 +11,7 @@
 //   group, u_i = beta_i (v_i - G_i S^T k_i - sum_{j < i} D_ij (k_j . k_i) u_j), D_ij = g_{j+1} .. g_i, G_i = g_1 .. g_i, a unit lower
 //   triangular system whose 8 x 8 inverse does not depend on the value column; delta_pairs computes it (and the read-out
 //   coefficients) for all groups in parallel, so that the sequential kernel only does three products with the state per token.
-//   Columns of S are independent: sixteen lanes share four columns, everything in fp32 with packed fma.f32x2.
+//   Columns of S are independent: sixteen lanes share eight columns, everything in fp32 with packed fma.f32x2.
 // * delta_output: output norm over vdim, weight, silu gate.
 // * delta_step: one decoded token per sequence: state read once and written once, output norm and gate in the same launch.
 //
@@ -832,9 +832,9 @@ static int launch_scan(const ScanArgs& p, cudaStream_t s) {
     launch_pdl(delta_pairs_kernel<T, false>, pgrid, dim3(128), 0, s, p);
   }
   auto grid = [&](int cpl) { return dim3((p.vdim + 8 * cpl - 1) / (8 * cpl), p.H, p.B); };
-  if (p.dim <= 64) launch_pdl(delta_scan_kernel<T, 4, 4, 5>, grid(4), dim3(128), 0, s, p);
-  else if (p.dim <= 128) launch_pdl(delta_scan_kernel<T, 8, 4, 5>, grid(4), dim3(128), 0, s, p);
-  else if (p.dim <= 256) launch_pdl(delta_scan_kernel<T, 16, 4, 3>, grid(4), dim3(128), 0, s, p);
+  if (p.dim <= 64) launch_pdl(delta_scan_kernel<T, 4, 8, 2>, grid(8), dim3(128), 0, s, p);
+  else if (p.dim <= 128) launch_pdl(delta_scan_kernel<T, 8, 8, 2>, grid(8), dim3(128), 0, s, p);
+  else if (p.dim <= 256) launch_pdl(delta_scan_kernel<T, 16, 4, 2>, grid(4), dim3(128), 0, s, p);
   else return 1006;
   return int(cudaGetLastError());
 }

@@ -50,9 +50,10 @@ struct HeadMmArgs {
   long long ldg;
   int B, H, N, K;
 };
+constexpr int HM_EXPAND_ROWS = 8;  // sequences per CTA of the expand form: its time is the gathering of the partial latents, not the MMAs
 constexpr int HM_MAX_CHUNKS = 64;  // two per lane in the merge
 
-// CTA: 16 sequences x (WARPS * NT * 8) output columns of one head.
+// CTA: 16 (expand: 8) sequences x (WARPS * NT * 8) output columns of one head.
 template <int WARPS, int NT, bool EXPAND>
 __global__ void __launch_bounds__(WARPS * 32) latent_head_mm_kernel(const HeadMmArgs p) {
   pdl_prologue();
@@ -60,7 +61,8 @@ __global__ void __launch_bounds__(WARPS * 32) latent_head_mm_kernel(const HeadMm
   __nv_bfloat16* sx = reinterpret_cast<__nv_bfloat16*>(smem_raw);  // [16][K + 32]
   __shared__ float s_f[EXPAND ? 16 : 1][EXPAND ? HM_MAX_CHUNKS : 1];
   const int ldx = p.K + 32, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
-  const int h = blockIdx.y, b0 = blockIdx.z * 16, nb = min(16, p.B - b0);
+  constexpr int ROWS = EXPAND ? HM_EXPAND_ROWS : 16;
+  const int h = blockIdx.y, b0 = blockIdx.z * ROWS, nb = min(ROWS, p.B - b0);
   const int n0 = (blockIdx.x * WARPS + warp) * NT * 8;
   // the first PRE steps of this lane's weights, requested before the inputs are gathered
   constexpr int PRE = 16 / NT;
@@ -87,7 +89,7 @@ __global__ void __launch_bounds__(WARPS * 32) latent_head_mm_kernel(const HeadMm
     // four rows of a column quad at a time: with the chunk loop unrolled, up to eight loads are in flight per thread
     const int quads = p.K >> 2;
     const long long row = (long long)p.H * p.n_chunks * p.K;  // elements between sequences
-    for (int i = tid; i < 4 * quads; i += WARPS * 32) {
+    for (int i = tid; i < (ROWS / 4) * quads; i += WARPS * 32) {
       const int j = (i / quads) * 4, r = (i % quads) * 4;
       float4 a[4];
 #pragma unroll
@@ -138,7 +140,8 @@ __global__ void __launch_bounds__(WARPS * 32) latent_head_mm_kernel(const HeadMm
     for (int u = 0; u < PRE; ++u) {
       const int k = k0 + 32 * u;
       if (k >= p.K) break;
-      const uint4 lo = *reinterpret_cast<const uint4*>(sx + g * ldx + k + 8 * t), hi = *reinterpret_cast<const uint4*>(sx + (g + 8) * ldx + k + 8 * t);
+      const uint4 lo = *reinterpret_cast<const uint4*>(sx + g * ldx + k + 8 * t);
+      const uint4 hi = ROWS > 8 ? *reinterpret_cast<const uint4*>(sx + (g + 8) * ldx + k + 8 * t) : make_uint4(0, 0, 0, 0);
 #pragma unroll
       for (int i = 0; i < NT; ++i) {
         mma_bf16_16816(acc[i], lo.x, hi.x, lo.y, hi.y, cur[u][i].x, cur[u][i].y);
@@ -395,6 +398,6 @@ ATS_API int ats_latent_decode_mma(const void* q, long long ldq, const void* w_uk
   x.out = static_cast<__nv_bfloat16*>(out); x.out_ld = ldo; x.out_hs = vdim;
   x.gate = static_cast<const __nv_bfloat16*>(gate); x.ldg = ldg;
   x.B = B; x.H = H; x.N = vdim; x.K = rank;
-  e = launch_pdl(latent_head_mm_kernel<8, 2, true>, dim3((vdim + 127) / 128, H, bt), dim3(256), size_t(16) * (rank + 32) * 2, s, x);
+  e = launch_pdl(latent_head_mm_kernel<8, 2, true>, dim3((vdim + 127) / 128, H, (B + HM_EXPAND_ROWS - 1) / HM_EXPAND_ROWS), dim3(256), size_t(16) * (rank + 32) * 2, s, x);
   return int(e != cudaSuccess ? e : cudaGetLastError());
 }
