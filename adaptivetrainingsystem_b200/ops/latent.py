@@ -259,8 +259,10 @@ def latent_decode(q: torch.Tensor, ring: torch.Tensor, w_uk: torch.Tensor, w_uv_
         return out
     dev = q.device
     if w_ukt is not None and w_uv is not None and R <= 64 * 4096:
-        # two CTAs per SM share the ring's chunks: as many chunks per sequence as fit one wave, of whole 64-row tiles, at most 64
-        n_chunks = max(1, min(64, (R + 63) // 64, 296 // (B * ((H + 15) // 16))))
+        # as many chunks per sequence as fit one wave of CTAs (two per SM for up to 16 heads, else one with 32 heads), of whole 64-row
+        # pieces, at most 64
+        slots, ctas = (296, B) if H <= 16 else (148, B * ((H + 31) // 32))
+        n_chunks = max(1, min(64, (R + 63) // 64, slots // ctas))
         chunk = ((R + n_chunks - 1) // n_chunks + 63) // 64 * 64
         n_chunks = (R + chunk - 1) // chunk
         qa = torch.empty(B, H, s.rank, dtype=q.dtype, device=dev)

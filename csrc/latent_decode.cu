@@ -188,30 +188,30 @@ constexpr int LR_KEYS = 32, LR_THREADS = 256;
 
 struct RingSmem {
   int ldt, qa, s, pr, al, total;  // row pitch of tile and queries (elements), byte offsets
-  __host__ __device__ explicit RingSmem(int cw) {
+  __host__ __device__ RingSmem(int cw, int groups) {
     ldt = cw + 8;
     qa = 2 * LR_KEYS * ldt * 2;
-    s = qa + 16 * ldt * 2;
-    pr = s + 4 * 16 * (LR_KEYS + 4) * 4;
-    al = pr + 16 * (LR_KEYS + 8) * 2;
-    total = al + 16 * 4;
+    s = qa + groups * 16 * ldt * 2;
+    pr = s + groups * 4 * 16 * (LR_KEYS + 4) * 4;
+    al = pr + groups * 16 * (LR_KEYS + 8) * 2;
+    total = al + groups * 16 * 4;
   }
 };
 
-// NTW: 8-column tiles of the latent per warp (rank = 64 * NTW).
-template <int NTW>
-__global__ void __launch_bounds__(LR_THREADS, 2) latent_ring_kernel(const RingArgs p) {
+// NTW: 8-column tiles of the latent per warp (rank = 64 * NTW).  HG: groups of 16 heads that share the CTA's ring tiles, eight warps each.
+template <int NTW, int HG>
+__global__ void __launch_bounds__(LR_THREADS * HG, 2 / HG) latent_ring_kernel(const RingArgs p) {
   pdl_prologue();
   extern __shared__ __align__(16) uint8_t smem_raw[];
   const int cw = p.rank + p.rot;
-  const RingSmem L(cw);
+  const RingSmem L(cw, HG);
+  const int tid = threadIdx.x % LR_THREADS, group = threadIdx.x / LR_THREADS, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
   __nv_bfloat16* tile = reinterpret_cast<__nv_bfloat16*>(smem_raw);
-  __nv_bfloat16* sq = reinterpret_cast<__nv_bfloat16*>(smem_raw + L.qa);
-  float* ss = reinterpret_cast<float*>(smem_raw + L.s);                  // [quarter of the reduction][16][LR_KEYS + 4]
-  __nv_bfloat16* sp = reinterpret_cast<__nv_bfloat16*>(smem_raw + L.pr);  // [16][LR_KEYS + 8]
-  float* sal = reinterpret_cast<float*>(smem_raw + L.al);                // [16]
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
-  const int chunk = blockIdx.x, h0 = blockIdx.y * 16, b = blockIdx.z, nh = min(16, p.H - h0);
+  __nv_bfloat16* sq = reinterpret_cast<__nv_bfloat16*>(smem_raw + L.qa) + group * 16 * L.ldt;
+  float* ss = reinterpret_cast<float*>(smem_raw + L.s) + group * 4 * 16 * (LR_KEYS + 4);                  // [quarter of the reduction][16][LR_KEYS + 4]
+  __nv_bfloat16* sp = reinterpret_cast<__nv_bfloat16*>(smem_raw + L.pr) + group * 16 * (LR_KEYS + 8);     // [16][LR_KEYS + 8]
+  float* sal = reinterpret_cast<float*>(smem_raw + L.al) + group * 16;                                   // [16]
+  const int chunk = blockIdx.x, h0 = (blockIdx.y * HG + group) * 16, b = blockIdx.z, nh = max(0, min(16, p.H - h0));
   const int pos = p.lengths[b], n = min(pos + 1, p.R), k0 = chunk * p.chunk, k1 = min(n, k0 + p.chunk);
   float* ml = p.part_ml + (((long long)b * p.H + h0) * p.n_chunks + chunk) * 2;
   if (k0 >= k1) {
@@ -222,11 +222,11 @@ __global__ void __launch_bounds__(LR_THREADS, 2) latent_ring_kernel(const RingAr
     return;
   }
   const __nv_bfloat16* ring = p.ring + (long long)b * p.ring_bs;
-  // rows 4 w .. 4 w + 3 of a tile belong to warp w: no divisions in the copy loop
+  // every warp of the CTA copies its own rows of a tile: no divisions in the copy loop
   auto fetch = [&](int first, int buf) {
 #pragma unroll
-    for (int x = 0; x < LR_KEYS / 8; ++x) {
-      const int r = warp * (LR_KEYS / 8) + x;
+    for (int x = 0; x < LR_KEYS / (8 * HG); ++x) {
+      const int r = (group * 8 + warp) * (LR_KEYS / (8 * HG)) + x;
       const bool ok = first + r < k1;
       const __nv_bfloat16* src = ring + (long long)(ok ? first + r : k0) * p.cwp;
       __nv_bfloat16* dst = tile + (buf * LR_KEYS + r) * L.ldt;
@@ -353,12 +353,16 @@ __global__ void __launch_bounds__(LR_THREADS, 2) latent_ring_kernel(const RingAr
     }
 }
 
+template <int NTW, int HG>
+static cudaError_t launch_ring_groups(const RingArgs& p, int B, cudaStream_t s) {
+  const RingSmem L(p.rank + p.rot, HG);
+  cudaError_t e = cudaFuncSetAttribute(latent_ring_kernel<NTW, HG>, cudaFuncAttributeMaxDynamicSharedMemorySize, L.total);
+  if (e != cudaSuccess) return e;
+  return launch_pdl(latent_ring_kernel<NTW, HG>, dim3(p.n_chunks, (p.H + 16 * HG - 1) / (16 * HG), B), dim3(LR_THREADS * HG), size_t(L.total), s, p);
+}
 template <int NTW>
 static cudaError_t launch_ring(const RingArgs& p, int B, cudaStream_t s) {
-  const RingSmem L(p.rank + p.rot);
-  cudaError_t e = cudaFuncSetAttribute(latent_ring_kernel<NTW>, cudaFuncAttributeMaxDynamicSharedMemorySize, L.total);
-  if (e != cudaSuccess) return e;
-  return launch_pdl(latent_ring_kernel<NTW>, dim3(p.n_chunks, (p.H + 15) / 16, B), dim3(LR_THREADS), size_t(L.total), s, p);
+  return p.H > 16 ? launch_ring_groups<NTW, 2>(p, B, s) : launch_ring_groups<NTW, 1>(p, B, s);
 }
 
 }  // namespace ats
