@@ -9,6 +9,7 @@ from __future__ import annotations
 
 import json
 import os
+import time
 from typing import Any, Callable, Dict, List, Optional
 
 import torch
@@ -124,6 +125,8 @@ class _Timer:
         self.iters, self.peak, self.rows = iters, peaks(), []
 
     def add(self, model: str, name: str, fn: Callable[[], Any], bytes_: float, flops: float = 0.0, fp32: float = 0.0) -> None:
+        torch.cuda.synchronize()
+        time.sleep(0.3)   # clocks that a heavy product before this one has pulled under the power cap recover
         for _ in range(3):
             fn()
         ts = []

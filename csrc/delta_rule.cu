@@ -388,6 +388,11 @@ struct RowPiece {
   }
 };
 
+template <int BYTES> struct Bits;
+template <> struct Bits<4> { using type = uint32_t; };
+template <> struct Bits<8> { using type = uint2; };
+template <> struct Bits<16> { using type = uint4; };
+
 // Sixteen lanes share CPL value columns: lane l holds EPL state rows (dim <= 16 * EPL) of each.  CTA = 4 warps of 2 lane groups ->
 // 8 * CPL columns of one head.  k and q rows stay in the element type in shared memory: with the state spread over sixteen lanes and
 // 16-byte reads of eight bf16 values the load pipe stays below the FMA pipe.  The next group's q, k, v and constants are requested before this group's products
@@ -421,9 +426,13 @@ __global__ void __launch_bounds__(128, OCC) delta_scan_kernel(const ScanArgs p) 
   T* obase = static_cast<T*>(p.o) + (long long)b * p.L * p.ldo + (long long)h * p.vdim + colh;
   const float* cbase = p.coef + ((long long)b * p.groups * p.H + h) * CO;
   const bool vec = (p.dim % VEC) == 0;  // rows are whole 16-byte pieces (p.ldm is a multiple of 8)
+  // the lane's HC values of a token are one aligned access when every head starts at a multiple of HC columns
+  using VBits = typename Bits<HC * int(sizeof(T))>::type;
+  const bool vecv = (p.vdim % HC) == 0 && ((2 * p.KH * p.dim) % HC) == 0 && (p.ldo % HC) == 0;
+  const bool inside = colh < p.vdim;  // with vecv: all HC columns or none
   uint4 piece[NP];
   float4 cpiece;
-  float vnext[HC];
+  union { VBits bits; T v[HC]; } vnext;  // as loaded: converting here would wait for the load
   auto request = [&](int grp) {
     const int t0 = grp * DC, n = min(DC, p.L - t0);
 #pragma unroll
@@ -441,7 +450,17 @@ __global__ void __launch_bounds__(128, OCC) delta_scan_kernel(const ScanArgs p) 
     }
     if (tid < CO / 4) cpiece = *reinterpret_cast<const float4*>(cbase + (long long)grp * p.H * CO + tid * 4);
 #pragma unroll
-    for (int c = 0; c < HC; ++c) vnext[c] = (tok < n && colh + c < p.vdim) ? Typed<T>::load(vbase + (long long)(t0 + tok) * p.ldm + c) : 0.f;
+    for (int c = 0; c < HC; ++c) Typed<T>::store(&vnext.v[c], 0.f);
+    if (tok < n) {
+      const T* src = vbase + (long long)(t0 + tok) * p.ldm;
+      if (vecv) {
+        if (inside) vnext.bits = *reinterpret_cast<const VBits*>(src);
+      } else {
+#pragma unroll
+        for (int c = 0; c < HC; ++c)
+          if (colh + c < p.vdim) vnext.v[c] = src[c];
+      }
+    }
   };
   auto deposit = [&](int buf) {
 #pragma unroll
@@ -497,7 +516,7 @@ __global__ void __launch_bounds__(128, OCC) delta_scan_kernel(const ScanArgs p) 
     {
       float v[HC];
 #pragma unroll
-      for (int c = 0; c < HC; ++c) v[c] = vnext[c];
+      for (int c = 0; c < HC; ++c) v[c] = Typed<T>::load(&vnext.v[c]);
       if (grp + 1 < p.groups) request(grp + 1);
       products(buf, 0, sk);
       const float gk = co[2 * DC * DC + tok];
@@ -533,10 +552,19 @@ __global__ void __launch_bounds__(128, OCC) delta_scan_kernel(const ScanArgs p) 
     }
     products(buf, 1, sk);
     const float gq = co[2 * DC * DC + DC + tok], GC = co[2 * DC * DC + 3 * DC];
-    if (tok < n)
+    if (tok < n) {
+      union { VBits bits; T v[HC]; } ov;
 #pragma unroll
-      for (int c = 0; c < HC; ++c)
-        if (colh + c < p.vdim) Typed<T>::store(obase + (long long)(t0 + tok) * p.ldo + c, o[c] + gq * sk[c]);
+      for (int c = 0; c < HC; ++c) Typed<T>::store(&ov.v[c], o[c] + gq * sk[c]);
+      T* dst = obase + (long long)(t0 + tok) * p.ldo;
+      if (vecv) {
+        if (inside) *reinterpret_cast<VBits*>(dst) = ov.bits;
+      } else {
+#pragma unroll
+        for (int c = 0; c < HC; ++c)
+          if (colh + c < p.vdim) dst[c] = ov.v[c];
+      }
+    }
 #pragma unroll
     for (int c = 0; c < CPL; ++c)
 #pragma unroll

@@ -7,7 +7,7 @@
 // * Portions of a prompt: latent_context gathers the window that precedes the portion from the ring and appends the portion's own
 //   entries (norms, rotation) -> ctx [n_old + L rows]; a GEMM expands ctx to per-head keys and values; window_attn attends; latent_finish
 //   rotates the queries before that and puts the portion's last R entries into the ring.
-// * Decoding works on the latents themselves: the query's unrotated part is multiplied by the key expansion (head_matmul), scores and
+// * Decoding works on the latents themselves: the query's unrotated part is multiplied by the key expansion (latent_absorb), scores and
 //   weighted sums run over the ring (latent_decode), and the merged latent is multiplied by the value expansion (latent_expand, with the
 //   output gate), so the per-head keys and values of the window never exist.
 //

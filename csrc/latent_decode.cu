@@ -6,8 +6,8 @@
 //                            the MMA), soft-max, weighted sum of the latents; chunks of the ring are merged by the next kernel
 //   latent_head_mm<expand>   out[b, h, :] = sigmoid(gate) * W_uv[h] (merged latent)   [16 sequences x rank] x [rank x vdim]
 //
-// A decode step is bound by the bytes of the ring, so warp-level MMAs are enough; a 32-row tile of the ring is fetched once with
-// cp.async (the next one while this one is used) and serves both products (plain and transposing ldmatrix; rows are padded by 16 bytes against bank conflicts).  Weights
+// A decode step is bound by the bytes of the ring, so warp-level MMAs are enough; a tile of 32 or 64 ring rows is fetched once with
+// cp.async (later ones while this one is used) and serves both products (plain and transposing ldmatrix; rows are padded by 16 bytes against bank conflicts).  Weights
 // stream straight from global memory into B fragments: the order of the reduction index is permuted so that the 16-byte piece a lane
 // loads is its fragment for two consecutive steps, and the A fragments are read with the same permutation.
 #include "common.cuh"
@@ -55,7 +55,7 @@ constexpr int HM_MAX_CHUNKS = 64;  // two per lane in the merge
 
 // CTA: 16 (expand: 8) sequences x (WARPS * NT * 8) output columns of one head.
 template <int WARPS, int NT, bool EXPAND>
-__global__ void __launch_bounds__(WARPS * 32) latent_head_mm_kernel(const HeadMmArgs p) {
+__global__ void __launch_bounds__(WARPS * 32, EXPAND ? 2 : 3) latent_head_mm_kernel(const HeadMmArgs p) {
   pdl_prologue();
   extern __shared__ __align__(16) uint8_t smem_raw[];
   __nv_bfloat16* sx = reinterpret_cast<__nv_bfloat16*>(smem_raw);  // [16][K + 32]
@@ -65,7 +65,7 @@ __global__ void __launch_bounds__(WARPS * 32) latent_head_mm_kernel(const HeadMm
   const int h = blockIdx.y, b0 = blockIdx.z * ROWS, nb = min(ROWS, p.B - b0);
   const int n0 = (blockIdx.x * WARPS + warp) * NT * 8;
   // the first PRE steps of this lane's weights, requested before the inputs are gathered
-  constexpr int PRE = 16 / NT;
+  constexpr int PRE = EXPAND ? 4 : 3;
   const __nv_bfloat16* w = p.w + h * p.w_hs + 8 * t;
   uint4 pre[PRE][NT];
 #pragma unroll
@@ -184,27 +184,29 @@ struct RingArgs {
   float* part_o;              // [B, H, n_chunks, rank]
   float* part_ml;             // [B, H, n_chunks, 2]
 };
-constexpr int LR_KEYS = 32, LR_THREADS = 256;
+constexpr int LR_THREADS = 256;
 
 struct RingSmem {
   int ldt, qa, s, pr, al, total;  // row pitch of tile and queries (elements), byte offsets
-  __host__ __device__ RingSmem(int cw, int groups) {
+  __host__ __device__ RingSmem(int cw, int groups, int stages, int keys) {
     ldt = cw + 8;
-    qa = 2 * LR_KEYS * ldt * 2;
+    qa = stages * keys * ldt * 2;
     s = qa + groups * 16 * ldt * 2;
-    pr = s + groups * 4 * 16 * (LR_KEYS + 4) * 4;
-    al = pr + groups * 16 * (LR_KEYS + 8) * 2;
+    pr = s + groups * 4 * 16 * (keys + 4) * 4;
+    al = pr + groups * 16 * (keys + 8) * 2;
     total = al + groups * 16 * 4;
   }
 };
 
 // NTW: 8-column tiles of the latent per warp (rank = 64 * NTW).  HG: groups of 16 heads that share the CTA's ring tiles, eight warps each.
-template <int NTW, int HG>
+// STAGES: ring tiles in shared memory.
+// LR_KEYS: rows of a tile (32 or 64; more rows spread the barriers and the soft-max reductions over more keys).
+template <int NTW, int HG, int STAGES, int LR_KEYS>
 __global__ void __launch_bounds__(LR_THREADS * HG, 2 / HG) latent_ring_kernel(const RingArgs p) {
   pdl_prologue();
   extern __shared__ __align__(16) uint8_t smem_raw[];
   const int cw = p.rank + p.rot;
-  const RingSmem L(cw, HG);
+  const RingSmem L(cw, HG, STAGES, LR_KEYS);
   const int tid = threadIdx.x % LR_THREADS, group = threadIdx.x / LR_THREADS, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
   __nv_bfloat16* tile = reinterpret_cast<__nv_bfloat16*>(smem_raw);
   __nv_bfloat16* sq = reinterpret_cast<__nv_bfloat16*>(smem_raw + L.qa) + group * 16 * L.ldt;
@@ -232,9 +234,12 @@ __global__ void __launch_bounds__(LR_THREADS * HG, 2 / HG) latent_ring_kernel(co
       __nv_bfloat16* dst = tile + (buf * LR_KEYS + r) * L.ldt;
       for (int c = lane * 8; c < cw; c += 256) cp_async_16(smem_u32(dst + c), src + c, ok);
     }
-    cp_async_commit();
   };
-  fetch(k0, 0);
+#pragma unroll
+  for (int x = 0; x < STAGES - 1; ++x) {
+    if (k0 + x * LR_KEYS < k1) fetch(k0 + x * LR_KEYS, x);
+    cp_async_commit();  // (possibly empty: the number of groups in flight stays the same)
+  }
   // absorbed queries (rows of heads that do not exist are zero), rotated parts
   for (int i = tid; i < 16 * (p.rank >> 3); i += LR_THREADS) {
     const int r = i / (p.rank >> 3), c = (i % (p.rank >> 3)) * 8;
@@ -261,7 +266,7 @@ __global__ void __launch_bounds__(LR_THREADS * HG, 2 / HG) latent_ring_kernel(co
 #pragma unroll
     for (int e = 0; e < 4; ++e) acc[i][e] = 0.f;
   float m_[2] = {-INFINITY, -INFINITY}, l_[2] = {0.f, 0.f};  // soft-max state of heads 2 * warp, + 1
-  // score phase: warp w takes keys 16 (w & 1) .. + 15 of a tile and a quarter of the reduction, whose query fragments stay in registers
+  // score phase: warp w takes keys 16 (w & 1) .. + 15 of every 32 keys of a tile and a quarter of the reduction, whose query fragments stay in registers
   const int steps = cw >> 4, per = (steps + 3) >> 2, q_lo = (warp >> 1) * per, q_n = max(0, min(per, steps - q_lo));
   __syncthreads();  // queries are complete
   uint32_t aq[NTW + 2][4];
@@ -273,44 +278,57 @@ __global__ void __launch_bounds__(LR_THREADS * HG, 2 / HG) latent_ring_kernel(co
   const uint32_t p_addr = smem_u32(sp + (lane & 15) * (LR_KEYS + 8) + (lane >> 4) * 8);
   const uint32_t v_addr = smem_u32(tile + (lane & 15) * L.ldt + warp * NTW * 8 + (lane >> 4) * 8);
   int buf = 0;
-  for (int first = k0; first < k1; first += LR_KEYS, buf ^= 1) {
-    if (first + LR_KEYS < k1) {
-      fetch(first + LR_KEYS, buf ^ 1);
-      cp_async_wait<1>();
-    } else {
-      cp_async_wait<0>();
-    }
-    __syncthreads();
+  for (int first = k0; first < k1; first += LR_KEYS) {
+    cp_async_wait<STAGES - 2>();
+    __syncthreads();  // this tile is complete, and every warp is done with the one before it: its stage takes the next fetch
+    const int ahead = first + (STAGES - 1) * LR_KEYS, into = buf == 0 ? STAGES - 1 : buf - 1;
+    if (ahead < k1) fetch(ahead, into);
+    cp_async_commit();
     const uint32_t stage = uint32_t(buf * LR_KEYS * L.ldt * 2);
     // ---- scores
     {
-      float c0[4] = {0.f, 0.f, 0.f, 0.f}, c1[4] = {0.f, 0.f, 0.f, 0.f};  // keys 0..7 / 8..15 of the warp's sixteen
 #pragma unroll
-      for (int x = 0; x < NTW + 2; ++x)
-        if (x < q_n) {
-          uint32_t bb[4];
-          ldmatrix_x4(b_addr + stage + x * 32, bb);
-          mma_bf16_16816(c0, aq[x][0], aq[x][1], aq[x][2], aq[x][3], bb[0], bb[1]);
-          mma_bf16_16816(c1, aq[x][0], aq[x][1], aq[x][2], aq[x][3], bb[2], bb[3]);
-        }
-      float* s0 = ss + ((warp >> 1) * 16 + g) * (LR_KEYS + 4) + (warp & 1) * 16 + 2 * t;
-      *reinterpret_cast<float2*>(s0) = make_float2(c0[0], c0[1]);
-      *reinterpret_cast<float2*>(s0 + 8) = make_float2(c1[0], c1[1]);
-      *reinterpret_cast<float2*>(s0 + 8 * (LR_KEYS + 4)) = make_float2(c0[2], c0[3]);
-      *reinterpret_cast<float2*>(s0 + 8 * (LR_KEYS + 4) + 8) = make_float2(c1[2], c1[3]);
+      for (int kg = 0; kg < LR_KEYS / 32; ++kg) {
+        float c0[4] = {0.f, 0.f, 0.f, 0.f}, c1[4] = {0.f, 0.f, 0.f, 0.f};  // keys 0..7 / 8..15 of the sixteen
+#pragma unroll
+        for (int x = 0; x < NTW + 2; ++x)
+          if (x < q_n) {
+            uint32_t bb[4];
+            ldmatrix_x4(b_addr + stage + (kg * 32 * L.ldt + x * 16) * 2, bb);
+            mma_bf16_16816(c0, aq[x][0], aq[x][1], aq[x][2], aq[x][3], bb[0], bb[1]);
+            mma_bf16_16816(c1, aq[x][0], aq[x][1], aq[x][2], aq[x][3], bb[2], bb[3]);
+          }
+        float* s0 = ss + ((warp >> 1) * 16 + g) * (LR_KEYS + 4) + kg * 32 + (warp & 1) * 16 + 2 * t;
+        *reinterpret_cast<float2*>(s0) = make_float2(c0[0], c0[1]);
+        *reinterpret_cast<float2*>(s0 + 8) = make_float2(c1[0], c1[1]);
+        *reinterpret_cast<float2*>(s0 + 8 * (LR_KEYS + 4)) = make_float2(c0[2], c0[3]);
+        *reinterpret_cast<float2*>(s0 + 8 * (LR_KEYS + 4) + 8) = make_float2(c1[2], c1[3]);
+      }
     }
     __syncthreads();
-    // ---- soft-max: two heads per warp, one key per lane
+    // ---- soft-max: two heads per warp, LR_KEYS / 32 keys per lane
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
       const int r = warp * 2 + e;
-      const float x = first + lane < k1 ? ((ss[r * (LR_KEYS + 4) + lane] + ss[(16 + r) * (LR_KEYS + 4) + lane]) +
-                                             (ss[(32 + r) * (LR_KEYS + 4) + lane] + ss[(48 + r) * (LR_KEYS + 4) + lane])) * p.scale : -INFINITY;
-      const float mn = fmaxf(m_[e], warp_max(x));  // the tile has at least one key: finite
-      const float al = __expf(m_[e] - mn), pr = __expf(x - mn);
+      float x[LR_KEYS / 32], mt = -INFINITY, sum = 0.f;
+#pragma unroll
+      for (int kg = 0; kg < LR_KEYS / 32; ++kg) {
+        const int key = kg * 32 + lane;
+        const float* s0 = ss + r * (LR_KEYS + 4) + key;
+        constexpr int Q = 16 * (LR_KEYS + 4);
+        x[kg] = first + key < k1 ? ((s0[0] + s0[Q]) + (s0[2 * Q] + s0[3 * Q])) * p.scale : -INFINITY;
+        mt = fmaxf(mt, x[kg]);
+      }
+      const float mn = fmaxf(m_[e], warp_max(mt));  // the tile has at least one key: finite
+      const float al = __expf(m_[e] - mn);
+#pragma unroll
+      for (int kg = 0; kg < LR_KEYS / 32; ++kg) {
+        const float pr = __expf(x[kg] - mn);
+        sum += pr;
+        sp[r * (LR_KEYS + 8) + kg * 32 + lane] = __float2bfloat16(pr);
+      }
       m_[e] = mn;
-      l_[e] = l_[e] * al + warp_sum(pr);
-      sp[r * (LR_KEYS + 8) + lane] = __float2bfloat16(pr);
+      l_[e] = l_[e] * al + warp_sum(sum);
       if (lane == 0) sal[r] = al;
     }
     __syncthreads();
@@ -333,7 +351,7 @@ __global__ void __launch_bounds__(LR_THREADS * HG, 2 / HG) latent_ring_kernel(co
         mma_bf16_16816(acc[i + 1], a[0], a[1], a[2], a[3], v[2], v[3]);
       }
     }
-    __syncthreads();  // the next fetch overwrites this stage's partner, and the scores are written again
+    buf = buf + 1 == STAGES ? 0 : buf + 1;
   }
 #pragma unroll
   for (int i = 0; i < NTW; ++i) {
@@ -353,16 +371,17 @@ __global__ void __launch_bounds__(LR_THREADS * HG, 2 / HG) latent_ring_kernel(co
     }
 }
 
-template <int NTW, int HG>
+template <int NTW, int HG, int STAGES, int KEYS>
 static cudaError_t launch_ring_groups(const RingArgs& p, int B, cudaStream_t s) {
-  const RingSmem L(p.rank + p.rot, HG);
-  cudaError_t e = cudaFuncSetAttribute(latent_ring_kernel<NTW, HG>, cudaFuncAttributeMaxDynamicSharedMemorySize, L.total);
+  const RingSmem L(p.rank + p.rot, HG, STAGES, KEYS);
+  cudaError_t e = cudaFuncSetAttribute(latent_ring_kernel<NTW, HG, STAGES, KEYS>, cudaFuncAttributeMaxDynamicSharedMemorySize, L.total);
   if (e != cudaSuccess) return e;
-  return launch_pdl(latent_ring_kernel<NTW, HG>, dim3(p.n_chunks, (p.H + 16 * HG - 1) / (16 * HG), B), dim3(LR_THREADS * HG), size_t(L.total), s, p);
+  return launch_pdl(latent_ring_kernel<NTW, HG, STAGES, KEYS>, dim3(p.n_chunks, (p.H + 16 * HG - 1) / (16 * HG), B), dim3(LR_THREADS * HG), size_t(L.total), s, p);
 }
 template <int NTW>
 static cudaError_t launch_ring(const RingArgs& p, int B, cudaStream_t s) {
-  return p.H > 16 ? launch_ring_groups<NTW, 2>(p, B, s) : launch_ring_groups<NTW, 1>(p, B, s);
+  const bool wide = p.H > 16 && RingSmem(p.rank + p.rot, 2, 2, 64).total <= 227 * 1024;
+  return wide ? launch_ring_groups<NTW, 2, 2, 64>(p, B, s) : launch_ring_groups<NTW, 1, 2, 32>(p, B, s);
 }
 
 }  // namespace ats
@@ -378,7 +397,7 @@ ATS_API int ats_latent_decode_mma(const void* q, long long ldq, const void* w_uk
   if (B < 1) return 0;
   const bool rank_ok = rank == 128 || rank == 256 || rank == 384 || rank == 512;
   if (!rank_ok || (dim & 31) || dim > 512 || (rot & 31) || rot < 32 || rot > 128 || (vdim & 7) || (ldq & 7) || (ldv & 7) || (cwp & 7) || (ring_bs & 7) || (ldo & 1) ||
-      (gate && (ldg & 1)) || chunk < LR_KEYS || (chunk % LR_KEYS) || n_chunks < 1 || n_chunks > HM_MAX_CHUNKS || (long long)chunk * n_chunks < R)
+      (gate && (ldg & 1)) || chunk < 64 || (chunk % 64) || n_chunks < 1 || n_chunks > HM_MAX_CHUNKS || (long long)chunk * n_chunks < R)
     return 1003;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   HeadMmArgs a = {};

@@ -55,7 +55,7 @@ def tokens(n, vocab=104, seed=1):
     return torch.randint(0, vocab, (n,), generator=torch.Generator().manual_seed(seed)).tolist()
 
 
-def run_portions(model, ids, sizes, rows=1):
+def run_portions(model, ids, sizes):
     """Logits of every position when the tokens come in portions of these sizes."""
     dev = model.embed.device
     cache, out, at = model.make_cache(1, len(ids)), [], 0
@@ -98,7 +98,7 @@ def test_norm_residual_gelu_steps(device, dtype):
 
 def _one_layer(layer, **kw):
     cfg = O.config([layer], **kw)
-    return cfg, O.random_weights(cfg, seed=3, sharp=kw.pop("sharp", 1.0))
+    return cfg, O.random_weights(cfg, seed=3)
 
 
 @pytest.mark.parametrize("device,dtype", PLACES)
