@@ -284,6 +284,99 @@ class VimodraConfig:
         return d
 
 
+@dataclass
+class NemipelConfig:
+    """Architecture of a Nemipel model: a list of layers with their own mixers (``lightning`` | ``attention`` | ``channel_delta``), norms
+    after the residual sum, capped logits (``models/nemipel.py``)."""
+    vocab_size: int
+    hidden_size: int
+    layers: List[LayerSpec]
+    norm_eps: float = 1e-6
+    postln_alpha: float = 1.0      # weight of the residual in the sum that is normed
+    logit_softcap: float = 0.0     # 0: logits are not capped
+    seq_length: int = 4096         # default cache length and size of the rotary tables (both grow on demand)
+
+    MIXERS = {"lightning": ("heads", "dim", "vdim"), "attention": ("heads", "kv_heads", "dim", "vdim"),
+              "channel_delta": ("heads", "kv_heads", "dim", "vdim", "conv")}
+
+    def __post_init__(self):
+        for layer in self.layers:
+            if layer.type == "channel_delta":   # inner widths of the low-rank projections; a model folder's tensors overrule these
+                layer.mixer.setdefault("decay_rank", layer.mixer.get("vdim"))
+                layer.mixer.setdefault("gate_rank", layer.mixer.get("vdim"))
+        self.validate()
+
+    @property
+    def num_layers(self) -> int:
+        return len(self.layers)
+
+    def validate(self) -> None:
+        if self.vocab_size < 1 or self.hidden_size < 1 or not self.layers:
+            raise ValueError("vocab_size, hidden_size and the layer list must not be empty")
+        if self.logit_softcap < 0 or self.norm_eps < 0:
+            raise ValueError("logit_softcap and norm eps must not be negative")
+        for i, layer in enumerate(self.layers):
+            if layer.type not in self.MIXERS:
+                raise ValueError(f"layer {i}: unknown mixer {layer.type!r} (known: {sorted(self.MIXERS)})")
+            m = layer.mixer
+            missing = [k for k in self.MIXERS[layer.type] if not isinstance(m.get(k), int) or m[k] < 1]
+            if missing:
+                raise ValueError(f"layer {i} ({layer.type}): sizes {missing} are missing or not positive")
+            if "kv_heads" in self.MIXERS[layer.type] and m["heads"] % m["kv_heads"]:
+                raise ValueError(f"layer {i}: heads {m['heads']} not divisible by kv_heads {m['kv_heads']}")
+            if layer.type == "lightning":
+                if len(m.get("decay") or ()) != m["heads"] or not all(0 <= float(x) <= 1 for x in m["decay"]):
+                    raise ValueError(f"layer {i}: one decay between 0 and 1 per head is needed")
+            if layer.type != "attention" and m["dim"] > 256:
+                raise ValueError(f"layer {i}: state rows of up to 256 are built")
+            if layer.type == "attention":
+                self._validate_attention(i, m)
+            if layer.mlp is not None and (layer.mlp.get("kind", "dense") != "dense" or int(layer.mlp.get("ff", 0)) < 1):
+                raise ValueError(f"layer {i}: unknown feed-forward {layer.mlp!r}")
+
+    def _validate_attention(self, i: int, m: Dict[str, Any]) -> None:
+        rot = m.get("rot") or {}
+        if "base" not in rot or "dims" not in rot or "scale" not in m:
+            raise ValueError(f"layer {i}: rot.base, rot.dims and scale are needed")
+        if rot["dims"] % 2 or not 0 < rot["dims"] <= m["dim"]:
+            raise ValueError(f"layer {i}: an even number of dimensions is rotated, at most {m['dim']}")
+        if float(m.get("softcap") or 0) < 0:
+            raise ValueError(f"layer {i}: softcap must not be negative")
+        if m["vdim"] > 512:
+            raise ValueError(f"layer {i}: value heads of up to 512 dimensions are built")
+        j = m.get("kv_from")
+        if j is None:
+            return
+        if not 0 <= j < i or self.layers[j].type != "attention" or self.layers[j].mixer.get("kv_from") is not None:
+            raise ValueError(f"layer {i}: kv_from {j} is not an earlier attention layer with keys and values of its own")
+        if any(self.layers[j].mixer[k] != m[k] for k in ("kv_heads", "dim", "vdim")):
+            raise ValueError(f"layer {i}: the keys and values of layer {j} have other sizes")
+
+    def with_ranks(self, shape_of) -> "NemipelConfig":
+        """This configuration with the inner widths of the low-rank projections taken from tensor shapes (``shape_of(name)`` or ``None``)."""
+        layers = []
+        for i, layer in enumerate(self.layers):
+            m = dict(layer.mixer)
+            if layer.type == "channel_delta":
+                for key, name in (("decay_rank", "a1"), ("gate_rank", "g1")):
+                    shape = shape_of(f"l{i}.mix.{name}")
+                    m[key] = shape[0] if shape else m[key]
+            layers.append(LayerSpec(layer.type, m, layer.mlp))
+        return dataclasses.replace(self, layers=layers)
+
+    @classmethod
+    def from_dict(cls, d: Dict[str, Any]) -> "NemipelConfig":
+        """From the keys of a model folder's ``config.json``."""
+        return cls(vocab_size=int(d["vocab"]), hidden_size=int(d["width"]), norm_eps=float((d.get("norm") or {}).get("eps", 1e-6)),
+                   postln_alpha=float(d.get("postln_alpha", 1.0)), logit_softcap=float(d.get("logit_softcap") or 0.0),
+                   layers=[LayerSpec(l["type"], dict(l["mixer"]), dict(l["mlp"]) if l.get("mlp") else None) for l in d["layers"]],
+                   **({"seq_length": int(d["seq_length"])} if "seq_length" in d else {}))
+
+    def to_dict(self) -> Dict[str, Any]:
+        return {"architecture": "Nemipel", "vocab": self.vocab_size, "width": self.hidden_size, "norm": {"eps": self.norm_eps}, "postln_alpha": self.postln_alpha,
+                "logit_softcap": self.logit_softcap, "seq_length": self.seq_length, "layers": [dataclasses.asdict(l) for l in self.layers]}
+
+
 # --------------------------------------------------------------------------- #
 # Run configuration
 # --------------------------------------------------------------------------- #

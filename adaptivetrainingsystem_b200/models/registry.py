@@ -9,11 +9,13 @@ import json
 import os
 import struct
 from dataclasses import dataclass
-from typing import Any, Callable, Dict, Iterator, Tuple
+from typing import Any, Callable, Dict, Iterator, Tuple, Type
 
 import torch
 
-from ..config import ModelConfig, VimodraConfig
+from ..config import ModelConfig, NemipelConfig, VimodraConfig
+from .layered import LayeredDecoder
+from .nemipel import Nemipel
 from .transformer import DeepSeekTransformer
 from .vimodra import Vimodra
 
@@ -63,13 +65,14 @@ def _load_deepseek(cfg: ModelConfig, file: SafetensorsFile, dtype, device):
     return model.to(device, dtype).eval()
 
 
-def _load_vimodra(cfg: VimodraConfig, file: SafetensorsFile, dtype, device):
-    return Vimodra.from_tensors(cfg, file.tensor, list(file.keys()), dtype, device)
+def _layered(config: Callable[[Dict[str, Any]], Any], cls: Type[LayeredDecoder]) -> ModelEntry:
+    return ModelEntry(config, lambda cfg, file, dtype, device: cls.from_tensors(cfg, file.tensor, list(file.keys()), dtype, device), cls)
 
 
 MODELS: Dict[str, ModelEntry] = {
     "DeepSeekTransformer": ModelEntry(ModelConfig.from_dict, _load_deepseek, DeepSeekTransformer),
-    "Vimodra": ModelEntry(VimodraConfig.from_dict, _load_vimodra, Vimodra),
+    "Vimodra": _layered(VimodraConfig.from_dict, Vimodra),
+    "Nemipel": _layered(NemipelConfig.from_dict, Nemipel),
 }
 
 

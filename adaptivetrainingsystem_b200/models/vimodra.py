@@ -10,35 +10,25 @@ that begins next; the input norm of whatever follows).
 """
 from __future__ import annotations
 
-from typing import Any, Callable, Dict, List, Optional, Sequence, Tuple
+from typing import Dict, List, Optional, Tuple
 
 import torch
 import torch.nn as nn
 
-from .. import ops
 from ..config import VimodraConfig
 from ..ops import dyt as dyt_ops
-from ..ops import gemm as G
 from ..ops.latent import pad8
 from .cache import LayerStateCache
-from .mixers import GatedDelta, GeluMLP, LatentAttention, Step, padded, vector
-from .transformer import RotaryEmbedding
+from .layered import LayeredDecoder
+from .mixers import GatedDelta, GeluMLP, LatentAttention, padded, vector
 
 
-class Vimodra(nn.Module):
-    """Inference model; build it with :meth:`from_tensors` or :meth:`random`.  ``dtype`` bf16: tcgen05 products and bf16 activations
-    around an fp32 residual; fp32: everything in true 32-bit."""
-
-    # csrc files a program needs that only runs this model's step function
+class Vimodra(LayeredDecoder):
     KERNEL_SOURCES = ("gemm_tcgen05.cu", "dyt.cu", "latent_attention.cu",
                       "latent_decode.cu", "attention_window_tcgen05.cu", "delta_rule.cu")
-    # decode steps over pool rows of different lengths work without a captured graph too
-    eager_row_decode = True
 
     def __init__(self, config: VimodraConfig):
-        super().__init__()
-        self.config = config
-        self._ropes: Dict[Tuple[int, float], RotaryEmbedding] = {}
+        super().__init__(config)
         mixers, mlps = [], []
         for spec in config.layers:
             m = spec.mixer
@@ -52,15 +42,8 @@ class Vimodra(nn.Module):
         self.runs = config.runs()
         self.eval()
 
-    def _rope(self, dims: int, base: float) -> RotaryEmbedding:
-        key = (dims, base)
-        if key not in self._ropes:
-            self._ropes[key] = RotaryEmbedding(dims, self.config.seq_length, base)
-        return self._ropes[key]
-
     # -- weights ----------------------------------------------------------------------------------------------
     def tensor_shapes(self) -> Dict[str, Tuple[int, ...]]:
-        """Name -> shape of every tensor of a model folder."""
         cfg = self.config
         D = cfg.hidden_size
         out: Dict[str, Tuple[int, ...]] = {"embed": (cfg.vocab_size, D), "head": (cfg.vocab_size, D)}
@@ -81,41 +64,17 @@ class Vimodra(nn.Module):
                 out.update({p + "mlp." + n: s for n, s in self.mlps[i].shapes().items()})
         return out
 
-    @classmethod
-    def from_tensors(cls, config: VimodraConfig, get: Callable[[str], torch.Tensor], names: Sequence[str], dtype=torch.bfloat16, device="cuda") -> "Vimodra":
-        """``get(name)`` for the names of :meth:`tensor_shapes`; ``names`` is what the source holds (a surplus or a gap is an error)."""
-        model = cls(config)
-        shapes = model.tensor_shapes()
-        missing, extra = sorted(set(shapes) - set(names)), sorted(set(names) - set(shapes))
-        if missing or extra:
-            raise ValueError(f"the tensors do not fit the configuration: missing {missing[:5]}, unexpected {extra[:5]}")
-
-        def take(name):
-            t = get(name)
-            if tuple(t.shape) != shapes[name] and not (shapes[name] == () and t.numel() == 1):
-                raise ValueError(f"{name}: shape {tuple(t.shape)}, the configuration says {shapes[name]}")
-            return t
-        model._load(take, dtype, torch.device(device))
-        return model
-
-    @classmethod
-    def random(cls, config: VimodraConfig, dtype=torch.bfloat16, device="cuda", seed: int = 0) -> "Vimodra":
-        model = cls(config)
-        shapes = model.tensor_shapes()
-        gen = torch.Generator(device=device).manual_seed(seed)
-
-        def take(name):
-            shape, leaf = shapes[name], name.rsplit(".", 1)[-1]
-            if leaf in ("alpha", "A_log") or leaf.startswith(("ls", "norm")):
-                return torch.full(shape, 0.0 if leaf == "A_log" else 0.5 if leaf == "alpha" else 1.0, device=device)
-            if len(shape) < 2:
-                return torch.zeros(shape, device=device)
-            return torch.randn(shape, generator=gen, device=device) * (1.0 if name == "embed" else shape[1] ** -0.5)
-        model._load(take, dtype, torch.device(device))
-        return model
+    @staticmethod
+    def random_tensor(name, shape, gen, device):
+        leaf = name.rsplit(".", 1)[-1]
+        if leaf in ("alpha", "A_log") or leaf.startswith(("ls", "norm")):
+            return torch.full(shape, 0.0 if leaf == "A_log" else 0.5 if leaf == "alpha" else 1.0, device=device)
+        if len(shape) < 2:
+            return torch.zeros(shape, device=device)
+        return torch.randn(shape, generator=gen, device=device) * (1.0 if name == "embed" else shape[1] ** -0.5)
 
     @torch.no_grad()
-    def _load(self, take: Callable[[str], torch.Tensor], dtype, device) -> None:
+    def _load(self, take, dtype, device) -> None:
         cfg = self.config
         D, Dp = cfg.hidden_size, pad8(cfg.hidden_size)
         self.register_parameter("embed", nn.Parameter(padded(take("embed"), cfg.vocab_size, Dp, dtype, device), requires_grad=False))
@@ -155,25 +114,12 @@ class Vimodra(nn.Module):
             self.adds.append(add)
 
     # -- forward ----------------------------------------------------------------------------------------------
-    def make_cache(self, batch: int, max_len: int, dtype=None, device=None) -> LayerStateCache:
-        dtype, device = dtype or self.embed.dtype, device or self.embed.device
-        return LayerStateCache(batch, max_len, device, [self.mixers[i].state(batch, max_len, dtype, device) for i, _ in self.runs])
+    def layer_states(self, batch: int, max_len: int, dtype, device) -> List[Dict[str, torch.Tensor]]:
+        return [self.mixers[i].state(batch, max_len, dtype, device) for i, _ in self.runs]
 
     def hidden_states(self, input_ids: torch.Tensor, cache: LayerStateCache, collect: Optional[List[torch.Tensor]] = None) -> torch.Tensor:
-        """Runs the tokens [B, L] that follow what ``cache`` holds -> normed hidden states [B * L, padded width].  ``collect`` receives the
-        residual stream [B, L, width] after every layer run."""
         B, L = input_ids.shape
-        on_device = cache.device_lengths is not None and L == 1   # graph-replayed (or pool) decode: positions live on the device
-        if not on_device and cache.length + L > cache.max_len:
-            raise RuntimeError(f"cache overflow: {cache.length}+{L} > {cache.max_len}")
-        for rope in self._ropes.values():
-            rope.ensure(cache.max_len, self.embed.device)
-        if on_device:
-            step = Step(B, 1, 0, cache.device_lengths, cache.device_active)
-        elif L == 1:
-            step = Step(B, 1, cache.length, torch.full((B,), cache.length, dtype=torch.int32, device=self.embed.device))
-        else:
-            step = Step(B, L, cache.length)
+        step = self._step(input_ids, cache)
         x, h = dyt_ops.embed_norm(input_ids.reshape(-1), self.embed, self.first_add, *self.first_norm)
         for r, (i, _) in enumerate(self.runs):
             mixer, (after_mixer, after_mlp) = self.mixers[i], self.chains[r]
@@ -184,35 +130,6 @@ class Vimodra(nn.Module):
             if collect is not None:
                 s = x if self.adds[r] is None else x - self.adds[r]
                 collect.append(s[:, :self.config.hidden_size].reshape(B, L, -1).clone())
-        if not on_device:
+        if not step.on_device:
             cache.advance(L)
         return h
-
-    def forward(self, input_ids: torch.Tensor, attention_mask: Optional[torch.Tensor] = None, return_aux_loss: Optional[bool] = None,
-                cache: Optional[LayerStateCache] = None, last_token_only: bool = False, logits_at: Optional[Sequence[int]] = None,
-                collect: Optional[List[torch.Tensor]] = None) -> torch.Tensor:
-        """-> fp32 logits [B, n, vocab] of all positions, of the last one, or of the positions ``logits_at``."""
-        if attention_mask is not None:
-            raise ValueError("sequences of a batch have equal length here: no attention mask")
-        B, L = input_ids.shape
-        if cache is None:
-            cache = self.make_cache(B, L)
-        h = self.hidden_states(input_ids, cache, collect).view(B, L, -1)
-        if last_token_only:
-            h = h[:, -1:]
-        elif logits_at is not None:
-            h = h[:, list(logits_at)]
-        n = h.shape[1]
-        h = h.reshape(B * n, -1)
-        logits = G.gemm_nt(h, self.head, out_fp32=True) if ops._lib.use_cuda_kernels(h) else ops.linear(h, self.head).float()
-        return logits.view(B, n, -1)[..., :self.config.vocab_size]
-
-    # -- statistics ---------------------------------------------------------------------------------------------
-    def num_parameters(self, trainable_only: bool = False) -> int:
-        n = 0
-        for shape in self.tensor_shapes().values():
-            k = 1
-            for d in shape:
-                k *= d
-            n += k
-        return 0 if trainable_only else n

@@ -34,7 +34,7 @@ HOST_LIB = os.path.join(OUT_DIR, "libats_host.so")
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
               "-Xcompiler", "-fPIC", "-Xcompiler", "-fvisibility=hidden"]
 # Every source is compiled with --use_fast_math except these: their kernels also serve models that run in true 32-bit.
-PRECISE_MATH = {"dyt.cu", "latent_attention.cu", "delta_rule.cu"}
+PRECISE_MATH = {"dyt.cu", "latent_attention.cu", "delta_rule.cu", "channel_delta.cu", "lightning.cu", "gqa_attention.cu", "postnorm.cu"}
 # Kernels that may only run in single-GPU jobs (none at present) would be listed here and built into a
 # separate library so the main one never names a multicast load.
 SINGLE_GPU_ONLY: List[str] = []

@@ -55,6 +55,38 @@ class DeltaShape:
         return self.b_col + pad8(self.heads)
 
 
+@dataclass(frozen=True)
+class ChannelDeltaShape(DeltaShape):
+    """One decay per state row, and a sigmoid output gate, both behind low-rank projections: the input projection is [q | k | v | decay
+    input | gate input | b], and a second product expands [decay input | gate input] to [decays | gate]."""
+    decay_rank: int = 8
+    gate_rank: int = 8
+
+    @property
+    def low_col(self) -> int:      # of the low-rank inputs in the input projection
+        return pad8(self.channels)
+
+    @property
+    def g_low(self) -> int:        # of the gate's part inside them
+        return pad8(self.decay_rank)
+
+    @property
+    def low_width(self) -> int:
+        return self.g_low + pad8(self.gate_rank)
+
+    @property
+    def b_col(self) -> int:
+        return self.low_col + self.low_width
+
+    @property
+    def g_col(self) -> int:        # of the gate in the second product (the decays start at 0)
+        return pad8(self.heads * self.dim)
+
+    @property
+    def scan_rows(self) -> int:    # state rows the portion kernel is built for
+        return 64 if self.dim <= 64 else 128 if self.dim <= 128 else 256
+
+
 class _Prep(ctypes.Structure):
     _fields_ = [("proj", _vp), ("ld", _cll), ("g_col", _ci), ("a_col", _ci), ("b_col", _ci), ("B", _ci), ("L", _ci), ("H", _ci), ("KH", _ci), ("dim", _ci),
                 ("vdim", _ci), ("taps", _ci), ("C", _ci), ("conv", _vp), ("neg_rate", _vp), ("dt_bias", _vp), ("tail", _vp), ("tail_bs", _cll), ("pos0", _ci),
@@ -68,12 +100,19 @@ class _Scan(ctypes.Structure):
 
 class _Out(ctypes.Structure):
     _fields_ = [("o", _vp), ("ldo", _cll), ("gate", _vp), ("ldg", _cll), ("w", _vp), ("eps", _cf), ("out", _vp), ("ldout", _cll), ("rows", _cll), ("H", _ci),
-                ("vdim", _ci)]
+                ("vdim", _ci), ("gate_sigmoid", _ci)]
 
 
 class _Step(ctypes.Structure):
     _fields_ = [("mixed", _vp), ("ldm", _cll), ("rlen", _vp), ("gb", _vp), ("state", _vp), ("state_bs", _cll), ("lengths", _vp), ("active", _vp), ("gate", _vp),
-                ("ldg", _cll), ("w", _vp), ("eps", _cf), ("out", _vp), ("ldout", _cll), ("B", _ci), ("H", _ci), ("KH", _ci), ("dim", _ci), ("vdim", _ci)]
+                ("ldg", _cll), ("w", _vp), ("eps", _cf), ("out", _vp), ("ldout", _cll), ("B", _ci), ("H", _ci), ("KH", _ci), ("dim", _ci), ("vdim", _ci),
+                ("gate_sigmoid", _ci), ("a", _vp), ("lda", _cll), ("neg_rate", _vp), ("dt_bias", _vp)]
+
+
+class _Channel(ctypes.Structure):
+    _fields_ = [("mixed", _vp), ("ldm", _cll), ("rlen", _vp), ("gb", _vp), ("a", _vp), ("lda", _cll), ("neg_rate", _vp), ("dt_bias", _vp), ("coef", _vp), ("state", _vp),
+                ("state_bs", _cll), ("o", _vp), ("ldo", _cll), ("B", _ci), ("L", _ci), ("H", _ci), ("KH", _ci), ("dim", _ci), ("vdim", _ci), ("groups", _ci),
+                ("fresh", _ci), ("DK", _ci)]
 
 
 # ----------------------------------------------------------------------------------------------------------
@@ -88,8 +127,8 @@ def _unit_qk(mixed: torch.Tensor, rlen: torch.Tensor, s: DeltaShape):
 
 
 def _advance(S: torch.Tensor, q, k, v, g, beta):
-    """One token of one sequence; S [H, dim, vdim] fp32 -> (new S, read-out [H, vdim])."""
-    S = S * g[:, None, None]
+    """One token of one sequence; S [H, dim, vdim] fp32, g [H] or [H, dim] -> (new S, read-out [H, vdim])."""
+    S = S * (g[:, None, None] if g.dim() == 1 else g[:, :, None])
     u = beta[:, None] * (v - torch.einsum("hdv,hd->hv", S, k))
     S = S + k[:, :, None] * u[:, None, :]
     return S, torch.einsum("hdv,hd->hv", S, q)
@@ -99,15 +138,22 @@ def _norm_gate(o: torch.Tensor, gate: torch.Tensor, w: torch.Tensor, s: DeltaSha
     rows = o.shape[0]
     o = o.float().view(rows, s.heads, s.vdim)
     o = o / torch.sqrt(o.pow(2).mean(-1, keepdim=True) + s.eps) * w
-    out[:, :s.heads * s.vdim] = (o.reshape(rows, -1) * torch.nn.functional.silu(gate[:, :s.heads * s.vdim].float())).to(out.dtype)
+    act = torch.sigmoid if isinstance(s, ChannelDeltaShape) else torch.nn.functional.silu
+    out[:, :s.heads * s.vdim] = (o.reshape(rows, -1) * act(gate[:, :s.heads * s.vdim].float())).to(out.dtype)
+
+
+def _row_decays(a: torch.Tensor, neg_rate: torch.Tensor, dt_bias: torch.Tensor, s: ChannelDeltaShape) -> torch.Tensor:
+    """a [rows, >= heads * dim] -> decays [rows, heads, dim]."""
+    z = torch.nn.functional.softplus(a[:, :s.heads * s.dim].float() + dt_bias)
+    return torch.exp(neg_rate[:, None] * z.view(-1, s.heads, s.dim))
 
 
 # ----------------------------------------------------------------------------------------------------------
 # operators
 # ----------------------------------------------------------------------------------------------------------
-def delta_prep(proj: torch.Tensor, s: DeltaShape, conv: torch.Tensor, neg_rate: torch.Tensor, dt_bias: torch.Tensor, tail: torch.Tensor, pos0: int = 0,
-               lengths: Optional[torch.Tensor] = None, active: Optional[torch.Tensor] = None) -> Tuple[torch.Tensor, torch.Tensor, torch.Tensor]:
-    """proj [B, L, proj_width]; conv [taps, channels] (last row: current token), neg_rate = -exp(A_log), dt_bias [H] in fp32; tail [B, taps - 1, channels] ->
+def delta_prep(proj: torch.Tensor, s: DeltaShape, conv: torch.Tensor, neg_rate: Optional[torch.Tensor], dt_bias: Optional[torch.Tensor], tail: torch.Tensor,
+               pos0: int = 0, lengths: Optional[torch.Tensor] = None, active: Optional[torch.Tensor] = None) -> Tuple[torch.Tensor, torch.Tensor, torch.Tensor]:
+    """proj [B, L, proj_width]; with a :class:`ChannelDeltaShape` neg_rate and dt_bias are ``None`` and no decays are computed; conv [taps, channels] (last row: current token), neg_rate = -exp(A_log), dt_bias [H] in fp32; tail [B, taps - 1, channels] ->
     (mixed [B * L, .], reciprocal lengths [B * L, 2 kv_heads], [decay, step size] [B * L, 2 H]); the tail moves on by the portion."""
     B, L, _ = proj.shape
     H, KH, C, n = s.heads, s.kv_heads, s.channels, s.taps - 1
@@ -124,8 +170,9 @@ def delta_prep(proj: torch.Tensor, s: DeltaShape, conv: torch.Tensor, neg_rate: 
         qk = mixed[:, :2 * KH * s.dim].view(B * L, 2 * KH, s.dim).float()
         rlen = 1 / torch.sqrt(qk.pow(2).sum(-1) + 1e-6)
         rlen[:, :KH] *= s.dim ** -0.5
-        a = proj[..., s.a_col:s.a_col + H].float().reshape(B * L, H) + dt_bias
-        g = torch.exp(neg_rate * torch.nn.functional.softplus(a))
+        g = torch.zeros(B * L, H)
+        if neg_rate is not None:
+            g = torch.exp(neg_rate * torch.nn.functional.softplus(proj[..., s.a_col:s.a_col + H].float().reshape(B * L, H) + dt_bias))
         beta = torch.sigmoid(proj[..., s.b_col:s.b_col + H].float().reshape(B * L, H))
         return mixed, rlen, torch.cat([g, beta], dim=-1)
     assert proj.stride(2) == 1 and proj.stride(0) == L * proj.stride(1) and (n == 0 or tail.stride(1) == C)
@@ -169,21 +216,25 @@ def delta_output(o: torch.Tensor, gate: torch.Tensor, w: torch.Tensor, s: DeltaS
         _norm_gate(o, gate, w, s, out)
         return out
     out = torch.empty(rows, s.o_pad, dtype=o.dtype, device=o.device)
-    _call("ats_delta_output", _Out(_p(o), o.stride(0), _p(gate), gate.stride(0), _p(w), s.eps, _p(out), out.stride(0), rows, s.heads, s.vdim), o)
+    _call("ats_delta_output", _Out(_p(o), o.stride(0), _p(gate), gate.stride(0), _p(w), s.eps, _p(out), out.stride(0), rows, s.heads, s.vdim,
+                                    int(isinstance(s, ChannelDeltaShape))), o)
     return out
 
 
 def delta_step(mixed: torch.Tensor, rlen: torch.Tensor, gb: torch.Tensor, state: torch.Tensor, gate: torch.Tensor, w: torch.Tensor, s: DeltaShape,
-               lengths: torch.Tensor, active: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """One token per sequence: state update, read-out, output norm and gate -> [B, o_pad]."""
+               lengths: torch.Tensor, active: Optional[torch.Tensor] = None, a: Optional[torch.Tensor] = None, neg_rate: Optional[torch.Tensor] = None,
+               dt_bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """One token per sequence: state update, read-out, output norm and gate -> [B, o_pad].  With a :class:`ChannelDeltaShape` the decays
+    come from their input ``a`` [B, >= heads * dim], neg_rate [heads] and dt_bias [heads * dim]."""
     B, H = state.shape[0], s.heads
     if not mixed.is_cuda:
         q, k, v = _unit_qk(mixed, rlen, s)
         out = torch.zeros(B, s.o_pad, dtype=mixed.dtype)
         o = torch.empty(B, H * s.vdim)
+        decay = gb[:, :H] if a is None else _row_decays(a, neg_rate, dt_bias, s)
         for b in range(B):
             S = torch.zeros_like(state[b]) if int(lengths[b]) == 0 else state[b]
-            S, r = _advance(S, q[b], k[b], v[b], gb[b, :H], gb[b, H:])
+            S, r = _advance(S, q[b], k[b], v[b], decay[b], gb[b, H:])
             if active is None or int(active[b]):
                 state[b] = S
             o[b] = r.reshape(-1)
@@ -191,5 +242,28 @@ def delta_step(mixed: torch.Tensor, rlen: torch.Tensor, gb: torch.Tensor, state:
         return out
     out = torch.empty(B, s.o_pad, dtype=mixed.dtype, device=mixed.device)
     _call("ats_delta_step", _Step(_p(mixed), mixed.stride(0), _p(rlen), _p(gb), _p(state), state.stride(0), _p(lengths), _p(active), _p(gate), gate.stride(0), _p(w),
-                                  s.eps, _p(out), out.stride(0), B, H, s.kv_heads, s.dim, s.vdim), mixed)
+                                  s.eps, _p(out), out.stride(0), B, H, s.kv_heads, s.dim, s.vdim, int(isinstance(s, ChannelDeltaShape)), _p(a),
+                                  0 if a is None else a.stride(0), _p(neg_rate if a is not None else None), _p(dt_bias if a is not None else None)), mixed)
     return out
+
+
+def channel_delta_scan(mixed: torch.Tensor, rlen: torch.Tensor, gb: torch.Tensor, a: torch.Tensor, neg_rate: torch.Tensor, dt_bias: torch.Tensor, state: torch.Tensor,
+                       s: ChannelDeltaShape, L: int, fresh: bool) -> torch.Tensor:
+    """:func:`delta_scan` with one decay per state row (``csrc/channel_delta.cu``): a [B * L, >= heads * dim] decay inputs."""
+    B, H = state.shape[0], s.heads
+    if not mixed.is_cuda:
+        q, k, v = _unit_qk(mixed, rlen, s)
+        g, out = _row_decays(a, neg_rate, dt_bias, s), torch.empty(B * L, H * s.vdim, dtype=mixed.dtype)
+        for b in range(B):
+            S = torch.zeros_like(state[b]) if fresh else state[b]
+            for t in range(b * L, (b + 1) * L):
+                S, o = _advance(S, q[t], k[t], v[t], g[t], gb[t, H:])
+                out[t] = o.reshape(-1).to(out.dtype)
+            state[b] = S
+        return out
+    groups, DK = (L + GROUP - 1) // GROUP, s.scan_rows
+    coef = torch.empty(B, groups, H, 2 * GROUP * GROUP + (3 * GROUP + 1) * DK, dtype=torch.float32, device=mixed.device)   # layout: csrc/channel_delta.cu
+    o = torch.empty(B * L, H * s.vdim, dtype=mixed.dtype, device=mixed.device)
+    _call("ats_channel_delta", _Channel(_p(mixed), mixed.stride(0), _p(rlen), _p(gb), _p(a), a.stride(0), _p(neg_rate), _p(dt_bias), _p(coef), _p(state), state.stride(0),
+                                        _p(o), o.stride(0), B, L, H, s.kv_heads, s.dim, s.vdim, groups, int(fresh), DK), mixed)
+    return o

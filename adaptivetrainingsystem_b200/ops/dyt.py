@@ -30,7 +30,7 @@ def _fns():
     if not _sig:
         for name, args in (("ats_fold_dyt", [_vp, _ci, _cll, _vp, _vp, _vp, _vp, _cf, _vp, _vp, _cf, _vp, _ci, _cll, _ci, _vp]),
                            ("ats_fold_gelu", [_vp, _ci, _cll, _vp, _vp, _ci, _cll, _ci, _vp]),
-                           ("ats_gemm_bf16_block", [_vp, _cll, _vp, _cll, _vp, _ci, _ci, _ci, _ci, _vp, _vp, _ci, _vp, _vp, _cf, _vp, _vp, _cf, _vp, _ci, _vp]),
+                           ("ats_gemm_bf16_block", [_vp, _cll, _vp, _cll, _vp, _ci, _ci, _ci, _ci, _vp, _vp, _ci, _vp, _vp, _cf, _vp, _vp, _cf, _ci, _vp, _ci, _vp]),
                            ("ats_embed_dyt", [_vp, _vp, _ci, _ci, _vp, _vp, _vp, _vp, _cf, _vp, _cll, _ci, _vp])):
             f = getattr(lib, name)
             f.restype, f.argtypes = _ci, args
@@ -100,7 +100,7 @@ def _block_gemm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: Optio
     (T, K), N = a.shape, w.shape[0]
     w1, b1, a1, w2, b2, a2 = (c.w1, c.b1, c.a1, c.w2, c.b2, c.a2) if c is not None else (None, None, 0.0, None, None, 0.0)
     _lib.check(_fns().ats_gemm_bf16_block(_lib.ptr(a), a.stride(0), _lib.ptr(w), w.stride(0), _lib.ptr(out), out.stride(0), T, N, K, _lib.ptr(bias), _lib.ptr(x),
-                                          0 if x is None else x.stride(0), _lib.ptr(w1), _lib.ptr(b1), a1, _lib.ptr(w2), _lib.ptr(b2), a2,
+                                          0 if x is None else x.stride(0), _lib.ptr(w1), _lib.ptr(b1), a1, _lib.ptr(w2), _lib.ptr(b2), a2, -1,
                                           _lib.ptr(_lib.status_tensor(a.device)), 0, _lib.stream_ptr(a.device)), "ats_gemm_bf16_block")
 
 

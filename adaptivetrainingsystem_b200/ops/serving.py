@@ -27,6 +27,8 @@ def _fns():
         lib.ats_decode_attn_chunks.argtypes = [_ci]
         lib.ats_decode_attn.restype = _ci
         lib.ats_decode_attn.argtypes = [_vp, _cll, _ci, _ci, _ci, _vp, _vp, _cll, _vp, _ci, _ci, _ci, _ci, _ci, _ci, _ci, _vp, _vp, _vp, _vp, _vp]
+        lib.ats_decode_attn_cached.restype = _ci
+        lib.ats_decode_attn_cached.argtypes = [_vp, _cll, _vp, _vp, _cll, _vp, _ci, _ci, _ci, _ci, _ci, _cf, _cf, _vp, _cll, _vp, _vp, _vp, _vp, _cll, _vp]
         lib.ats_fold_rope.restype = _ci
         lib.ats_fold_rope.argtypes = [_vp, _ci, _vp, _vp, _vp, _vp, _ci, _ci, _ci, _ci, _ci, _vp]
         lib.ats_fold_add_norm.restype = _ci
@@ -150,6 +152,28 @@ def decode_attention(qkv: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Te
                               _lib.stream_ptr(qkv.device))
     _lib.check(err, "ats_decode_attn")
     return out
+
+
+MAX_COUNTERS = 1 << 16   # (sequence, key head) pairs of one decode_attention_cached call
+
+
+def decode_attention_cached(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, lengths: torch.Tensor, n_q: int, n_kv: int, d: int, scale: float,
+                            cap: float, gate: Optional[torch.Tensor], out: torch.Tensor) -> None:
+    """The kernel of :func:`decode_attention` for a cache [B, max_len, n_kv * d] that holds the new token's row already: q [B, >= n_q d]
+    (prepared), lengths int32 [B] (position of the new token), ``cap`` > 0: scores become ``cap tanh(score / cap)``, gate [B, .] (strided view,
+    one column per head) or ``None`` -> out [B, >= n_q d], merged and gated in the same launch."""
+    B, max_len, dev = q.shape[0], k_cache.shape[1], q.device
+    lib = _fns()
+    chunks = lib.ats_decode_attn_chunks(max_len)
+    part_o = torch.empty(B * n_q * chunks * d, dtype=torch.float32, device=dev)
+    part_ml = torch.empty(B * n_q * chunks * 2, dtype=torch.float32, device=dev)
+    done = _scratch.get(("dec_cached_cnt", dev.index))
+    if done is None:
+        # arrival counters, back at zero after every launch; one allocation for good, because captured graphs keep its address
+        done = _scratch[("dec_cached_cnt", dev.index)] = torch.zeros(MAX_COUNTERS, dtype=torch.int32, device=dev)
+    _lib.check(lib.ats_decode_attn_cached(_lib.ptr(q), q.stride(0), _lib.ptr(k_cache), _lib.ptr(v_cache), k_cache.stride(0), _lib.ptr(lengths), B, n_q, n_kv, d, max_len,
+                                          scale, cap, _lib.ptr(gate), 0 if gate is None else gate.stride(0), _lib.ptr(part_o), _lib.ptr(part_ml), _lib.ptr(done),
+                                          _lib.ptr(out), out.stride(0), _lib.stream_ptr(dev)), "ats_decode_attn_cached")
 
 
 def decode_attention_reference(qkv, k_cache, v_cache, length, n_q, n_kv, d) -> torch.Tensor:

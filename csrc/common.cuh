@@ -432,6 +432,9 @@ EncodeTiledFn get_encode_tiled();
 // 128-byte swizzle. Returns 0 on success.
 int make_tmap_2d(CUtensorMap* out, const void* base, uint64_t rows, uint64_t cols, uint64_t ld, int elem_bytes,
                  uint32_t box_cols, uint32_t box_rows);
+// The same for bf16 rows of `heads` heads of `dim` columns each, box = 64 columns x 1 head x 128 rows: columns at and beyond `dim` read
+// as zero, so a head that is not a whole number of 64-column pieces does not run into the next one (dim a multiple of 8).
+int make_tmap_heads(CUtensorMap* out, const void* base, uint64_t rows, uint64_t heads, uint64_t dim, uint64_t ld);
 
 // ----------------------------------------------------------------------------------------------
 // Programmatic dependent launch for chains of short kernels (the decode step: ~17 dependent launches of a few microseconds per

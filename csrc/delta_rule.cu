@@ -15,8 +15,11 @@
 // * delta_output: output norm over vdim, weight, silu gate.
 // * delta_step: one decoded token per sequence: state read once and written once, output norm and gate in the same launch.
 //
+// channel_delta.cu holds the portion kernels of the form with one decay per state row; it shares delta_prep (without the decays),
+// delta_output and delta_step.
+//
 // A sequence at position 0 starts from a zero state and zero convolution inputs whatever its buffers hold.
-#include "typed.cuh"
+#include "delta_common.cuh"
 
 namespace ats {
 
@@ -26,7 +29,7 @@ struct DeltaArgs {
   int g_col, a_col, b_col;
   int B, L, H, KH, dim, vdim, taps, C;   // C = 2 * KH * dim + H * vdim convolved channels
   const float* conv;       // [taps, C], last row = current token
-  const float* neg_rate;   // [H] -exp(A_log)
+  const float* neg_rate;   // [H] -exp(A_log), or null: step sizes only (the decays come from elsewhere)
   const float* dt_bias;    // [H]
   void* tail;              // [B, taps - 1, C] last inputs of the convolutions (oldest first)
   long long tail_bs;
@@ -42,9 +45,8 @@ struct DeltaArgs {
 template <typename T>
 __device__ __forceinline__ void delta_gate(const DeltaArgs& p, long long row, int h) {
   const T* in = static_cast<const T*>(p.proj) + row * p.ld;
-  const float a = Typed<T>::load(in + p.a_col + h) + p.dt_bias[h], bt = Typed<T>::load(in + p.b_col + h);
-  const float sp = a > 20.f ? a : log1pf(expf(a));
-  p.gb[row * 2 * p.H + h] = expf(p.neg_rate[h] * sp);
+  const float bt = Typed<T>::load(in + p.b_col + h);
+  if (p.neg_rate) p.gb[row * 2 * p.H + h] = decay_of(Typed<T>::load(in + p.a_col + h) + p.dt_bias[h], p.neg_rate[h]);
   p.gb[row * 2 * p.H + p.H + h] = 1.f / (1.f + expf(-bt));
 }
 
@@ -203,7 +205,6 @@ __global__ void __launch_bounds__(256) delta_tail_kernel(const DeltaArgs p) {
 }
 
 // ------------------------------------------------------------------------------------------------ portions
-constexpr int DC = 8;  // tokens per group
 // Per group and head: [DC][2 * DC] inverse of the triangular system (times beta) and read-out coefficients, then per token
 // G_i / |k_i|, G_i dim^-1/2 / |q_i|, D_Ci / |k_i| (G_i = g_1 .. g_i, D_Ci = g_{i+1} .. g_C), then G_C: with the lengths folded in
 // here, the sequential kernel works on the raw q and k.
@@ -348,17 +349,6 @@ __global__ void __launch_bounds__(128) delta_pairs_kernel(const ScanArgs p) {
   }
 }
 
-__device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) { return __ffma2_rn(a, b, c); }  // one packed instruction
-// Keeps the compiler from requesting the shared-memory rows of more tokens than registers can hold.
-__device__ __forceinline__ void pace() { asm volatile("" ::: "memory"); }
-
-// One step of a transposing reduction over lanes: of the pair (lo, hi) this lane keeps hi when its bit `s` is set, else lo, and adds
-// what the lane across sends.
-__device__ __forceinline__ float keep_add(float lo, float hi, int lane, int s) {
-  const bool up = (lane & s) != 0;
-  return (up ? hi : lo) + __shfl_xor_sync(0xffffffffu, up ? lo : hi, s);
-}
-
 // A lane's EPL values of a k or q row in shared memory: pieces of up to eight consecutive elements, sixteen lanes side by side.
 template <typename T, int EPL>
 struct RowPiece {
@@ -387,11 +377,6 @@ struct RowPiece {
     }
   }
 };
-
-template <int BYTES> struct Bits;
-template <> struct Bits<4> { using type = uint32_t; };
-template <> struct Bits<8> { using type = uint2; };
-template <> struct Bits<16> { using type = uint4; };
 
 // Sixteen lanes share CPL value columns: lane l holds EPL state rows (dim <= 16 * EPL) of each.  CTA = 4 warps of 2 lane groups ->
 // 8 * CPL columns of one head.  k and q rows stay in the element type in shared memory: with the state spread over sixteen lanes and
@@ -611,6 +596,7 @@ struct DeltaOutArgs {
   long long ldout;
   long long rows;
   int H, vdim;
+  int gate_sigmoid;        // gate activation: 0 silu, 1 sigmoid
 };
 
 template <typename T>
@@ -632,7 +618,7 @@ __global__ void __launch_bounds__(256) delta_output_kernel(const DeltaOutArgs p)
   const float r = 1.f / sqrtf(warp_sum(ss) / float(p.vdim) + p.eps);
   for (int c = lane; c < p.vdim; c += 32) {
     const float z = Typed<T>::load(g + c);
-    Typed<T>::store(out + (long long)h * p.vdim + c, Typed<T>::load(o + c) * r * p.w[c] * z * Typed<T>::sigmoid_(z));
+    Typed<T>::store(out + (long long)h * p.vdim + c, Typed<T>::load(o + c) * r * p.w[c] * (p.gate_sigmoid ? 1.f : z) * Typed<T>::sigmoid_(z));
   }
   if (h == 0)
     for (int c = p.H * p.vdim + lane; c < p.ldout; c += 32) Typed<T>::store(out + c, 0.f);
@@ -655,7 +641,7 @@ __global__ void __launch_bounds__(256) delta_output_vec_kernel(const DeltaOutArg
   for (int off = lanes >> 1; off > 0; off >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, off);
   const float r = 1.f / sqrtf(ss / float(p.vdim) + p.eps);
 #pragma unroll
-  for (int e = 0; e < 8; ++e) v[e] *= r * p.w[c + e] * z[e] * Typed<T>::sigmoid_(z[e]);
+  for (int e = 0; e < 8; ++e) v[e] *= r * p.w[c + e] * (p.gate_sigmoid ? 1.f : z[e]) * Typed<T>::sigmoid_(z[e]);
   if (live) Typed<T>::store8(static_cast<T*>(p.out) + row * p.ldout + (long long)h * p.vdim + c, v);
 }
 
@@ -676,7 +662,21 @@ struct StepArgs {
   void* out;               // [B, ldout]
   long long ldout;
   int B, H, KH, dim, vdim;
+  int gate_sigmoid;        // gate activation: 0 silu, 1 sigmoid
+  // one decay per state row instead of one per head: exp(neg_rate[h] softplus(a[b, h * dim + d] + dt_bias[h * dim + d])); a null: gb's
+  const void* a;           // [B, lda]
+  long long lda;
+  const float* neg_rate;   // [H]
+  const float* dt_bias;    // [H * dim]
 };
+
+// Decays of the state rows of head h -> s_g [dim].
+template <typename T>
+__device__ __forceinline__ void row_decays(const StepArgs& p, int b, int h, float* s_g, int threads) {
+  const T* a = p.a ? static_cast<const T*>(p.a) + (long long)b * p.lda + (long long)h * p.dim : nullptr;
+  const float g = p.a ? 0.f : p.gb[(long long)b * 2 * p.H + h], rate = p.a ? p.neg_rate[h] : 0.f;
+  for (int d = threadIdx.x; d < p.dim; d += threads) s_g[d] = a ? decay_of(Typed<T>::load(a + d) + p.dt_bias[(long long)h * p.dim + d], rate) : g;
+}
 
 constexpr int ST_THREADS = 512;
 // One CTA per (head, sequence).  Threads are (row group, column): CW columns, 512 / CW row groups, RPT rows per thread in registers.
@@ -687,7 +687,8 @@ __global__ void __launch_bounds__(ST_THREADS) delta_step_kernel(const StepArgs p
   const int RG = ST_THREADS / CW, tid = threadIdx.x, c = tid % CW, rg = tid / CW, h = blockIdx.x, b = blockIdx.y;
   float* s_k = sm;                 // [dim]
   float* s_q = s_k + p.dim;        // [dim]
-  float* s_o = s_q + p.dim;        // [vdim]
+  float* s_g = s_q + p.dim;        // [dim]
+  float* s_o = s_g + p.dim;        // [vdim]
   float* s_r = s_o + p.vdim;       // [RG][CW]
   float* s_red = s_r + ST_THREADS; // [40]
   const int kh = h / (p.H / p.KH);
@@ -698,7 +699,8 @@ __global__ void __launch_bounds__(ST_THREADS) delta_step_kernel(const StepArgs p
     s_k[d] = Typed<T>::load(mixed + (long long)(p.KH + kh) * p.dim + d) * rk;
     s_q[d] = Typed<T>::load(mixed + (long long)kh * p.dim + d) * rq;
   }
-  const float g = p.gb[(long long)b * 2 * p.H + h], beta = p.gb[(long long)b * 2 * p.H + p.H + h];
+  row_decays<T>(p, b, h, s_g, ST_THREADS);
+  const float beta = p.gb[(long long)b * 2 * p.H + p.H + h];
   float* st = p.state + (long long)b * p.state_bs + (long long)h * p.dim * p.vdim;
   __syncthreads();
   float ss = 0.f;
@@ -709,7 +711,7 @@ __global__ void __launch_bounds__(ST_THREADS) delta_step_kernel(const StepArgs p
 #pragma unroll
     for (int i = 0; i < RPT; ++i) {
       const int d = rg + i * RG;
-      S[i] = (ok && d < p.dim && !fresh) ? st[(long long)d * p.vdim + v] * g : 0.f;
+      S[i] = (ok && d < p.dim && !fresh) ? st[(long long)d * p.vdim + v] * s_g[d] : 0.f;
     }
 #pragma unroll
     for (int i = 0; i < RPT; ++i) {
@@ -748,7 +750,7 @@ __global__ void __launch_bounds__(ST_THREADS) delta_step_kernel(const StepArgs p
   const T* gt = static_cast<const T*>(p.gate) + (long long)b * p.ldg + (long long)h * p.vdim;
   for (int v = tid; v < p.vdim; v += ST_THREADS) {
     const float z = Typed<T>::load(gt + v);
-    Typed<T>::store(out + (long long)h * p.vdim + v, s_o[v] * r * p.w[v] * z * Typed<T>::sigmoid_(z));
+    Typed<T>::store(out + (long long)h * p.vdim + v, s_o[v] * r * p.w[v] * (p.gate_sigmoid ? 1.f : z) * Typed<T>::sigmoid_(z));
   }
   if (h == 0)
     for (int v = p.H * p.vdim + tid; v < p.ldout; v += ST_THREADS) Typed<T>::store(out + v, 0.f);
@@ -764,14 +766,15 @@ __global__ void __launch_bounds__(SV_THREADS, RPT <= 8 ? 4 : RPT <= 16 ? 2 : 1) 
   float4* s_r = reinterpret_cast<float4*>(smv);                   // [8][32]
   float* s_k = smv + 8 * 32 * 4;                                  // [dim]
   float* s_q = s_k + p.dim;                                       // [dim]
-  float* s_o = s_q + p.dim;                                       // [vdim]
+  float* s_g = s_q + p.dim;                                       // [dim]
+  float* s_o = s_g + p.dim;                                       // [vdim]
   float* s_red = s_o + p.vdim;                                    // [40]
   const int kh = h / (p.H / p.KH);
   const bool fresh = p.lengths[b] == 0, keep = !(p.active && !p.active[b]);
   const T* mixed = static_cast<const T*>(p.mixed) + (long long)b * p.ldm;
   float* st = p.state + (long long)b * p.state_bs + (long long)h * p.dim * p.vdim;
   const float rq = p.rlen[(long long)b * 2 * p.KH + kh], rk = p.rlen[(long long)b * 2 * p.KH + p.KH + kh];
-  const float g = p.gb[(long long)b * 2 * p.H + h], beta = p.gb[(long long)b * 2 * p.H + p.H + h];
+  const float beta = p.gb[(long long)b * 2 * p.H + p.H + h];
   float ss = 0.f;
   for (int v0 = 0; v0 < p.vdim; v0 += 128) {
     const int v = v0 + c * 4;
@@ -787,14 +790,15 @@ __global__ void __launch_bounds__(SV_THREADS, RPT <= 8 ? 4 : RPT <= 16 ? 2 : 1) 
         s_k[d] = Typed<T>::load(mixed + (long long)(p.KH + kh) * p.dim + d) * rk;
         s_q[d] = Typed<T>::load(mixed + (long long)kh * p.dim + d) * rq;
       }
+      row_decays<T>(p, b, h, s_g, SV_THREADS);
       __syncthreads();
     }
     float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
     for (int i = 0; i < RPT; ++i) {
       const int d = rg + i * 8;
+      const float g = d < p.dim ? s_g[d] : 0.f, k = d < p.dim ? s_k[d] : 0.f;
       S[i].x *= g; S[i].y *= g; S[i].z *= g; S[i].w *= g;
-      const float k = d < p.dim ? s_k[d] : 0.f;
       a.x += S[i].x * k; a.y += S[i].y * k; a.z += S[i].z * k; a.w += S[i].w * k;
     }
     s_r[rg * 32 + c] = a;
@@ -843,7 +847,7 @@ __global__ void __launch_bounds__(SV_THREADS, RPT <= 8 ? 4 : RPT <= 16 ? 2 : 1) 
   const T* gt = static_cast<const T*>(p.gate) + (long long)b * p.ldg + (long long)h * p.vdim;
   for (int v = tid; v < p.vdim; v += SV_THREADS) {
     const float z = Typed<T>::load(gt + v);
-    Typed<T>::store(out + (long long)h * p.vdim + v, s_o[v] * r * p.w[v] * z * Typed<T>::sigmoid_(z));
+    Typed<T>::store(out + (long long)h * p.vdim + v, s_o[v] * r * p.w[v] * (p.gate_sigmoid ? 1.f : z) * Typed<T>::sigmoid_(z));
   }
   if (h == 0)
     for (int v = p.H * p.vdim + tid; v < p.ldout; v += SV_THREADS) Typed<T>::store(out + v, 0.f);
@@ -870,7 +874,7 @@ static int launch_scan(const ScanArgs& p, cudaStream_t s) {
 template <typename T>
 static int launch_step(const StepArgs& p, cudaStream_t s) {
   if ((p.vdim & 3) == 0 && p.dim <= 256 && (p.state_bs & 3) == 0 && (reinterpret_cast<uintptr_t>(p.state) & 15) == 0) {
-    const size_t sm = size_t(8 * 32 * 4 + 2 * p.dim + p.vdim + 40) * sizeof(float);
+    const size_t sm = size_t(8 * 32 * 4 + 3 * p.dim + p.vdim + 40) * sizeof(float);
     if (sm <= 48 * 1024) {
       const dim3 vgrid(p.H, p.B);
       if (p.dim <= 64) launch_pdl(delta_step_vec_kernel<T, 8>, vgrid, dim3(SV_THREADS), sm, s, p);
@@ -882,7 +886,7 @@ static int launch_step(const StepArgs& p, cudaStream_t s) {
   int CW = 32;
   while (CW < p.vdim && CW < 128) CW *= 2;
   const int rg = ST_THREADS / CW, rows = (p.dim + rg - 1) / rg;
-  const size_t smem = size_t(2 * p.dim + p.vdim + ST_THREADS + 40) * sizeof(float);
+  const size_t smem = size_t(3 * p.dim + p.vdim + ST_THREADS + 40) * sizeof(float);
   if (smem > 48 * 1024) return 1010;
   const dim3 grid(p.H, p.B);
   if (rows <= 8) launch_pdl(delta_step_kernel<T, 8>, grid, dim3(ST_THREADS), smem, s, p, CW);

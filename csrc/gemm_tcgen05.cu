@@ -36,7 +36,7 @@ constexpr int GEMM_THREADS = 256;  // TMA, MMA, 4 epilogue warps, 2 copy warps (
 constexpr int MAX_GROUPS = 256;
 constexpr int GEMM_SMEM_BYTES = STAGES * STAGE_BYTES + 1024 /*align*/ + 256 /*barriers*/ + (MAX_GROUPS + 1) * 4;
 
-enum Epilogue : int { kStore = 0, kAddC = 1, kF32 = 2, kSwiGLU = 3, kSwiGLUBwd = 4, kGelu = 5, kDyt = 6 };
+enum Epilogue : int { kStore = 0, kAddC = 1, kF32 = 2, kSwiGLU = 3, kSwiGLUBwd = 4, kGelu = 5, kDyt = 6, kSilu = 7 };
 
 struct GemmArgs {
   int M, N, K;
@@ -60,6 +60,8 @@ struct GemmArgs {
   int k_segs;            // ragged == 2: the reduction of group g runs over k_segs blocks of rows, seg_stride apart,
   int seg_stride;        //              block s holding counts[g * k_segs + s] rows
   void* const* d_table;  // optional per-group output base pointers (e.g. buffers on peer GPUs)
+  // kSilu: D = silu(acc) in the first act_cols columns (a multiple of 8), acc in the others.
+  int act_cols;
   // kGelu: D = gelu_tanh(acc + bias).  kDyt: the residual step of a block with Dynamic-Tanh norms, x <- x + tanh(a1 (acc + bias)) w1 + b1,
   // D = tanh(a2 x) w2 + b2, with x fp32 [M, ldx] (csrc/dyt.cu is the stand-alone form).  All vectors fp32 [N]; bias may be null.
   const float* bias;
@@ -312,7 +314,7 @@ __device__ __forceinline__ void epilogue_tile(const GemmArgs& p, const TileCoord
         }
       }
     }
-  } else if (p.epilogue == kGelu || p.epilogue == kDyt) {
+  } else if (p.epilogue == kGelu || p.epilogue == kDyt || p.epilogue == kSilu) {
     const bool dyt = p.epilogue == kDyt;
     __nv_bfloat16* drow = p.D + (long long)row * p.ldd;
     float* xrow = dyt ? p.x + (long long)row * p.ldx : nullptr;
@@ -355,6 +357,10 @@ __device__ __forceinline__ void epilogue_tile(const GemmArgs& p, const TileCoord
             f[4 * q + 3] = tanh_fast(p.a2 * xf[4 * q + 3]) * w2.w + b2.w;
           }
           st_global_32B(xrow + col, xq[2 * v], xq[2 * v + 1]);
+        } else if (p.epilogue == kSilu) {
+          if (col < p.act_cols)
+#pragma unroll
+            for (int e = 0; e < 8; ++e) f[e] = __fdividef(f[e], 1.f + __expf(-f[e]));
         } else {
 #pragma unroll
           for (int e = 0; e < 8; ++e) f[e] = 0.5f * f[e] * (1.f + tanh_fast(0.7978845608028654f * (f[e] + 0.044715f * f[e] * f[e] * f[e])));
@@ -1070,6 +1076,19 @@ int make_tmap_2d(CUtensorMap* out, const void* base, uint64_t rows, uint64_t col
   return r == CUDA_SUCCESS ? 0 : 1100 + int(r);
 }
 
+int make_tmap_heads(CUtensorMap* out, const void* base, uint64_t rows, uint64_t heads, uint64_t dim, uint64_t ld) {
+  EncodeTiledFn enc = get_encode_tiled();
+  if (!enc) return 1000;
+  if ((reinterpret_cast<uintptr_t>(base) & 15) || (dim & 7) || (ld & 7)) return 1001;
+  cuuint64_t dims[3] = {dim, heads, rows};
+  cuuint64_t strides[2] = {dim * 2, ld * 2};
+  cuuint32_t box[3] = {64, 1, 128};
+  cuuint32_t estr[3] = {1, 1, 1};
+  CUresult r = enc(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                   CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  return r == CUDA_SUCCESS ? 0 : 1100 + int(r);
+}
+
 static int g_num_sms = 0;
 static int num_sms() {
   if (!g_num_sms) {
@@ -1162,7 +1181,7 @@ ATS_API int ats_gemm_bf16(const void* A, long long a_rows, long long a_cols, lon
   p.n_copy = 0; p.n_rot = 0; p.own_row0 = 0; p.own_rows = 0; p.prof = g_gemm_prof;
   p.n_edge = 0; p.edge_chunk[0] = p.edge_chunk[1] = -1;
   p.out2 = nullptr; p.ldout2 = 0; p.out2_gs = 0;
-  if (epilogue == kGelu || epilogue == kDyt) return 1004;  // ats_gemm_bf16_block
+  if (epilogue == kGelu || epilogue == kDyt || epilogue == kSilu) return 1004;  // ats_gemm_bf16_block
   if (epilogue == kSwiGLUBwd) {
     // second output (h) travels in the C slot of this entry point: C / ldc / c_gs
     if (!aux || (up_offset & 7) || (ldaux & 7)) return 1004;
@@ -1172,16 +1191,18 @@ ATS_API int ats_gemm_bf16(const void* A, long long a_rows, long long a_cols, lon
   return launch_gemm(ma, mb, p, epilogue, groups, M, N, max_ctas, stream);
 }
 
-// D [M, N] = epilogue(A [M, K] B [N, K]^T), both operands K-major, with the element-wise block steps kGelu (x == nullptr) and kDyt.
+// D [M, N] = epilogue(A [M, K] B [N, K]^T), both operands K-major, with the element-wise block steps kSilu (act_cols >= 0), kGelu
+// (act_cols < 0, x == nullptr) and kDyt.
 ATS_API int ats_gemm_bf16_block(const void* A, long long lda, const void* B, long long ldb, void* D, int ldd, int M, int N, int K, const void* bias, void* x,
-                                int ldx, const void* w1, const void* b1, float a1, const void* w2, const void* b2, float a2, int* status, int max_ctas,
-                                void* stream) {
+                                int ldx, const void* w1, const void* b1, float a1, const void* w2, const void* b2, float a2, int act_cols, int* status,
+                                int max_ctas, void* stream) {
   static thread_local bool ctx_bound = false;
   if (!ctx_bound) {
     cudaFree(0);
     ctx_bound = true;
   }
   const bool dyt = x != nullptr;
+  if (act_cols >= 0 && ((act_cols & 7) || dyt || bias)) return 1004;
   if ((N & 7) || (ldd & 7) || K < 1 || (dyt && ((ldx & 7) || (reinterpret_cast<uintptr_t>(x) & 31) || !w1 || !b1 || !w2 || !b2))) return 1003;
   CUtensorMap ma, mb;
   int e;
@@ -1191,7 +1212,8 @@ ATS_API int ats_gemm_bf16_block(const void* A, long long lda, const void* B, lon
   p.M = M; p.N = N; p.K = K; p.groups = 1; p.b_div = 1; p.k_split = 1; p.k_segs = 1; p.alpha = 1.f;
   p.b_kblocks = int(K / 64);
   p.D = static_cast<__nv_bfloat16*>(D); p.ldd = ldd;
-  p.epilogue = dyt ? kDyt : kGelu;
+  p.epilogue = act_cols >= 0 ? kSilu : dyt ? kDyt : kGelu;
+  p.act_cols = act_cols;
   p.bias = static_cast<const float*>(bias); p.x = static_cast<float*>(x); p.ldx = ldx;
   p.w1 = static_cast<const float*>(w1); p.b1 = static_cast<const float*>(b1); p.a1 = a1;
   p.w2 = static_cast<const float*>(w2); p.b2 = static_cast<const float*>(b2); p.a2 = a2;

@@ -37,6 +37,11 @@ struct DecodeArgs {
   int n_chunks;
   __nv_bfloat16* out;  // [B, Hq * D]
   int* chunk_done;     // [B, Hkv] arrival counters (zero between launches) or nullptr: the last CTA of a (sequence, KV head) merges
+  // k_new == nullptr: the cache holds the new token's row already.  cap > 0: scores become cap tanh(score / cap).  gate ([B, ld_gate] + head
+  // or null): head h's output is multiplied by sigmoid(gate).  out rows are ld_out elements apart.  (decode_attn_mma_kernel only)
+  float cap;
+  const __nv_bfloat16* gate;
+  long long ld_gate, ld_out;
 };
 
 template <int D, int REP>
@@ -226,17 +231,18 @@ __global__ void __launch_bounds__(DEC_THREADS, OCC) decode_attn_mma_kernel(const
   const int g = lane >> 2, t = lane & 3;
   int n_old = p.lengths ? p.lengths[b] : p.length;
   if (!ATS_DBG_CHECK(n_old >= 0 && n_old < p.max_len, kDbgDecodeAttn, n_old)) return;
-  const int n_tot = n_old + 1;  // the new token attends to itself
+  const int n_tot = min(n_old + 1, p.max_len);  // the new token attends to itself
   const int k0 = chunk * DEC_CHUNK;
   const bool active = k0 < n_tot;
   const int k_end = min(k0 + DEC_CHUNK, n_tot);
   __nv_bfloat16* kc = p.k_cache + (long long)b * p.cache_b_stride + (long long)hk * D;
   __nv_bfloat16* vc = p.v_cache + (long long)b * p.cache_b_stride + (long long)hk * D;
   const long long row_stride = (long long)p.Hkv * D;
-  const __nv_bfloat16* k_new = p.k_new + (long long)b * p.ld_qkv + hk * D;
-  const __nv_bfloat16* v_new = p.v_new + (long long)b * p.ld_qkv + hk * D;
+  const bool appended = p.k_new == nullptr;
+  const __nv_bfloat16* k_new = appended ? kc + n_old * row_stride : p.k_new + (long long)b * p.ld_qkv + hk * D;
+  const __nv_bfloat16* v_new = appended ? vc + n_old * row_stride : p.v_new + (long long)b * p.ld_qkv + hk * D;
   // the new token's K / V row goes into the cache (by the CTA that owns its position); this CTA reads it from the projection
-  if (active && n_old >= k0 && n_old < k0 + DEC_CHUNK && n_old < p.max_len) {
+  if (!appended && active && n_old >= k0 && n_old < k0 + DEC_CHUNK && n_old < p.max_len) {
     for (int d = tid; d < D; d += DEC_THREADS) {
       kc[n_old * row_stride + d] = k_new[d];
       vc[n_old * row_stride + d] = v_new[d];
@@ -271,8 +277,14 @@ __global__ void __launch_bounds__(DEC_THREADS, OCC) decode_attn_mma_kernel(const
       }
       if (g < REP) {  // c[0], c[1]: head g, keys 2t and 2t + 1 of the tile
         const int c0 = kw0 + nt * 8 + 2 * t;
-        s_p[g][c0] = (active && k0 + c0 < k_end) ? c[0] * p.scale : -INFINITY;
-        s_p[g][c0 + 1] = (active && k0 + c0 + 1 < k_end) ? c[1] * p.scale : -INFINITY;
+        float s0 = c[0] * p.scale, s1 = c[1] * p.scale;
+        if (p.cap > 0.f) {
+          const float inv = __fdividef(1.f, p.cap);
+          s0 = p.cap * tanh_fast(s0 * inv);
+          s1 = p.cap * tanh_fast(s1 * inv);
+        }
+        s_p[g][c0] = (active && k0 + c0 < k_end) ? s0 : -INFINITY;
+        s_p[g][c0 + 1] = (active && k0 + c0 + 1 < k_end) ? s1 : -INFINITY;
       }
     }
   }
@@ -381,7 +393,8 @@ __global__ void __launch_bounds__(DEC_THREADS, OCC) decode_attn_mma_kernel(const
     const float mc = __ldcg(ml + 2 * c);
     l += __ldcg(ml + 2 * c + 1) * ((mc == -INFINITY) ? 0.f : __expf(mc - m));
   }
-  const float inv = l > 0.f ? 1.f / l : 0.f;
+  float inv = l > 0.f ? 1.f / l : 0.f;
+  if (p.gate) inv = __fdividef(inv, 1.f + __expf(-__bfloat162float(p.gate[(long long)b * p.ld_gate + hk * REP + warp])));
   for (int d = lane; d < D; d += 32) {
     float acc = 0.f;
     for (int c = 0; c < p.n_chunks; ++c) {
@@ -389,7 +402,7 @@ __global__ void __launch_bounds__(DEC_THREADS, OCC) decode_attn_mma_kernel(const
       const float f = (mc == -INFINITY) ? 0.f : __expf(mc - m);
       acc += __ldcg(p.part_o + (wq * p.n_chunks + c) * D + d) * f;
     }
-    p.out[wq * D + d] = __float2bfloat16(acc * inv);
+    p.out[(long long)b * p.ld_out + (hk * REP + warp) * D + d] = __float2bfloat16(acc * inv);
   }
 }
 
@@ -888,6 +901,7 @@ ATS_API int ats_decode_attn(const void* qkv, long long ld_qkv, int q_col0, int k
   p.B = B; p.Hq = Hq; p.Hkv = Hkv; p.D = D; p.max_len = max_len;
   p.scale = 1.f / sqrtf(float(D));
   p.part_o = part_o; p.part_ml = part_ml;
+  p.cap = 0.f; p.gate = nullptr; p.ld_gate = 0; p.ld_out = (long long)Hq * D;
   // chunks to launch: enough for the longest sequence (+ the new token)
   p.n_chunks = (min(max_tokens + 1, max_len) + DEC_CHUNK - 1) / DEC_CHUNK;
   if (p.n_chunks < 1) p.n_chunks = 1;
@@ -910,6 +924,32 @@ ATS_API int ats_decode_attn(const void* qkv, long long ld_qkv, int q_col0, int k
   const int BH = B * Hq;
   launch_pdl(decode_merge_kernel, dim3((BH * 32 + 255) / 256), dim3(256), 0, s, (const float*)part_o, (const float*)part_ml, p.out, BH, p.n_chunks, D);
   return int(cudaGetLastError());
+}
+
+// The same for a cache that holds the new token's row already (written by the kernel that prepared the queries, or by the layer whose
+// keys and values this one shares): q [B, ldq], scale given, optionally capped scores and one output gate per head.  Heads of 64 or 128
+// dimensions, 1, 2, 4 or 8 query heads per key head; anything else returns 1003.
+ATS_API int ats_decode_attn_cached(const void* q, long long ldq, void* k_cache, void* v_cache, long long cache_b_stride, const int* lengths, int B, int Hq,
+                                   int Hkv, int D, int max_len, float scale, float cap, const void* gate, long long ld_gate, float* part_o, float* part_ml,
+                                   int* chunk_done, void* out, long long ld_out, void* stream) {
+  if ((D != 64 && D != 128) || Hkv < 1 || Hq % Hkv || (ldq & 7) || !lengths || !chunk_done || max_len < 1) return 1003;
+  const int rep = Hq / Hkv;
+  DecodeArgs p = {};
+  p.q = static_cast<const __nv_bfloat16*>(q); p.ld_qkv = ldq;
+  p.k_cache = static_cast<__nv_bfloat16*>(k_cache); p.v_cache = static_cast<__nv_bfloat16*>(v_cache);
+  p.cache_b_stride = cache_b_stride; p.lengths = lengths;
+  p.B = B; p.Hq = Hq; p.Hkv = Hkv; p.D = D; p.max_len = max_len; p.scale = scale; p.cap = cap;
+  p.gate = static_cast<const __nv_bfloat16*>(gate); p.ld_gate = ld_gate;
+  p.part_o = part_o; p.part_ml = part_ml; p.n_chunks = (max_len + DEC_CHUNK - 1) / DEC_CHUNK; p.chunk_done = chunk_done;
+  p.out = static_cast<__nv_bfloat16*>(out); p.ld_out = ld_out;
+  const dim3 grid(p.n_chunks, Hkv, B);
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  cudaError_t ce = cudaErrorInvalidValue;
+#define ATS_DEC(DD, RR) if (D == DD && rep == RR) ce = launch_pdl(decode_attn_mma_kernel<DD, RR, 2>, grid, dim3(DEC_THREADS), 0, s, p);
+  ATS_DEC(64, 1) ATS_DEC(64, 2) ATS_DEC(64, 4) ATS_DEC(64, 8) ATS_DEC(128, 1) ATS_DEC(128, 2) ATS_DEC(128, 4) ATS_DEC(128, 8)
+#undef ATS_DEC
+  if (rep != 1 && rep != 2 && rep != 4 && rep != 8) return 1003;
+  return int(ce != cudaSuccess ? ce : cudaGetLastError());
 }
 
 // logits [B, V] (row pitch ld elements; fp32 when logits_fp32 else bf16) -> out [B] int64.  work: [B, V] fp32 scratch;
