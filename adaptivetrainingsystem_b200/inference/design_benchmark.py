@@ -1,5 +1,6 @@
-"""Serving throughput of the Vimodra design beside the closest other model of the framework (the dense grouped-query decoder) at equal
-width, depth, head count and feed-forward size, with random weights; ``bench.py --design vimodra`` prints it.
+"""Serving throughput of a layer-listed design (``vimodra``, ``nemipel``) beside the closest other models of the framework (the dense
+grouped-query decoder; for Nemipel also Vimodra) at equal width, depth, head count and feed-forward size, with random weights;
+``bench.py --design NAME`` prints it.
 
 ``end_to_end`` times whole prompts and graph-replayed decode steps; ``kernels`` times the kernels of one layer of either model alone, with
 L2 flushed before every launch, and puts each beside its roofline (the larger of FLOPs over the tensor or fp32 rate and bytes over the
@@ -14,12 +15,14 @@ from typing import Any, Callable, Dict, List, Optional
 
 import torch
 
-# nominal sizes of a mid-size decoder; layers: three latent-attention layers to one recurrent layer
+# nominal sizes of a mid-size decoder; Vimodra: three latent-attention layers to one recurrent layer; Nemipel: lightning, attention and
+# channel-wise delta layers in turn, the second attention layer on the first one's keys and values
 SIZES: Dict[str, Dict[str, int]] = {
     "w2048": dict(width=2048, heads=16, kv_rank=512, q_rank=768, ff=8192),
     "w4096": dict(width=4096, heads=32, kv_rank=512, q_rank=1536, ff=16384),
 }
 LAYERS, VOCAB, WINDOW = 8, 32000, 1024
+PEERS: Dict[str, List[str]] = {"vimodra": ["dense"], "nemipel": ["dense", "vimodra"]}   # models timed beside a design
 
 
 def vimodra_config(size: str):
@@ -32,19 +35,38 @@ def vimodra_config(size: str):
     return VimodraConfig.from_dict({"vocab": VOCAB, "width": z["width"], "norm": {"eps": 1e-5}, "layers": [rec if i % 4 == 3 else attn for i in range(LAYERS)]})
 
 
+def gated_ff(size: str) -> int:
+    """A gated feed-forward has three matrices: two thirds of the width for the same size."""
+    return (2 * SIZES[size]["ff"] // 3 + 127) // 128 * 128
+
+
+def nemipel_config(size: str):
+    from ..config import NemipelConfig
+    z = SIZES[size]
+    H, mlp = z["heads"], {"kind": "dense", "ff": gated_ff(size)}
+    light = {"type": "lightning", "mlp": mlp, "mixer": {"heads": H, "dim": 128, "vdim": 128, "decay": [1.0 - 2.0 ** (-1 - 8.0 * i / H) for i in range(H)]}}
+    rec = {"type": "channel_delta", "mlp": mlp, "mixer": {"heads": H, "kv_heads": H // 2, "dim": 128, "vdim": 128, "conv": 4}}
+
+    def attn(**kw):
+        return {"type": "attention", "mlp": mlp, "mixer": {"heads": H, "kv_heads": H // 4, "dim": 128, "vdim": 128, "rot": {"base": 10000.0, "dims": 64},
+                                                            "scale": 128 ** -0.5, "softcap": 30.0, **kw}}
+    layers = [light, attn(), rec, light, attn(kv_from=1), rec, light, attn()]
+    assert len(layers) == LAYERS
+    return NemipelConfig.from_dict({"vocab": VOCAB, "width": z["width"], "norm": {"eps": 1e-6}, "postln_alpha": 3.0, "logit_softcap": 30.0, "layers": layers})
+
+
 def dense_config(size: str, seq: int):
     from ..config import ModelConfig
     z = SIZES[size]
-    # a gated feed-forward has three matrices: two thirds of the width for the same size
     return ModelConfig(vocab_size=VOCAB, hidden_size=z["width"], num_layers=LAYERS, num_heads=z["heads"], num_kv_heads=z["heads"] // 4,
-                       intermediate_size=(2 * z["ff"] // 3 + 127) // 128 * 128, seq_length=seq, tie_word_embeddings=False)
+                       intermediate_size=gated_ff(size), seq_length=seq, tie_word_embeddings=False)
 
 
 def build(design: str, size: str, seq: int):
     dev = torch.device("cuda", torch.cuda.current_device())
-    if design == "vimodra":
-        from ..models import Vimodra
-        return Vimodra.random(vimodra_config(size), torch.bfloat16, dev)
+    if design != "dense":
+        from ..models import Nemipel, Vimodra
+        return Vimodra.random(vimodra_config(size), torch.bfloat16, dev) if design == "vimodra" else Nemipel.random(nemipel_config(size), torch.bfloat16, dev)
     from ..models import DeepSeekTransformer
     torch.manual_seed(0)
     with torch.device(dev):
@@ -144,15 +166,29 @@ class _Timer:
         self.rows.append({"model": model, "kernel": name, "us": round(ms * 1e3, 1), "roofline_us": round(roof * 1e3, 2), "of_roofline": round(roof / ms, 3)})
 
 
+def _bf(*shape):
+    return torch.randn(*shape, device="cuda").to(torch.bfloat16)
+
+
+def _gemm_cost(T, N, K, extra=0):
+    return dict(bytes_=2.0 * (T * K + N * K + T * N) + extra, flops=2.0 * T * N * K)
+
+
 @torch.no_grad()
-def kernels(size: str, B: int = 8, L: int = 2048, decode_batch: int = 64) -> List[Dict[str, Any]]:
+def kernels(design: str, size: str, B: int = 8, L: int = 2048, decode_batch: int = 64) -> List[Dict[str, Any]]:
+    """The kernels of one layer of every kind of ``design``, then those of the models beside it."""
+    t = _Timer(torch.device("cuda", torch.cuda.current_device()))
+    for name in [design] + PEERS[design]:
+        {"vimodra": _vimodra_kernels, "nemipel": _nemipel_kernels, "dense": _dense_kernels}[name](t, size, B, L, decode_batch)
+        torch.cuda.empty_cache()
+    return t.rows
+
+
+def _vimodra_kernels(t: _Timer, size: str, B: int, L: int, n: int) -> None:
     from .. import ops
-    from ..models.mixers import Step
     from ..ops import delta as D, dyt, latent as A
-    from ..ops import gemm as G
     m = build("vimodra", size, L)
     dev = next(m.parameters()).device
-    t = _Timer(dev)
     z, W = SIZES[size], SIZES[size]["width"]
     att, rec, mlp = m.mixers[0], m.mixers[3], m.mlps[0]
     s, d = att.s, rec.s
@@ -161,11 +197,7 @@ def kernels(size: str, B: int = 8, L: int = 2048, decode_batch: int = 64) -> Lis
     T = B * L
     H, ff = s.heads, z["ff"]
 
-    def bf(*shape):
-        return torch.randn(*shape, device=dev).to(torch.bfloat16)
-
-    def gemm_cost(T, N, K, extra=0):
-        return dict(bytes_=2.0 * (T * K + N * K + T * N) + extra, flops=2.0 * T * N * K)
+    bf, gemm_cost = _bf, _gemm_cost
     # ---- portions
     h, x = bf(T, W), torch.randn(T, W, device=dev)
     c1, c2 = m.chains[0]
@@ -200,7 +232,6 @@ def kernels(size: str, B: int = 8, L: int = 2048, decode_batch: int = 64) -> Lis
     t.add("vimodra", "prefill delta_output", lambda: D.delta_output(o, dg, rec.norm, d), 2.0 * T * 3 * d.heads * d.vdim)
     del u, mixed, o, dproj, q, kv, a
     # ---- one token per sequence
-    n = decode_batch
     hd, xd = bf(n, W), torch.randn(n, W, device=dev)
     lengths = torch.full((n,), L - 1, dtype=torch.int32, device=dev)
     active = torch.ones(n, dtype=torch.int32, device=dev)
@@ -227,9 +258,112 @@ def kernels(size: str, B: int = 8, L: int = 2048, decode_batch: int = 64) -> Lis
     t.add("vimodra", "decode delta_step", lambda: D.delta_step(mx, rl, gbd, dd["S"], dpd.view(n, -1)[:, d.g_col:], rec.norm, d, lengths, active),
           8.0 * n * d.heads * d.dim * d.vdim)
     ops.check_status()
-    del m, att, rec, mlp, st, ds, sd, dd
-    torch.cuda.empty_cache()
-    # ---- the dense grouped-query model
+
+
+def _nemipel_kernels(t: _Timer, size: str, B: int, L: int, n: int) -> None:
+    from .. import ops
+    from ..ops import delta as D, gqa as Q, lightning as N, postnorm as pn
+    m = build("nemipel", size, L)
+    dev = next(m.parameters()).device
+    W, T = SIZES[size]["width"], B * L
+    light, att, rec, mlp = m.mixers[0], m.mixers[1], m.mixers[2], m.mlps[0]
+    ls, s, d, ff = light.s, att.s, rec.s, mlp.ff
+    H, rope = s.heads, att._rope[0]
+    rope.ensure(L + 1, dev)
+    c1, c2 = m.steps[0]
+    bf, gemm_cost, name = _bf, _gemm_cost, "nemipel"
+    state = 4.0 * H * 128 * 128
+    # ---- portions
+    h, x = bf(T, W), torch.randn(T, W, device=dev)
+    t.add(name, "prefill gemm + silu: lightning q, k, v, gate", lambda: pn.linear_silu(h, light.w_in, ls.g_col), **gemm_cost(T, ls.proj_width, W))
+    proj, S = pn.linear_silu(h, light.w_in, ls.g_col), light.state(B, L, torch.bfloat16, dev)["S"]
+    # products inside chunks of 128 tokens and with the state, everything once
+    t.add(name, "prefill lightning attention", lambda: N.lightning_scan(proj, S, light.powers, ls, L, True), 2.0 * T * (ls.v_col + 2 * ls.o_pad),
+          flops=2.0 * T * H * (64 * 256 + 2 * 128 * 128))
+    o = N.lightning_scan(proj, S, light.powers, ls, L, True)
+    t.add(name, "prefill norm_gate", lambda: pn.norm_gate(o, proj[:, ls.g_col:], light.norm, ls.eps, ls.o_pad), 2.0 * T * 3 * ls.o_pad)
+    a = pn.norm_gate(o, proj[:, ls.g_col:], light.norm, ls.eps, ls.o_pad)
+    t.add(name, "prefill gemm + post-norm step: attention output", lambda: pn.linear_postnorm(a, light.w_o, x, c1), **gemm_cost(T, W, ls.o_pad, 8.0 * T * W))
+    part = torch.randn(1, T, W, device=dev)
+    t.add(name, "prefill post-norm step alone", lambda: _fold_alone(pn, part, x, c1), 4.0 * T * W * 3 + 2.0 * T * W)
+    del part
+    t.add(name, "prefill gemm + swiglu: up", lambda: mlp(h), **gemm_cost(T, 2 * ff, W, -2.0 * T * ff))
+    u = mlp(h)
+    t.add(name, "prefill gemm + post-norm step: down", lambda: pn.linear_postnorm(u, mlp.w_down, x, c2), **gemm_cost(T, W, ff, 8.0 * T * W))
+    del proj, o, a, u
+    t.add(name, "prefill gemm: q, k, v, gate", lambda: ops.linear(h, att.w_in), **gemm_cost(T, s.proj_width, W))
+    proj = ops.linear(h, att.w_in).view(B, L, -1)
+    st = att.state(B, L, torch.bfloat16, dev)
+    t.add(name, "prefill gqa_prepare (norms, rotation, cache)", lambda: Q.gqa_prepare(proj, s, att.q_norm, att.k_norm, rope.cos, rope.sin, st["k"], st["v"]),
+          2.0 * T * 2 * (s.q_pad + s.k_pad + s.v_pad))
+    q, gate = Q.gqa_prepare(proj, s, att.q_norm, att.k_norm, rope.cos, rope.sin, st["k"], st["v"]), proj.view(T, -1)[:, s.g_col:]
+    t.add(name, "prefill attention (causal, capped)", lambda: Q.gqa_portion(q, st["k"], st["v"], gate, s, L, 0), 2.0 * T * (2 * s.q_pad + s.k_pad + s.v_pad),
+          flops=2.0 * B * H * (L * (L + 1) / 2) * 2 * s.dim)
+    del proj, q, gate, st
+    t.add(name, "prefill gemm: delta q, k, v, low-rank inputs", lambda: ops.linear(h, rec.w_in), **gemm_cost(T, d.proj_width, W))
+    proj = ops.linear(h, rec.w_in)
+    low = proj[:, d.low_col:d.low_col + d.low_width]
+    t.add(name, "prefill gemm: delta decays, gate", lambda: ops.linear(low, rec.w_low), **gemm_cost(T, d.g_col + d.o_pad, d.low_width / 2))
+    wide, ds = ops.linear(low, rec.w_low), rec.state(B, L, torch.bfloat16, dev)
+    t.add(name, "prefill delta_prep", lambda: D.delta_prep(proj.view(B, L, -1), d, rec.conv, None, None, ds["tail"]), 2.0 * T * 2 * d.channels)
+    mixed, rlen, gb = D.delta_prep(proj.view(B, L, -1), d, rec.conv, None, None, ds["tail"])
+    t.add(name, "prefill channel_delta_scan", lambda: D.channel_delta_scan(mixed, rlen, gb, wide, rec.neg_rate, rec.dt_bias, ds["S"], d, L, True),
+          2.0 * T * (d.channels + d.heads * (d.dim + d.vdim)), fp32=2.0 * T * d.heads * 3 * d.dim * d.vdim)
+    o = D.channel_delta_scan(mixed, rlen, gb, wide, rec.neg_rate, rec.dt_bias, ds["S"], d, L, True)
+    t.add(name, "prefill delta_output", lambda: D.delta_output(o, wide[:, d.g_col:], rec.norm, d), 2.0 * T * 3 * d.heads * d.vdim)
+    del proj, low, wide, mixed, o, h, x
+    # ---- one token per sequence
+    hd, xd = bf(n, W), torch.randn(n, W, device=dev)
+    lengths, active = torch.full((n,), L - 1, dtype=torch.int32, device=dev), torch.ones(n, dtype=torch.int32, device=dev)
+    t.add(name, "decode gemm + silu: lightning q, k, v, gate", lambda: pn.linear_silu(hd, light.w_in, ls.g_col), 2.0 * light.w_in.numel())
+    pd, Sd = pn.linear_silu(hd, light.w_in, ls.g_col), light.state(n, L, torch.bfloat16, dev)["S"]
+    t.add(name, "decode lightning_step", lambda: N.lightning_step(pd, Sd, light.decay, ls, lengths, active), 2 * n * state)
+    od = N.lightning_step(pd, Sd, light.decay, ls, lengths, active)
+    t.add(name, "decode norm_gate", lambda: pn.norm_gate(od, pd[:, ls.g_col:], light.norm, ls.eps, ls.o_pad), 2.0 * n * 3 * ls.o_pad)
+    ad = bf(n, ls.o_pad)
+    t.add(name, "decode gemm + post-norm step: attention output", lambda: pn.linear_postnorm(ad, light.w_o, xd, c1), 2.0 * light.w_o.numel())
+    t.add(name, "decode gemm + swiglu: up", lambda: mlp(hd), 2.0 * mlp.w_gate_up.numel())
+    ud = bf(n, ff)
+    t.add(name, "decode gemm + post-norm step: down", lambda: pn.linear_postnorm(ud, mlp.w_down, xd, c2), 2.0 * mlp.w_down.numel())
+    w = min(WINDOW, L)   # the cache length of the dense model's row
+    sd = att.state(n, w + 8, torch.bfloat16, dev)
+    sd["k"].normal_(), sd["v"].normal_()
+    at = torch.full((n,), w - 1, dtype=torch.int32, device=dev)
+    t.add(name, "decode gemm: q, k, v, gate", lambda: ops.linear(hd, att.w_in), 2.0 * att.w_in.numel())
+    pa = ops.linear(hd, att.w_in).view(n, 1, -1)
+    t.add(name, "decode gqa_prepare", lambda: Q.gqa_prepare(pa, s, att.q_norm, att.k_norm, rope.cos, rope.sin, sd["k"], sd["v"], 0, at, active),
+          2.0 * n * 2 * (s.q_pad + s.k_pad + s.v_pad))
+    qd, gd = bf(n, s.q_pad), pa.view(n, -1)[:, s.g_col:]
+    t.add(name, "decode attention (capped, gated)", lambda: Q.gqa_decode(qd, sd["k"], sd["v"], gd, s, at), 2.0 * n * w * (s.k_pad + s.v_pad))
+    t.add(name, "decode gemm: delta q, k, v, low-rank inputs", lambda: ops.linear(hd, rec.w_in), 2.0 * rec.w_in.numel())
+    pr = ops.linear(hd, rec.w_in)
+    t.add(name, "decode gemm: delta decays, gate", lambda: ops.linear(pr[:, d.low_col:d.low_col + d.low_width], rec.w_low), 2.0 * rec.w_low.numel())
+    wd, dd = ops.linear(pr[:, d.low_col:d.low_col + d.low_width], rec.w_low), rec.state(n, L, torch.bfloat16, dev)
+    t.add(name, "decode delta_prep", lambda: D.delta_prep(pr.view(n, 1, -1), d, rec.conv, None, None, dd["tail"], 0, lengths, active),
+          2.0 * n * d.channels * (2 + 2 * (d.taps - 1)))
+    mx, rl, gbd = D.delta_prep(pr.view(n, 1, -1), d, rec.conv, None, None, dd["tail"], 0, lengths, active)
+    t.add(name, "decode delta_step", lambda: D.delta_step(mx, rl, gbd, dd["S"], wd[:, d.g_col:], rec.norm, d, lengths, active, wd, rec.neg_rate, rec.dt_bias),
+          2 * n * state)
+    lg = torch.randn(n, VOCAB, device=dev)
+    t.add(name, "decode softcap of the logits", lambda: pn.softcap_(lg, 30.0, True), 8.0 * n * VOCAB)
+    ops.check_status()
+
+
+def _fold_alone(pn, part, x, c) -> None:
+    """The fold launch of ``linear_postnorm`` without its product."""
+    from .. import ops
+    h = torch.empty(x.shape, dtype=torch.bfloat16, device=x.device)
+    a = pn._PostNorm(part.data_ptr(), 1, x.numel(), x.data_ptr(), c.alpha, c.w.data_ptr(), 0, c.eps, h.data_ptr(), x.shape[0], x.shape[1], c.width)
+    ops._lib.check(pn._fns().ats_fold_postnorm(pn.ctypes.byref(a), 0, ops._lib.stream_ptr(x.device)), "ats_fold_postnorm")
+
+
+def _dense_kernels(t: _Timer, size: str, B: int, L: int, n: int) -> None:
+    from .. import ops
+    from ..ops import gemm as G
+    bf, gemm_cost = _bf, _gemm_cost
+    W, T, w = SIZES[size]["width"], B * L, min(WINDOW, L)
+    dev = t.flush.device
+    h, hd, ad = bf(T, W), bf(n, W), bf(n, W)
     p = build("dense", size, L)
     blk = p.layers[0]
     at = blk.self_attn
@@ -260,20 +394,19 @@ def kernels(size: str, B: int = 8, L: int = 2048, decode_batch: int = 64) -> Lis
     t.add("dense", "decode gemm + residual: down", lambda: ops.linear(ud2, blk.ffn.down_proj, residual=hd), 2.0 * blk.ffn.down_proj.numel())
     t.add("dense", "decode rms_norm", lambda: ops.rms_norm(hd, blk.input_norm.weight), 2.0 * 2 * n * W)
     ops.check_status()
-    return t.rows
 
 
-def run(sizes: Optional[List[str]] = None, per_kernel: bool = True) -> Dict[str, Any]:
-    res: Dict[str, Any] = {"metric": "vimodra_serving_tokens_per_sec", "unit": "tokens/s", "n_gpus": 1, "higher_is_better": True, "dtype": "bf16", "data": "synthetic",
+def run(design: str = "vimodra", sizes: Optional[List[str]] = None, per_kernel: bool = True) -> Dict[str, Any]:
+    res: Dict[str, Any] = {"metric": f"{design}_serving_tokens_per_sec", "unit": "tokens/s", "n_gpus": 1, "higher_is_better": True, "dtype": "bf16", "data": "synthetic",
                            "config": {"layers": LAYERS, "vocab": VOCAB, "window": WINDOW, "prefill": "8 x 2048 tokens", "decode": "after 1024 tokens, CUDA graph",
                                       "l2": "kernel timings flush L2 before every launch; whole steps exceed it"},
                            "roofline": peaks()["kind"], "sizes": {}}
     for size in sizes or list(SIZES):
-        r: Dict[str, Any] = {d: end_to_end(d, size) for d in ("vimodra", "dense")}
+        r: Dict[str, Any] = {d: end_to_end(d, size) for d in [design] + PEERS[design]}
         if per_kernel:
-            r["kernels"] = kernels(size)
+            r["kernels"] = kernels(design, size)
             torch.cuda.empty_cache()
         res["sizes"][size] = r
     first = res["sizes"][(sizes or list(SIZES))[0]]
-    res["value"] = first["vimodra"]["prefill_tokens_per_s"]
+    res["value"] = first[design]["prefill_tokens_per_s"]
     return res

@@ -372,15 +372,15 @@ def main():
     ap.add_argument("--no-decode", action="store_true", help="skip the serving half of the metric")
     ap.add_argument("--no-fused-check", action="store_true", help="skip the fused-vs-NCCL check that precedes a multi-GPU run")
     ap.add_argument("--decode-layers", type=int, default=0, help="debug only: serving models with fewer layers")
-    ap.add_argument("--design", default="", choices=["", "vimodra"], help="instead of the headline workload: serving throughput and per-kernel times of this model "
-                    "design beside the dense decoder of equal size (one GPU)")
+    ap.add_argument("--design", default="", choices=["", "vimodra", "nemipel"], help="instead of the headline workload: serving throughput and per-kernel times of "
+                    "this model design beside the closest other models of equal size (one GPU)")
     ap.add_argument("--design-sizes", default="", help="with --design: comma-separated sizes (default: all)")
     args = ap.parse_args()
     if args.design:
         import torch
         from adaptivetrainingsystem_b200.inference import design_benchmark
         with ClockSampler(torch.cuda.current_device()) as clk:
-            res = design_benchmark.run([x for x in args.design_sizes.split(",") if x] or None)
+            res = design_benchmark.run(args.design, [x for x in args.design_sizes.split(",") if x] or None)
         res["clocks"] = clk.summary()
         print(json.dumps(res), flush=True)
         return

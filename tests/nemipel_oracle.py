@@ -212,7 +212,7 @@ def with_mlp(layer, ff):
     return {**layer, "mlp": {"kind": "dense", "ff": ff}}
 
 
-def config(layers, width=72, vocab=104, eps=1e-5, alpha=1.7, cap=11.0):
+def config(layers, width=72, vocab=104, eps=1e-3, alpha=1.7, cap=11.0):
     return {"architecture": "Nemipel", "vocab": vocab, "width": width, "norm": {"eps": eps}, "postln_alpha": alpha, "logit_softcap": cap, "layers": layers}
 
 

@@ -18,53 +18,17 @@ from adaptivetrainingsystem_b200.models import Vimodra, load_model
 from adaptivetrainingsystem_b200.ops import delta as delta_ops
 from adaptivetrainingsystem_b200.ops import dyt as dyt_ops
 from adaptivetrainingsystem_b200.ops import latent as latent_ops
-
-gpu = pytest.mark.gpu
-PLACES = [pytest.param("cpu", torch.float32, id="cpu"), pytest.param("cuda", torch.float32, id="gpu-fp32", marks=gpu),
-          pytest.param("cuda", torch.bfloat16, id="gpu-bf16", marks=gpu)]
-EXACT = PLACES[:2]
-# root-mean-square error of the logits of a position over the root mean square of all logits: the worst position may reach TOL, the
-# mean over the positions 40 % of it (random bf16 models scatter: near ties of the scores and large gates amplify a rounding)
-TOL = {torch.float32: 1e-4, torch.bfloat16: 0.12}
+from layered_utils import EXACT, PLACES, TOL, close, gpu, position_errors, run_portions, tokens
 
 
 def build(cfg, weights, device, dtype):
     return Vimodra.from_tensors(VimodraConfig.from_dict(cfg), lambda n: weights[n], list(weights), dtype, device)
 
 
-def position_errors(got, want):
-    want = want.float()
-    d = got.float().cpu() - want
-    d = d - d.mean(-1, keepdim=True)
-    return d.pow(2).mean(-1).sqrt() / want.pow(2).mean().sqrt()
-
-
-def close(got, want, dtype, factor=1.0):
-    e = position_errors(got, want)
-    assert float(e.max()) < factor * TOL[dtype], f"worst position {int(e.flatten().argmax())}: {float(e.max()):.3g}"
-    assert float(e.mean()) < factor * TOL[dtype] * 0.4, f"mean {float(e.mean()):.3g}"
-
-
 def mixed_config(**kw):
     layers = [O.with_mlp(O.latent_spec(size=9), 88), O.with_mlp(O.delta_spec(), 40), O.latent_spec(heads=5, dim=8, rot_dim=16, vdim=8, kv_rank=24, q_rank=32, size=21),
               O.with_mlp(O.delta_spec(heads=6, kv_heads=2, dim=24, vdim=16, conv=5), 56)]
     return O.config(layers, **{"width": 72, "loop": (1, 3, 2), **kw})
-
-
-def tokens(n, vocab=104, seed=1):
-    return torch.randint(0, vocab, (n,), generator=torch.Generator().manual_seed(seed)).tolist()
-
-
-def run_portions(model, ids, sizes):
-    """Logits of every position when the tokens come in portions of these sizes."""
-    dev = model.embed.device
-    cache, out, at = model.make_cache(1, len(ids)), [], 0
-    for n in sizes:
-        part = torch.tensor([ids[at:at + n]], device=dev)
-        out.append(model(part, cache=cache)[0].float().cpu())
-        at += n
-    assert at == len(ids)
-    return torch.cat(out)
 
 
 # ------------------------------------------------------------------------------------------------ mechanisms alone
