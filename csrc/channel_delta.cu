@@ -39,9 +39,10 @@ struct ChannelArgs {
   __host__ __device__ int size() const { return 2 * DC * DC + (3 * DC + 1) * DK; }
 };
 
-// One warp per (group, head, sequence); lane l holds channels l, l + 32, ...
-template <typename T>
-__global__ void __launch_bounds__(128) channel_pairs_kernel(const ChannelArgs p) {
+// One warp per (group, head, sequence).  VC channels per lane side by side, so that all of a warp's loads of a pass are in flight together
+// and are whole lines; DK = 32 * VC * passes.
+template <typename T, int VC, bool VEC>
+__global__ void __launch_bounds__(128, 3) channel_pairs_kernel(const ChannelArgs p) {
   pdl_prologue();
   __shared__ float s_kk[4][DC][DC + 1], s_kq[4][DC][DC + 1];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -57,46 +58,82 @@ __global__ void __launch_bounds__(128) channel_pairs_kernel(const ChannelArgs p)
   float* co = p.coef + w * p.size();
   float* rows = co + 2 * DC * DC;
   const float rate = p.neg_rate[h];
-  float rk[DC], rq[DC];
-#pragma unroll
-  for (int i = 0; i < DC; ++i) {
-    rq[i] = i < n ? rl[(long long)i * 2 * p.KH + kh] : 0.f;
-    rk[i] = i < n ? rl[(long long)i * 2 * p.KH + p.KH + kh] : 0.f;
-  }
   // sums[8 i + j]: i >= j: kq_ij; i < j: kk_ji
   float sums[DC * DC];
 #pragma unroll
   for (int i = 0; i < DC * DC; ++i) sums[i] = 0.f;
-  for (int d = lane; d < p.DK; d += 32) {
-    const bool ok = d < p.dim;
-    const float dt = ok ? p.dt_bias[(long long)h * p.dim + d] : 0.f;
-    float kv[DC], qv[DC], g[DC];
+  using Bits_ = typename Bits<VC * int(sizeof(T))>::type;
+  for (int d0 = lane * VC; d0 < p.DK; d0 += 32 * VC) {
+    union Piece { Bits_ bits; T v[VC]; };
+    Piece pk[DC], pq[DC], pa[DC];
+    float dt[VC];
+    auto fetch = [&](Piece& x, const T* src, bool in) {
+#pragma unroll
+      for (int c = 0; c < VC; ++c) Typed<T>::store(&x.v[c], 0.f);
+      if (!in) return;
+      if constexpr (VEC) {
+        if (d0 < p.dim) x.bits = *reinterpret_cast<const Bits_*>(src + d0);
+      } else {
+#pragma unroll
+        for (int c = 0; c < VC; ++c)
+          if (d0 + c < p.dim) x.v[c] = src[d0 + c];
+      }
+    };
 #pragma unroll
     for (int i = 0; i < DC; ++i) {
-      const bool in = ok && i < n;
-      kv[i] = in ? Typed<T>::load(k + i * p.ldm + d) * rk[i] : 0.f;
-      qv[i] = in ? Typed<T>::load(q + i * p.ldm + d) * rq[i] : 0.f;
-      g[i] = in ? decay_of(Typed<T>::load(a + i * p.lda + d) + dt, rate) : 1.f;
+      fetch(pk[i], k + i * p.ldm, i < n);
+      fetch(pq[i], q + i * p.ldm, i < n);
+      fetch(pa[i], a + i * p.lda, i < n);
     }
-    float P = 1.f;
+#pragma unroll
+    for (int c = 0; c < VC; ++c) dt[c] = d0 + c < p.dim ? p.dt_bias[(long long)h * p.dim + d0 + c] : 0.f;
+    float kv[DC][VC], qv[DC][VC], g[DC][VC], P[VC];
 #pragma unroll
     for (int i = 0; i < DC; ++i) {
-      P *= g[i];
-      rows[i * p.DK + d] = kv[i] * P;
-      rows[(DC + i) * p.DK + d] = qv[i] * P;
+      const float rk = i < n ? rl[(long long)i * 2 * p.KH + p.KH + kh] : 0.f, rq = i < n ? rl[(long long)i * 2 * p.KH + kh] : 0.f;
+#pragma unroll
+      for (int c = 0; c < VC; ++c) {
+        kv[i][c] = Typed<T>::load(&pk[i].v[c]) * rk;
+        qv[i][c] = Typed<T>::load(&pq[i].v[c]) * rq;
+        g[i][c] = i < n && d0 + c < p.dim ? decay_of<T>(Typed<T>::load(&pa[i].v[c]) + dt[c], rate) : 1.f;
+      }
     }
-    rows[3 * DC * p.DK + d] = P;
+    auto put = [&](int row, const float (&x)[VC]) {
+      static_assert(VC == 2, "one access per row");
+      *reinterpret_cast<float2*>(rows + row * p.DK + d0) = make_float2(x[0], x[1]);
+    };
+#pragma unroll
+    for (int c = 0; c < VC; ++c) P[c] = 1.f;
+#pragma unroll
+    for (int i = 0; i < DC; ++i) {
+      float x[VC], y[VC];
+#pragma unroll
+      for (int c = 0; c < VC; ++c) {
+        P[c] *= g[i][c];
+        x[c] = kv[i][c] * P[c];
+        y[c] = qv[i][c] * P[c];
+      }
+      put(i, x);
+      put(DC + i, y);
+    }
+    put(3 * DC, P);
 #pragma unroll
     for (int j = 0; j < DC; ++j) {
-      float r = kv[j];
-      sums[j * DC + j] += qv[j] * r;
+      float r[VC];
 #pragma unroll
-      for (int i = j + 1; i < DC; ++i) {
-        r *= g[i];
-        sums[i * DC + j] += qv[i] * r;
-        sums[j * DC + i] += kv[i] * r;
+      for (int c = 0; c < VC; ++c) {
+        r[c] = kv[j][c];
+        sums[j * DC + j] += qv[j][c] * r[c];
       }
-      rows[(2 * DC + j) * p.DK + d] = r;
+#pragma unroll
+      for (int i = j + 1; i < DC; ++i)
+#pragma unroll
+        for (int c = 0; c < VC; ++c) {
+          r[c] *= g[i][c];
+          sums[i * DC + j] += qv[i][c] * r[c];
+          sums[j * DC + i] += kv[i][c] * r[c];
+        }
+      put(2 * DC + j, r);
     }
   }
   // transposing reduction: after the steps, lane l holds the sums 2 l and 2 l + 1 over all lanes
@@ -334,7 +371,11 @@ static int launch_channel_scan(const ChannelArgs& p, cudaStream_t s) {
 template <typename T>
 static int launch_channel(const ChannelArgs& p, cudaStream_t s) {
   const long long warps = (long long)p.B * p.groups * p.H;
-  launch_pdl(channel_pairs_kernel<T>, dim3(unsigned((warps + 3) / 4)), dim3(128), 0, s, p);
+  const dim3 grid(unsigned((warps + 3) / 4)), block(128);
+  // pairs of channels: one aligned access when every head and row starts at an even element
+  const bool even = !((p.dim | p.ldm | p.lda) & 1);
+  if (even) launch_pdl(channel_pairs_kernel<T, 2, true>, grid, block, 0, s, p);
+  else launch_pdl(channel_pairs_kernel<T, 2, false>, grid, block, 0, s, p);
   if (p.DK == 64) return launch_channel_scan<T, 4, 8>(p, s);
   if (p.DK == 128) return launch_channel_scan<T, 8, 8>(p, s);
   return launch_channel_scan<T, 16, 4>(p, s);

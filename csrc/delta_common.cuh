@@ -6,8 +6,18 @@ namespace ats {
 
 constexpr int DC = 8;  // tokens per group
 
-// exp(rate softplus(a)), rate < 0
-__device__ __forceinline__ float decay_of(float a, float rate) { return expf(rate * (a > 20.f ? a : log1pf(expf(a)))); }
+// exp(rate softplus(a)), rate < 0.  The bf16 form uses the fast functions and, where exp(a) is small, the series of log(1 + x), so that a
+// slow decay keeps its digits.
+template <typename T>
+__device__ __forceinline__ float decay_of(float a, float rate) {
+  if constexpr (sizeof(T) == 4) {
+    return expf(rate * (a > 20.f ? a : log1pf(expf(a))));
+  } else {
+    const float x = __expf(fminf(a, 20.f));
+    const float l = x < 0.02f ? x * (1.f - x * (0.5f - x * (0.33333333f - 0.25f * x))) : __logf(1.f + x);
+    return __expf(rate * (a > 20.f ? a : l));
+  }
+}
 
 __device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) { return __ffma2_rn(a, b, c); }  // one packed instruction
 // Keeps the compiler from requesting the shared-memory rows of more tokens than registers can hold.

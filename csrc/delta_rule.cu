@@ -46,7 +46,7 @@ template <typename T>
 __device__ __forceinline__ void delta_gate(const DeltaArgs& p, long long row, int h) {
   const T* in = static_cast<const T*>(p.proj) + row * p.ld;
   const float bt = Typed<T>::load(in + p.b_col + h);
-  if (p.neg_rate) p.gb[row * 2 * p.H + h] = decay_of(Typed<T>::load(in + p.a_col + h) + p.dt_bias[h], p.neg_rate[h]);
+  if (p.neg_rate) p.gb[row * 2 * p.H + h] = decay_of<T>(Typed<T>::load(in + p.a_col + h) + p.dt_bias[h], p.neg_rate[h]);
   p.gb[row * 2 * p.H + p.H + h] = 1.f / (1.f + expf(-bt));
 }
 
@@ -675,7 +675,7 @@ template <typename T>
 __device__ __forceinline__ void row_decays(const StepArgs& p, int b, int h, float* s_g, int threads) {
   const T* a = p.a ? static_cast<const T*>(p.a) + (long long)b * p.lda + (long long)h * p.dim : nullptr;
   const float g = p.a ? 0.f : p.gb[(long long)b * 2 * p.H + h], rate = p.a ? p.neg_rate[h] : 0.f;
-  for (int d = threadIdx.x; d < p.dim; d += threads) s_g[d] = a ? decay_of(Typed<T>::load(a + d) + p.dt_bias[(long long)h * p.dim + d], rate) : g;
+  for (int d = threadIdx.x; d < p.dim; d += threads) s_g[d] = a ? decay_of<T>(Typed<T>::load(a + d) + p.dt_bias[(long long)h * p.dim + d], rate) : g;
 }
 
 constexpr int ST_THREADS = 512;

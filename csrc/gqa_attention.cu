@@ -7,7 +7,7 @@
 // The cache holds k [B, max_len, ldk] as the scores use it (normed and rotated) and v [B, max_len, ldv]; a layer that shares another
 // layer's keys and values reads that layer's cache and prepares only its queries.
 //
-// * gqa_prepare: norm, rotation, cache append, one CTA per token.
+// * gqa_prepare: norm, rotation, cache append, one warp per token for the queries and one for key and value.
 // * gqa_portion: L queries of a prompt at positions pos0 .. against the cache, any sizes, bf16 and fp32 (gqa_attention_tcgen05.cu is the
 //   tensor-core form).
 // * gqa_decode + gqa_merge: one query token per sequence, any sizes (decode_attn_mma_kernel in inference.cu serves bf16 heads of 64 and 128).
@@ -54,75 +54,87 @@ __device__ __forceinline__ float rotated(const T* in, const float* w, float r, i
   return (d & 1) ? x * cos[m] + y * sin[m] : x * cos[m] - y * sin[m];
 }
 
+// One warp's row of n values: out = rotate(in r w).  VEC: dim, dims multiples of 8, so that eight consecutive values belong to one head and
+// are rotated or pass as a whole.
 template <typename T, bool VEC>
-__device__ __forceinline__ void norm_rotate_row(const T* in, const float* w, float r, int n, int dim, int dims, const float* cos, const float* sin, T* out) {
-  if constexpr (VEC) {  // dim a multiple of 8: eight consecutive values belong to one head and hold whole pairs
-    for (int c = threadIdx.x * 8; c < n; c += 256 * 8) {
+__device__ __forceinline__ void norm_rotate_row(const T* in, const float* w, float r, int n, int dim, int dims, const float* cos, const float* sin, T* out,
+                                                int lane) {
+  if constexpr (VEC) {
+#pragma unroll 4
+    for (int c = lane * 8; c < n; c += 256) {
       float v[8], g[8];
       Typed<T>::load8(in + c, v);
       Typed<float>::load8(w + c, g);
 #pragma unroll
       for (int e = 0; e < 8; ++e) v[e] *= r * g[e];
-      const int d = c % dim;
+      const unsigned d = unsigned(c) % unsigned(dim);
+      if (d < unsigned(dims)) {
+        const float4 cs = *reinterpret_cast<const float4*>(cos + (d >> 1)), sn = *reinterpret_cast<const float4*>(sin + (d >> 1));
+        const float c4[4] = {cs.x, cs.y, cs.z, cs.w}, s4[4] = {sn.x, sn.y, sn.z, sn.w};
 #pragma unroll
-      for (int e = 0; e < 8; e += 2) {
-        if (d + e < dims) {
-          const float cs = cos[(d + e) >> 1], sn = sin[(d + e) >> 1], a = v[e], b = v[e + 1];
-          v[e] = a * cs - b * sn;
-          v[e + 1] = b * cs + a * sn;
+        for (int e = 0; e < 4; ++e) {
+          const float a = v[2 * e], b = v[2 * e + 1];
+          v[2 * e] = a * c4[e] - b * s4[e];
+          v[2 * e + 1] = b * c4[e] + a * s4[e];
         }
       }
       Typed<T>::store8(out + c, v);
     }
   } else {
-    for (int c = threadIdx.x; c < n; c += 256) Typed<T>::store(out + c, rotated<T>(in, w, r, c, dim, dims, cos, sin));
+    for (int c = lane; c < n; c += 32) Typed<T>::store(out + c, rotated<T>(in, w, r, c, dim, dims, cos, sin));
   }
 }
 
 template <typename T, bool VEC>
-__device__ __forceinline__ float row_square_sum(const T* in, int n) {
+__device__ __forceinline__ float row_square_sum(const T* in, int n, int lane) {
   float ss = 0.f;
   if constexpr (VEC) {
-    for (int c = threadIdx.x * 8; c < n; c += 256 * 8) {
+#pragma unroll 4
+    for (int c = lane * 8; c < n; c += 256) {
       float v[8];
       Typed<T>::load8(in + c, v);
 #pragma unroll
       for (int e = 0; e < 8; ++e) ss += v[e] * v[e];
     }
   } else {
-    for (int c = threadIdx.x; c < n; c += 256) {
+    for (int c = lane; c < n; c += 32) {
       const float v = Typed<T>::load(in + c);
       ss += v * v;
     }
   }
-  return ss;
+  return warp_sum(ss);
 }
 
+// One warp per (token, part): queries, or key and value.
 template <typename T, bool VEC>
-__global__ void __launch_bounds__(256) gqa_prepare_kernel(const GqaPrepArgs p) {
+__global__ void __launch_bounds__(128) gqa_prepare_kernel(const GqaPrepArgs p) {
   pdl_prologue();
-  __shared__ float red[40];
-  const long long row = blockIdx.x;
+  const int parts = p.k_col >= 0 ? 2 : 1, lane = threadIdx.x & 31;
+  const long long w = blockIdx.x * 4ll + (threadIdx.x >> 5);
+  if (w >= (long long)p.B * p.L * parts) return;  // whole warp
+  const long long row = w / parts;
   const int b = int(row / p.L), t = int(row % p.L), pos = p.lengths ? p.lengths[b] : p.pos0 + t;
   const T* in = static_cast<const T*>(p.proj) + row * p.ld;
   const float* cs = p.cos + (long long)pos * (p.dims >> 1);
   const float* sn = p.sin + (long long)pos * (p.dims >> 1);
-  const int nq = p.H * p.dim, nk = p.G * p.dim, nv = p.G * p.vdim;
-  const bool append = p.k_col >= 0 && pos < p.max_len && !(p.active && !p.active[b]);
-  const float sq = row_square_sum<T, VEC>(in, nq), sk = append ? row_square_sum<T, VEC>(in + p.k_col, nk) : 0.f;
-  const float rq = 1.f / sqrtf(block_sum(sq, red) / float(nq) + p.eps);
-  T* q = static_cast<T*>(p.q) + row * p.ldq;
-  norm_rotate_row<T, VEC>(in, p.q_w, rq, nq, p.dim, p.dims, cs, sn, q);
-  for (int c = nq + threadIdx.x; c < p.ldq; c += 256) Typed<T>::store(q + c, 0.f);
-  if (!append) return;  // the whole CTA
-  const float rk = 1.f / sqrtf(block_sum(sk, red) / float(nk) + p.eps);
-  norm_rotate_row<T, VEC>(in + p.k_col, p.k_w, rk, nk, p.dim, p.dims, cs, sn, static_cast<T*>(p.k) + (long long)b * p.k_bs + pos * p.ldk);
+  if (w % parts == 0) {
+    const int nq = p.H * p.dim;
+    const float rq = 1.f / sqrtf(row_square_sum<T, VEC>(in, nq, lane) / float(nq) + p.eps);
+    T* q = static_cast<T*>(p.q) + row * p.ldq;
+    norm_rotate_row<T, VEC>(in, p.q_w, rq, nq, p.dim, p.dims, cs, sn, q, lane);
+    for (int c = nq + lane; c < p.ldq; c += 32) Typed<T>::store(q + c, 0.f);
+    return;
+  }
+  if (pos >= p.max_len || (p.active && !p.active[b])) return;
+  const int nk = p.G * p.dim, nv = p.G * p.vdim;
   T* v = static_cast<T*>(p.v) + (long long)b * p.v_bs + pos * p.ldv;
   if constexpr (VEC) {
-    for (int c = threadIdx.x * 8; c < nv; c += 256 * 8) Typed<T>::store_raw8(v + c, Typed<T>::raw8(in + p.v_col + c));
+    for (int c = lane * 8; c < nv; c += 256) Typed<T>::store_raw8(v + c, Typed<T>::raw8(in + p.v_col + c));
   } else {
-    for (int c = threadIdx.x; c < nv; c += 256) v[c] = in[p.v_col + c];
+    for (int c = lane; c < nv; c += 32) v[c] = in[p.v_col + c];
   }
+  const float rk = 1.f / sqrtf(row_square_sum<T, VEC>(in + p.k_col, nk, lane) / float(nk) + p.eps);
+  norm_rotate_row<T, VEC>(in + p.k_col, p.k_w, rk, nk, p.dim, p.dims, cs, sn, static_cast<T*>(p.k) + (long long)b * p.k_bs + pos * p.ldk, lane);
 }
 
 struct GqaArgs {
@@ -332,14 +344,15 @@ template <typename T>
 static int launch_prepare(const GqaPrepArgs& p, cudaStream_t s) {
   const bool kv = p.k_col >= 0;
   uintptr_t at = reinterpret_cast<uintptr_t>(p.proj) | reinterpret_cast<uintptr_t>(p.q) | reinterpret_cast<uintptr_t>(p.q_w);
-  long long n = p.ld | p.ldq | p.dim;
+  long long n = p.ld | p.ldq | p.dim | p.dims;
+  at |= reinterpret_cast<uintptr_t>(p.cos) | reinterpret_cast<uintptr_t>(p.sin);
   if (kv) {
     at |= reinterpret_cast<uintptr_t>(p.k) | reinterpret_cast<uintptr_t>(p.v) | reinterpret_cast<uintptr_t>(p.k_w);
     n |= p.k_col | p.v_col | p.ldk | p.ldv | p.k_bs | p.v_bs | (long long)p.G * p.vdim;
   }
-  const dim3 grid{unsigned((long long)p.B * p.L)};
-  if (!(at & 15) && !(n & 7)) launch_pdl(gqa_prepare_kernel<T, true>, grid, dim3(256), 0, s, p);
-  else launch_pdl(gqa_prepare_kernel<T, false>, grid, dim3(256), 0, s, p);
+  const dim3 grid{unsigned(((long long)p.B * p.L * (kv ? 2 : 1) + 3) / 4)};
+  if (!(at & 15) && !(n & 7)) launch_pdl(gqa_prepare_kernel<T, true>, grid, dim3(128), 0, s, p);
+  else launch_pdl(gqa_prepare_kernel<T, false>, grid, dim3(128), 0, s, p);
   return int(cudaGetLastError());
 }
 

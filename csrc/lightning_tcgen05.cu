@@ -7,12 +7,13 @@
 // that enters a product -- the state, the decayed scores and the decayed values -- goes in as the sum of two bf16 numbers (16 bits of
 // mantissa).  The state itself stays in fp32 accumulators in tensor memory from the first chunk to the last.
 //
-// Per chunk: Q K^T and Q S (first products) -> group A (warps 0-3) decays and masks the scores, group B (warps 4-7) decays the read-out
-// and the state and writes the decayed values -> P V and K^T V' (second products) -> A stores the outputs while B rewrites the state as
-// the next chunk's operand.  Two CTAs share an SM, so one's products run under the other's arithmetic.
+// Per chunk: Q K^T and Q S (first products) | group A (warps 0-3) decays and masks the scores, block of 32 keys by block, while group B (warps
+// 4-7) writes the decayed values and decays the read-out | K^T V' as soon as the values are there, then P V | B rewrites the state as the
+// next chunk's operand (and leaves it decayed in tensor memory) while P V runs, A stores the outputs.  The next chunk's tiles are
+// prefetched into L2 from the start of a chunk.  Two CTAs share an SM, so one's products run under the other's arithmetic.
 //
-// Tensor memory (256 columns): scores / P 128, read-out 64, state 64 (lanes = state rows).  P overwrites the scores as two sets of 64
-// packed columns.  The state operand and the decayed values share one buffer in turn.
+// Tensor memory (256 columns): scores / P 128, read-out 64, state 64 (lanes = state rows).  The P of 32 keys overwrites their scores: 16
+// packed columns of high parts, 16 of low parts.  The state operand and the decayed values share one buffer in turn.
 // Every wait is bounded (status word + clean unwind); no load uses cluster multicast.
 #include "common.cuh"
 
@@ -35,6 +36,9 @@ constexpr int LS_Q = 0, LS_K = 32768, LS_V = 65536, LS_S = 81920;  // Q, K: two 
 constexpr int LS_AUX = 114688;                                     // powers, barriers
 constexpr int LS_TOTAL = LS_AUX + 1024;
 
+__device__ __forceinline__ void prefetch_3d(const CUtensorMap* map, int c0, int c1, int c2) {  // into L2
+  asm volatile("cp.async.bulk.prefetch.tensor.3d.L2.global [%0, {%1, %2, %3}];" ::"l"(reinterpret_cast<uint64_t>(map)), "r"(c0), "r"(c1), "r"(c2) : "memory");
+}
 // Two values as bf16 pairs hi + lo.
 __device__ __forceinline__ void split_bf16x2(float a, float b, uint32_t& hi, uint32_t& lo) {
   hi = pack_bf16x2(a, b);
@@ -55,11 +59,12 @@ lightning_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
   uint64_t* in_full = bars;       // Q, K, V of a chunk
   uint64_t* s_done = bars + 1;    // scores
   uint64_t* r_done = bars + 2;    // read-out of the state
-  uint64_t* p_ready = bars + 3;   // 8 arrivals: P, decayed read-out, decayed state, decayed values
-  uint64_t* o_done = bars + 4;    // P V
+  uint64_t* v_ready = bars + 3;   // 4 arrivals: decayed values
+  uint64_t* p_ready = bars + 4;   // 8 arrivals: P, decayed read-out
   uint64_t* u_done = bars + 5;    // K^T V'
-  uint64_t* s_ready = bars + 6;   // 8 arrivals: state operand written, outputs taken
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 7);
+  uint64_t* o_done = bars + 6;    // P V (and everything before it)
+  uint64_t* s_ready = bars + 7;   // 8 arrivals: state operand written, state decayed, outputs taken
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 8);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -73,6 +78,7 @@ lightning_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
     mbar_init(in_full, 1);
     mbar_init(s_done, 1);
     mbar_init(r_done, 1);
+    mbar_init(v_ready, 4);
     mbar_init(p_ready, 8);
     mbar_init(o_done, 1);
     mbar_init(u_done, 1);
@@ -119,6 +125,15 @@ lightning_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
       load_kv(0);
       for (int c = 0; c < chunks; ++c) {
         if (!mbar_wait_bounded(in_full, c & 1, abort_flag, p.status, kTimeoutFull)) break;
+        const bool more = c + 1 < chunks;
+        if (more) {
+          const int row = b * p.L + (c + 1) * LC;
+          prefetch_3d(&map_q, 0, h, row);
+          prefetch_3d(&map_q, 64, h, row);
+          prefetch_3d(&map_k, 0, h, row);
+          prefetch_3d(&map_k, 64, h, row);
+          prefetch_3d(&map_v, v0, h, row);
+        }
         if (!mbar_wait_bounded(s_ready, c & 1, abort_flag, p.status, kTimeoutTmemEmpty)) break;
         tc_fence_after();
 #pragma unroll
@@ -133,24 +148,26 @@ lightning_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
           for (int k = 0; k < 8; ++k)
             tc_mma_f16(t_out, desc_advance(q_k, (k >> 2) * 16384 + (k & 3) * 32), desc_advance(s_mn, part * 16384 + k * 2048), id_r, part | k);
         tc_commit(r_done);
-        if (!mbar_wait_bounded(p_ready, c & 1, abort_flag, p.status, kTimeoutTmemFull)) break;
+        if (!mbar_wait_bounded(v_ready, c & 1, abort_flag, p.status, kTimeoutTmemFull)) break;
         tc_fence_after();
-        if (c + 1 < chunks) {  // the products that read Q have completed: both groups waited for them
+        if (more) {  // the products that read Q have completed: group B waited for them
           mbar_expect_tx(in_full, 81920);
           load_q(c + 1);
         }
 #pragma unroll
         for (int part = 0; part < 2; ++part)
 #pragma unroll
-          for (int k = 0; k < 8; ++k) tc_mma_f16_ts(t_out, t_scores + part * 64 + k * 8, desc_advance(v_mn, k * 2048), id_r, 1);
-        tc_commit(o_done);
+          for (int k = 0; k < 8; ++k) tc_mma_f16(t_state, desc_advance(k_mn, k * 2048), desc_advance(s_mn, part * 16384 + k * 2048), id_u, 1);
+        tc_commit(u_done);
+        if (!mbar_wait_bounded(p_ready, c & 1, abort_flag, p.status, kTimeoutTmemFull)) break;
+        tc_fence_after();
 #pragma unroll
         for (int part = 0; part < 2; ++part)
 #pragma unroll
-          for (int k = 0; k < 8; ++k) tc_mma_f16(t_state, desc_advance(k_mn, k * 2048), desc_advance(s_mn, part * 16384 + k * 2048), id_u, 1);
-        tc_commit(u_done);
-        if (c + 1 < chunks) {
-          if (!mbar_wait_bounded(u_done, c & 1, abort_flag, p.status, kTimeoutTmemFull)) break;
+          for (int k = 0; k < 8; ++k) tc_mma_f16_ts(t_out, t_scores + (k >> 1) * 32 + part * 16 + (k & 1) * 8, desc_advance(v_mn, k * 2048), id_r, 1);
+        tc_commit(o_done);
+        if (more) {
+          if (!mbar_wait_bounded(o_done, c & 1, abort_flag, p.status, kTimeoutTmemFull)) break;
           load_kv(c + 1);
         }
       }
@@ -190,6 +207,9 @@ lightning_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
           f[e] = t.x; f[e + 1] = t.y; f[e + 2] = t.z; f[e + 3] = t.w;
         }
         put16(q, f);
+        const float fs = s_pow[min(LC, p.L)];
+#pragma unroll
+        for (int e = 0; e < 16; ++e) f[e] *= fs;
         tmem_st_32x16(t_state + lane_base + 16 * q, reinterpret_cast<uint32_t(&)[16]>(f));
       }
       tmem_st_wait();
@@ -204,44 +224,32 @@ lightning_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
       if (warp < 4) {
         // ---------------------------------------------------------------- group A: P = decayed, masked scores
         if (!mbar_wait_bounded(s_done, c & 1, abort_flag, p.status, kTimeoutTmemFull)) break;
-        // (the loads of Q for the next chunk start after p_ready: both products that read Q must be behind it)
-        if (!mbar_wait_bounded(r_done, c & 1, abort_flag, p.status, kTimeoutTmemFull)) break;
         tc_fence_after();
-        const uint32_t t_s = t_scores + lane_base;
-        // Blocks of 32 keys, last first: a block's scores are read before anything overwrites them (hi of block k goes to columns
-        // 16 k, lo to 64 + 16 k; the hi parts of blocks 3 and 2 wait until block 1 has been read).
-        uint32_t hi3[16], hi2[16], hi1[16];
-        auto block = [&](int k, uint32_t (&hi)[16]) {
-          uint32_t lo[16];
+#pragma unroll 1
+        for (int k = 0; k < 4; ++k) {   // 32 keys
+          const uint32_t at = t_scores + lane_base + 32 * k;
+          uint32_t pk[32];              // 16 high, 16 low
           if (k > warp) {  // all keys after all of this warp's queries
 #pragma unroll
-            for (int e = 0; e < 16; ++e) hi[e] = lo[e] = 0u;
+            for (int e = 0; e < 32; ++e) pk[e] = 0u;
           } else {
             uint32_t s[32];
-            tmem_ld_32x32(t_s + 32 * k, s);
+            tmem_ld_32x32(at, s);
             tmem_ld_wait();
             if (k < warp) {
               const float f = s_pow[r - 32 * k - 31];
 #pragma unroll
               for (int e = 0; e < 16; ++e)
-                split_bf16x2(__uint_as_float(s[2 * e]) * (f * s_pow[31 - 2 * e]), __uint_as_float(s[2 * e + 1]) * (f * s_pow[30 - 2 * e]), hi[e], lo[e]);
+                split_bf16x2(__uint_as_float(s[2 * e]) * (f * s_pow[31 - 2 * e]), __uint_as_float(s[2 * e + 1]) * (f * s_pow[30 - 2 * e]), pk[e], pk[16 + e]);
             } else {
 #pragma unroll
               for (int e = 0; e < 16; ++e)
                 split_bf16x2(2 * e <= lane ? __uint_as_float(s[2 * e]) * s_pow[max(lane - 2 * e, 0)] : 0.f,
-                             2 * e + 1 <= lane ? __uint_as_float(s[2 * e + 1]) * s_pow[max(lane - 2 * e - 1, 0)] : 0.f, hi[e], lo[e]);
+                             2 * e + 1 <= lane ? __uint_as_float(s[2 * e + 1]) * s_pow[max(lane - 2 * e - 1, 0)] : 0.f, pk[e], pk[16 + e]);
             }
           }
-          tmem_st_32x16(t_s + 64 + 16 * k, lo);
-        };
-        block(3, hi3);
-        block(2, hi2);
-        block(1, hi1);
-        tmem_st_32x16(t_s + 48, hi3);
-        tmem_st_32x16(t_s + 32, hi2);
-        block(0, hi2);
-        tmem_st_32x16(t_s + 16, hi1);
-        tmem_st_32x16(t_s, hi2);
+          tmem_st_32x32(at, pk);
+        }
         tmem_st_wait();
         tc_fence_before();
         __syncwarp();
@@ -250,80 +258,91 @@ lightning_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
         if (!mbar_wait_bounded(o_done, c & 1, abort_flag, p.status, kTimeoutTmemFull)) break;
         tc_fence_after();
         __nv_bfloat16* orow = p.o + ((long long)b * p.L + c * LC + r) * p.ldo + (long long)h * p.vdim + v0;
-#pragma unroll
-        for (int q = 0; q < 2; ++q) {
-          uint32_t f[32];
-          tmem_ld_32x32(t_out + lane_base + 32 * q, f);
-          tmem_ld_wait();
-          if (r < n) {
-#pragma unroll
-            for (int e = 0; e < 4; ++e)
-              if (32 * q + 8 * e < cols)
-                *reinterpret_cast<uint4*>(orow + 32 * q + 8 * e) =
-                    make_uint4(pack_bf16x2(__uint_as_float(f[8 * e]), __uint_as_float(f[8 * e + 1])),
-                               pack_bf16x2(__uint_as_float(f[8 * e + 2]), __uint_as_float(f[8 * e + 3])),
-                               pack_bf16x2(__uint_as_float(f[8 * e + 4]), __uint_as_float(f[8 * e + 5])),
-                               pack_bf16x2(__uint_as_float(f[8 * e + 6]), __uint_as_float(f[8 * e + 7])));
-          }
-        }
+        uint32_t f[64];
+        tmem_ld_32x32(t_out + lane_base, reinterpret_cast<uint32_t(&)[32]>(f[0]));
+        tmem_ld_32x32(t_out + lane_base + 32, reinterpret_cast<uint32_t(&)[32]>(f[32]));
+        tmem_ld_wait();
         tc_fence_before();
         __syncwarp();
         if (lane == 0) mbar_arrive(s_ready);
+        if (r < n) {
+#pragma unroll
+          for (int e = 0; e < 64; e += 8)
+            if (e < cols)
+              *reinterpret_cast<uint4*>(orow + e) =
+                  make_uint4(pack_bf16x2(__uint_as_float(f[e]), __uint_as_float(f[e + 1])), pack_bf16x2(__uint_as_float(f[e + 2]), __uint_as_float(f[e + 3])),
+                             pack_bf16x2(__uint_as_float(f[e + 4]), __uint_as_float(f[e + 5])), pack_bf16x2(__uint_as_float(f[e + 6]), __uint_as_float(f[e + 7])));
+        }
       } else {
-        // ---------------------------------------------------------------- group B: read-out, state, values
-        if (!mbar_wait_bounded(r_done, c & 1, abort_flag, p.status, kTimeoutTmemFull)) break;
+        // ---------------------------------------------------------------- group B: values
+        if (!mbar_wait_bounded(in_full, c & 1, abort_flag, p.status, kTimeoutFull)) break;
+        const float fo = s_pow[r + 1], fv = r < n ? s_pow[n - 1 - r] : 0.f;
+        const uint8_t* vrow = sV + r * 128;
+        {
+          uint32_t hi[32], lo[32];
+#pragma unroll
+          for (int u = 0; u < 8; ++u) {
+            const uint4 w = *reinterpret_cast<const uint4*>(vrow + ((uint32_t(u) << 4) ^ swz));
+            const uint32_t x[4] = {w.x, w.y, w.z, w.w};
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+              const float2 t = unpack_bf16x2(x[e]);
+              split_bf16x2(r < n ? t.x * fv : 0.f, r < n ? t.y * fv : 0.f, hi[4 * u + e], lo[4 * u + e]);
+            }
+          }
+          // the buffer is free once the read-out of the state is done
+          if (!mbar_wait_bounded(r_done, c & 1, abort_flag, p.status, kTimeoutTmemFull)) break;
+#pragma unroll
+          for (int u = 0; u < 8; ++u) {
+            const uint32_t at = (uint32_t(u) << 4) ^ swz;
+            *reinterpret_cast<uint4*>(my_hi + at) = make_uint4(hi[4 * u], hi[4 * u + 1], hi[4 * u + 2], hi[4 * u + 3]);
+            *reinterpret_cast<uint4*>(my_lo + at) = make_uint4(lo[4 * u], lo[4 * u + 1], lo[4 * u + 2], lo[4 * u + 3]);
+          }
+          fence_proxy_async_smem();
+          __syncwarp();
+          if (lane == 0) mbar_arrive(v_ready);
+        }
+        // ---------------------------------------------------------------- read-out
         tc_fence_after();
-        const float fo = s_pow[r + 1], fs = s_pow[n], fv = r < n ? s_pow[n - 1 - r] : 0.f;
-#pragma unroll 1
-        for (int q = 0; q < 8; ++q) {   // four pieces of the read-out, four of the state
-          const uint32_t at = (q < 4 ? t_out : t_state) + lane_base + 16 * (q & 3);
-          const float f = q < 4 ? fo : fs;
-          uint32_t x[16];
-          tmem_ld_32x16(at, x);
+        {
+          uint32_t x[64];
+          tmem_ld_32x32(t_out + lane_base, reinterpret_cast<uint32_t(&)[32]>(x[0]));
+          tmem_ld_32x32(t_out + lane_base + 32, reinterpret_cast<uint32_t(&)[32]>(x[32]));
           tmem_ld_wait();
 #pragma unroll
-          for (int e = 0; e < 16; ++e) x[e] = __float_as_uint(__uint_as_float(x[e]) * f);
-          tmem_st_32x16(at, x);
+          for (int e = 0; e < 64; ++e) x[e] = __float_as_uint(__uint_as_float(x[e]) * fo);
+          tmem_st_32x32(t_out + lane_base, reinterpret_cast<uint32_t(&)[32]>(x[0]));
+          tmem_st_32x32(t_out + lane_base + 32, reinterpret_cast<uint32_t(&)[32]>(x[32]));
+          tmem_st_wait();
         }
-        if (!mbar_wait_bounded(in_full, c & 1, abort_flag, p.status, kTimeoutFull)) break;  // (complete already: r_done came after it)
-        const uint8_t* vrow = sV + r * 128;
-#pragma unroll 1
-        for (int q = 0; q < 4; ++q) {
-          float f[16];
-#pragma unroll
-          for (int u = 0; u < 2; ++u) {
-            const uint4 w = *reinterpret_cast<const uint4*>(vrow + ((uint32_t(2 * q + u) << 4) ^ swz));
-            const float2 a = unpack_bf16x2(w.x), b2 = unpack_bf16x2(w.y), c2 = unpack_bf16x2(w.z), d2 = unpack_bf16x2(w.w);
-            f[8 * u] = a.x; f[8 * u + 1] = a.y; f[8 * u + 2] = b2.x; f[8 * u + 3] = b2.y;
-            f[8 * u + 4] = c2.x; f[8 * u + 5] = c2.y; f[8 * u + 6] = d2.x; f[8 * u + 7] = d2.y;
-          }
-#pragma unroll
-          for (int e = 0; e < 16; ++e) f[e] = r < n ? f[e] * fv : 0.f;
-          put16(q, f);
-        }
-        tmem_st_wait();
         tc_fence_before();
-        fence_proxy_async_smem();
         __syncwarp();
         if (lane == 0) mbar_arrive(p_ready);
         // ---------------------------------------------------------------- the state as the next chunk's operand
         if (!mbar_wait_bounded(u_done, c & 1, abort_flag, p.status, kTimeoutTmemFull)) break;
         tc_fence_after();
         const bool end = c + 1 == chunks;
-#pragma unroll 1
-        for (int q = 0; q < 4; ++q) {
-          uint32_t x[16];
-          tmem_ld_32x16(t_state + lane_base + 16 * q, x);
+        const float fs = end ? 1.f : s_pow[min(LC, p.L - (c + 1) * LC)];
+#pragma unroll
+        for (int q = 0; q < 2; ++q) {
+          uint32_t x[32];
+          tmem_ld_32x32(t_state + lane_base + 32 * q, x);
           tmem_ld_wait();
-          float(&f)[16] = reinterpret_cast<float(&)[16]>(x);
           if (!end) {
-            put16(q, f);
+#pragma unroll
+            for (int u = 0; u < 2; ++u) put16(2 * q + u, reinterpret_cast<float(&)[16]>(x[16 * u]));
+#pragma unroll
+            for (int e = 0; e < 32; ++e) x[e] = __float_as_uint(__uint_as_float(x[e]) * fs);
+            tmem_st_32x32(t_state + lane_base + 32 * q, x);
           } else if (r < p.dim) {
 #pragma unroll
-            for (int e = 0; e < 16; e += 4)
-              if (16 * q + e < cols) *reinterpret_cast<float4*>(st + 16 * q + e) = make_float4(f[e], f[e + 1], f[e + 2], f[e + 3]);
+            for (int e = 0; e < 32; e += 4)
+              if (32 * q + e < cols)
+                *reinterpret_cast<float4*>(st + 32 * q + e) =
+                    make_float4(__uint_as_float(x[e]), __uint_as_float(x[e + 1]), __uint_as_float(x[e + 2]), __uint_as_float(x[e + 3]));
           }
         }
+        tmem_st_wait();
         tc_fence_before();
         fence_proxy_async_smem();
         __syncwarp();
