@@ -68,6 +68,7 @@ class RotaryEmbedding(nn.Module):
     def __init__(self, dim: int, max_position: int = 2048, theta: float = 10000.0, scaling_factor: float = 1.0):
         super().__init__()
         self.dim, self.theta, self.scaling_factor = dim, theta, scaling_factor
+        self._outgrown: List[Tuple[torch.Tensor, torch.Tensor]] = []
         cos, sin = ops.rope_tables(max_position, dim, theta, scaling_factor)
         self.register_buffer("cos", cos, persistent=False)
         self.register_buffer("sin", sin, persistent=False)
@@ -79,6 +80,7 @@ class RotaryEmbedding(nn.Module):
             if length > self.cos.shape[0]:
                 n = max(length, 2 * self.cos.shape[0])
             cos, sin = ops.rope_tables(n, self.dim, self.theta, self.scaling_factor, device)
+            self._outgrown.append((self.cos, self.sin))   # captured decode steps keep reading the tables they were captured with
             self.cos, self.sin = cos, sin
 
     def forward(self, length: int, device=None) -> Tuple[torch.Tensor, torch.Tensor]:

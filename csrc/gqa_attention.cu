@@ -7,7 +7,7 @@
 // The cache holds k [B, max_len, ldk] as the scores use it (normed and rotated) and v [B, max_len, ldv]; a layer that shares another
 // layer's keys and values reads that layer's cache and prepares only its queries.
 //
-// * gqa_prepare: norm, rotation, cache append, one warp per token for the queries and one for key and value.
+// * gqa_prepare: norm, rotation, cache append; a warp (few tokens: a CTA) for a token's queries and one for its key and value.
 // * gqa_portion: L queries of a prompt at positions pos0 .. against the cache, any sizes, bf16 and fp32 (gqa_attention_tcgen05.cu is the
 //   tensor-core form).
 // * gqa_decode + gqa_merge: one query token per sequence, any sizes (decode_attn_mma_kernel in inference.cu serves bf16 heads of 64 and 128).
@@ -54,14 +54,14 @@ __device__ __forceinline__ float rotated(const T* in, const float* w, float r, i
   return (d & 1) ? x * cos[m] + y * sin[m] : x * cos[m] - y * sin[m];
 }
 
-// One warp's row of n values: out = rotate(in r w).  VEC: dim, dims multiples of 8, so that eight consecutive values belong to one head and
-// are rotated or pass as a whole.
+// One row of n values by `threads` threads: out = rotate(in r w).  VEC: dim, dims multiples of 8, so that eight consecutive values belong to one
+// head and are rotated or pass as a whole.
 template <typename T, bool VEC>
 __device__ __forceinline__ void norm_rotate_row(const T* in, const float* w, float r, int n, int dim, int dims, const float* cos, const float* sin, T* out,
-                                                int lane) {
+                                                int id, int threads) {
   if constexpr (VEC) {
 #pragma unroll 4
-    for (int c = lane * 8; c < n; c += 256) {
+    for (int c = id * 8; c < n; c += 8 * threads) {
       float v[8], g[8];
       Typed<T>::load8(in + c, v);
       Typed<float>::load8(w + c, g);
@@ -81,37 +81,43 @@ __device__ __forceinline__ void norm_rotate_row(const T* in, const float* w, flo
       Typed<T>::store8(out + c, v);
     }
   } else {
-    for (int c = lane; c < n; c += 32) Typed<T>::store(out + c, rotated<T>(in, w, r, c, dim, dims, cos, sin));
+    for (int c = id; c < n; c += threads) Typed<T>::store(out + c, rotated<T>(in, w, r, c, dim, dims, cos, sin));
   }
 }
 
 template <typename T, bool VEC>
-__device__ __forceinline__ float row_square_sum(const T* in, int n, int lane) {
+__device__ __forceinline__ float row_square_sum(const T* in, int n, int id, int threads) {
   float ss = 0.f;
   if constexpr (VEC) {
 #pragma unroll 4
-    for (int c = lane * 8; c < n; c += 256) {
+    for (int c = id * 8; c < n; c += 8 * threads) {
       float v[8];
       Typed<T>::load8(in + c, v);
 #pragma unroll
       for (int e = 0; e < 8; ++e) ss += v[e] * v[e];
     }
   } else {
-    for (int c = lane; c < n; c += 32) {
+    for (int c = id; c < n; c += threads) {
       const float v = Typed<T>::load(in + c);
       ss += v * v;
     }
   }
-  return warp_sum(ss);
+  return ss;
 }
 
-// One warp per (token, part): queries, or key and value.
-template <typename T, bool VEC>
+// One warp (WPR = 1) or one CTA of four (WPR = 4, for a handful of tokens) per (token, part): queries, or key and value.
+template <typename T, bool VEC, int WPR>
 __global__ void __launch_bounds__(128) gqa_prepare_kernel(const GqaPrepArgs p) {
   pdl_prologue();
-  const int parts = p.k_col >= 0 ? 2 : 1, lane = threadIdx.x & 31;
-  const long long w = blockIdx.x * 4ll + (threadIdx.x >> 5);
-  if (w >= (long long)p.B * p.L * parts) return;  // whole warp
+  __shared__ float red[40];
+  constexpr int threads = 32 * WPR;
+  const int parts = p.k_col >= 0 ? 2 : 1, id = threadIdx.x % threads;
+  const long long w = WPR == 4 ? blockIdx.x : blockIdx.x * 4ll + (threadIdx.x >> 5);
+  if (w >= (long long)p.B * p.L * parts) return;  // whole warp, or whole CTA
+  auto sum = [&](float v) {
+    if constexpr (WPR == 4) return block_sum(v, red);
+    else return warp_sum(v);
+  };
   const long long row = w / parts;
   const int b = int(row / p.L), t = int(row % p.L), pos = p.lengths ? p.lengths[b] : p.pos0 + t;
   const T* in = static_cast<const T*>(p.proj) + row * p.ld;
@@ -119,22 +125,22 @@ __global__ void __launch_bounds__(128) gqa_prepare_kernel(const GqaPrepArgs p) {
   const float* sn = p.sin + (long long)pos * (p.dims >> 1);
   if (w % parts == 0) {
     const int nq = p.H * p.dim;
-    const float rq = 1.f / sqrtf(row_square_sum<T, VEC>(in, nq, lane) / float(nq) + p.eps);
+    const float rq = 1.f / sqrtf(sum(row_square_sum<T, VEC>(in, nq, id, threads)) / float(nq) + p.eps);
     T* q = static_cast<T*>(p.q) + row * p.ldq;
-    norm_rotate_row<T, VEC>(in, p.q_w, rq, nq, p.dim, p.dims, cs, sn, q, lane);
-    for (int c = nq + lane; c < p.ldq; c += 32) Typed<T>::store(q + c, 0.f);
+    norm_rotate_row<T, VEC>(in, p.q_w, rq, nq, p.dim, p.dims, cs, sn, q, id, threads);
+    for (int c = nq + id; c < p.ldq; c += threads) Typed<T>::store(q + c, 0.f);
     return;
   }
   if (pos >= p.max_len || (p.active && !p.active[b])) return;
   const int nk = p.G * p.dim, nv = p.G * p.vdim;
   T* v = static_cast<T*>(p.v) + (long long)b * p.v_bs + pos * p.ldv;
   if constexpr (VEC) {
-    for (int c = lane * 8; c < nv; c += 256) Typed<T>::store_raw8(v + c, Typed<T>::raw8(in + p.v_col + c));
+    for (int c = id * 8; c < nv; c += 8 * threads) Typed<T>::store_raw8(v + c, Typed<T>::raw8(in + p.v_col + c));
   } else {
-    for (int c = lane; c < nv; c += 32) v[c] = in[p.v_col + c];
+    for (int c = id; c < nv; c += threads) v[c] = in[p.v_col + c];
   }
-  const float rk = 1.f / sqrtf(row_square_sum<T, VEC>(in + p.k_col, nk, lane) / float(nk) + p.eps);
-  norm_rotate_row<T, VEC>(in + p.k_col, p.k_w, rk, nk, p.dim, p.dims, cs, sn, static_cast<T*>(p.k) + (long long)b * p.k_bs + pos * p.ldk, lane);
+  const float rk = 1.f / sqrtf(sum(row_square_sum<T, VEC>(in + p.k_col, nk, id, threads)) / float(nk) + p.eps);
+  norm_rotate_row<T, VEC>(in + p.k_col, p.k_w, rk, nk, p.dim, p.dims, cs, sn, static_cast<T*>(p.k) + (long long)b * p.k_bs + pos * p.ldk, id, threads);
 }
 
 struct GqaArgs {
@@ -350,9 +356,13 @@ static int launch_prepare(const GqaPrepArgs& p, cudaStream_t s) {
     at |= reinterpret_cast<uintptr_t>(p.k) | reinterpret_cast<uintptr_t>(p.v) | reinterpret_cast<uintptr_t>(p.k_w);
     n |= p.k_col | p.v_col | p.ldk | p.ldv | p.k_bs | p.v_bs | (long long)p.G * p.vdim;
   }
-  const dim3 grid{unsigned(((long long)p.B * p.L * (kv ? 2 : 1) + 3) / 4)};
-  if (!(at & 15) && !(n & 7)) launch_pdl(gqa_prepare_kernel<T, true>, grid, dim3(128), 0, s, p);
-  else launch_pdl(gqa_prepare_kernel<T, false>, grid, dim3(128), 0, s, p);
+  const long long units = (long long)p.B * p.L * (kv ? 2 : 1);
+  const bool vec = !(at & 15) && !(n & 7), few = units <= 1024;
+  const dim3 grid{unsigned(few ? units : (units + 3) / 4)}, block(128);
+  if (vec && few) launch_pdl(gqa_prepare_kernel<T, true, 4>, grid, block, 0, s, p);
+  else if (vec) launch_pdl(gqa_prepare_kernel<T, true, 1>, grid, block, 0, s, p);
+  else if (few) launch_pdl(gqa_prepare_kernel<T, false, 4>, grid, block, 0, s, p);
+  else launch_pdl(gqa_prepare_kernel<T, false, 1>, grid, block, 0, s, p);
   return int(cudaGetLastError());
 }
 

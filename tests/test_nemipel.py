@@ -21,6 +21,7 @@ from adaptivetrainingsystem_b200.ops import lightning as lightning_ops
 from adaptivetrainingsystem_b200.ops import postnorm as pn
 from layered_utils import EXACT, PLACES, TOL, close, gpu, position_errors, run_portions, tokens
 
+GPU_PLACES = PLACES[1:]
 ALONE, WHOLE = 0.3, 0.6   # of the shared tolerance: one layer, and the mixed model (whose weight of the residual keeps roundings from growing)
 
 
@@ -190,6 +191,24 @@ def test_prepare_norms_rotates_and_appends(device, dtype):
             rows = [i for i in range(n) if (b, i) != (1, 5)]
             assert worst(k[b, rows, :G * dim].float(), O.rotate_pairs(kn, rot, 70.0).reshape(n, -1)[rows]) < tol
             assert torch.equal(v[b, rows, :G * vdim].cpu(), proj[b, rows, s.v_col:s.v_col + G * vdim])
+
+
+@pytest.mark.parametrize("device,dtype", GPU_PLACES)
+@pytest.mark.parametrize("dim,rot", [(16, 8), (10, 4)])
+def test_prepare_long_and_short_portions_agree(device, dtype, dim, rot):
+    """Many tokens and a handful of tokens are distributed over threads differently."""
+    s = gqa_ops.GqaShape(4, 2, dim, 24, rot, 1.0, 0.0, 1e-3)
+    n, g = 700, torch.Generator().manual_seed(1)
+    proj = torch.randn(2, n, s.proj_width, generator=g).to(dtype).to(device)
+    ang = torch.arange(n + 1).double()[:, None] * 50.0 ** (-torch.arange(0, rot, 2).double() / rot)
+    consts = (s, torch.rand(4 * dim, generator=g).to(device), torch.rand(2 * dim, generator=g).to(device), ang.cos().float().to(device), ang.sin().float().to(device))
+    results = []
+    for step in (n, 100):
+        k, v = torch.zeros(2, n, s.k_pad, dtype=dtype, device=device), torch.zeros(2, n, s.v_pad, dtype=dtype, device=device)
+        q = [gqa_ops.gqa_prepare(proj[:, i:i + step].contiguous(), *consts, k, v, pos0=i).view(2, step, -1) for i in range(0, n, step)]
+        results.append((torch.cat(q, 1).float(), k.float(), v.float()))
+    for x, y in zip(*results):
+        assert float((x - y).abs().max()) < (1e-5 if dtype == torch.float32 else 4e-2)
 
 
 @pytest.mark.parametrize("device,dtype", PLACES)
