@@ -49,10 +49,10 @@ def nemipel_config(size: str):
 
     def attn(**kw):
         return {"type": "attention", "mlp": mlp, "mixer": {"heads": H, "kv_heads": H // 4, "dim": 128, "vdim": 128, "rot": {"base": 10000.0, "dims": 64},
-                                                            "scale": 128 ** -0.5, "softcap": 30.0, **kw}}
+                                                            "scale": 128 ** -0.5, "softcap": 25.0, **kw}}
     layers = [light, attn(), rec, light, attn(kv_from=1), rec, light, attn()]
     assert len(layers) == LAYERS
-    return NemipelConfig.from_dict({"vocab": VOCAB, "width": z["width"], "norm": {"eps": 1e-6}, "postln_alpha": 3.0, "logit_softcap": 30.0, "layers": layers})
+    return NemipelConfig.from_dict({"vocab": VOCAB, "width": z["width"], "norm": {"eps": 1e-6}, "postln_alpha": 2.0, "logit_softcap": 20.0, "layers": layers})
 
 
 def dense_config(size: str, seq: int):
@@ -142,7 +142,7 @@ FP32_FLOPS = 148 * 128 * 2 * 1.965e9   # nominal: 128 FMA lanes per SM (the recu
 
 
 class _Timer:
-    def __init__(self, dev, iters: int = 10):
+    def __init__(self, dev, iters: int = 20):
         self.flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
         self.iters, self.peak, self.rows = iters, peaks(), []
 
@@ -345,7 +345,7 @@ def _nemipel_kernels(t: _Timer, size: str, B: int, L: int, n: int) -> None:
     t.add(name, "decode delta_step", lambda: D.delta_step(mx, rl, gbd, dd["S"], wd[:, d.g_col:], rec.norm, d, lengths, active, wd, rec.neg_rate, rec.dt_bias),
           2 * n * state)
     lg = torch.randn(n, VOCAB, device=dev)
-    t.add(name, "decode softcap of the logits", lambda: pn.softcap_(lg, 30.0, True), 8.0 * n * VOCAB)
+    t.add(name, "decode softcap of the logits", lambda: pn.softcap_(lg, 20.0, True), 8.0 * n * VOCAB)
     ops.check_status()
 
 

@@ -2,7 +2,7 @@
 capped scores (optionally on another layer's keys and values), a gated delta rule with one decay per state row -- and whose norms follow
 the residual sum.
 
-    x <- norm1(alpha x + mixer(x));   x <- norm2(alpha x + mlp(x));   logits = cap tanh(head norm(x) / cap)
+    f = mixer, then feed-forward:   x <- rms(alpha x + f(x)) w_f;       logits = cap tanh(W rms(x) w / cap)
 
 There is no norm in front of a sublayer: it reads x itself.  One launch per sublayer folds the output product, adds, normalises and
 leaves both the fp32 residual and the next product's input (:func:`~..ops.postnorm.linear_postnorm`); the last one applies the

@@ -38,7 +38,7 @@ struct DecodeArgs {
   __nv_bfloat16* out;  // [B, Hq * D]
   int* chunk_done;     // [B, Hkv] arrival counters (zero between launches) or nullptr: the last CTA of a (sequence, KV head) merges
   // k_new == nullptr: the cache holds the new token's row already.  cap > 0: scores become cap tanh(score / cap).  gate ([B, ld_gate] + head
-  // or null): head h's output is multiplied by sigmoid(gate).  out rows are ld_out elements apart.  (decode_attn_mma_kernel only)
+  // or null): sigmoid(gate) scales the head's output.  out rows are ld_out elements apart.  (decode_attn_mma_kernel only)
   float cap;
   const __nv_bfloat16* gate;
   long long ld_gate, ld_out;
